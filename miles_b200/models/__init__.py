@@ -5,9 +5,19 @@ from .torch_impl import InferMeta, TorchQwen3  # noqa: F401
 
 
 def build_model(cfg, store, backend: str = "auto", ep=None, tp=None):
-    """``backend``: "b200" (hand-written kernels, CUDA bf16), "torch" (reference ops) or "auto"."""
+    """``backend``: "b200" (hand-written kernels, CUDA; bf16, planned layers also fp32), "torch" (reference ops) or "auto"."""
     import torch
 
+    if cfg.plan is not None:
+        if (tp is not None and tp.n > 1) or ep is not None:
+            raise NotImplementedError("models with a layer plan run without tensor or expert parallelism")
+        if backend == "torch" or (backend == "auto" and store.device.type != "cuda"):
+            from .torch_hybrid import TorchHybrid
+
+            return TorchHybrid(cfg, store)
+        from .b200_hybrid import B200Hybrid
+
+        return B200Hybrid(cfg, store)
     if backend == "auto":
         backend = "b200" if (store.device.type == "cuda" and store.dtype == torch.bfloat16 and cfg.head_dim == 128) else "torch"
     if backend == "b200":

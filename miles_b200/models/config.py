@@ -12,6 +12,8 @@ from dataclasses import asdict, dataclass, field
 from pathlib import Path
 from typing import Any, Optional
 
+from .layer_plan import DESIGNS, LayerPlan, plan_specs, read_plan, write_plan
+
 
 @dataclass
 class ModelConfig:
@@ -61,6 +63,9 @@ class ModelConfig:
     rope_scaling: Optional[dict] = None
     hf_architecture: str = "Qwen3ForCausalLM"
     extra: dict[str, Any] = field(default_factory=dict)
+    # models whose layers differ from one another: mixers, sizes and constants layer by layer (models/layer_plan.py). The
+    # flat attention / MLP fields above then describe nothing
+    plan: Optional[LayerPlan] = None
 
     @property
     def is_moe(self) -> bool:
@@ -82,6 +87,14 @@ class ModelConfig:
         return self.is_moe and i >= self.first_dense_layers and ((i + 1) % self.moe_layer_freq == 0)
 
     def num_params(self) -> int:
+        if self.plan is not None:
+            n = 0
+            for _, shape, _ in plan_specs(self.plan, self.vocab_size, self.hidden_size, 0, self.num_layers, True, True):
+                k = 1
+                for d in shape:
+                    k *= d
+                n += k
+            return n
         n = self.vocab_size * self.hidden_size * (1 if self.tie_embeddings else 2) + self.hidden_size
         for i in range(self.num_layers):
             n += (4 if self.post_norms else 2) * self.hidden_size + self.qkv_dim * self.hidden_size + self.q_dim * self.hidden_size
@@ -113,9 +126,13 @@ class ModelConfig:
     @property
     def family(self) -> str:
         """The HuggingFace ``model_type`` of this architecture (decides config keys and tensor names)."""
+        if self.plan is not None:
+            return self.plan.design.lower()
         return HF_FAMILIES.get(self.hf_architecture, "qwen3_moe" if self.is_moe else "qwen3")
 
     def to_hf_config(self) -> dict:
+        if self.plan is not None:
+            return write_plan(self.plan, self.vocab_size, self.hidden_size)
         cfg = {
             "architectures": [self.hf_architecture],
             "model_type": self.family,
@@ -168,19 +185,27 @@ class ModelConfig:
         return cfg
 
     @classmethod
+    def from_plan(cls, plan: LayerPlan, vocab: int, width: int, name: str | None = None) -> "ModelConfig":
+        return cls(name=name or plan.design, num_layers=len(plan.layers), hidden_size=width, vocab_size=vocab, rms_eps=plan.eps,
+                   num_q_heads=0, num_kv_heads=0, head_dim=0, ffn_hidden_size=0, qk_norm=False, hf_architecture=plan.design, plan=plan,
+                   max_position_embeddings=1 << 20)
+
+    @classmethod
     def from_hf_config(cls, cfg: dict | str | Path, name: str | None = None) -> "ModelConfig":
         if not isinstance(cfg, dict):
             p = Path(cfg)
             if p.is_dir():
                 p = p / "config.json"
             cfg = json.loads(p.read_text())
+        if cfg.get("architecture") in DESIGNS:
+            return cls.from_plan(*read_plan(cfg), name=name)
         arch = (cfg.get("architectures") or ["Qwen3ForCausalLM"])[0]
         heads = cfg["num_attention_heads"]
         head_dim = cfg.get("head_dim") or cfg["hidden_size"] // heads
         mtype = (cfg.get("model_type") or HF_FAMILIES.get(arch, "qwen3")).lower()
         if arch not in HF_FAMILIES:
             raise NotImplementedError(f"{arch} ({mtype}) is not one of the architectures this package implements: "
-                                      f"{', '.join(sorted(HF_FAMILIES))}")
+                                      f"{', '.join(sorted([*HF_FAMILIES, *DESIGNS]))}")
         is_qwen3 = "qwen3" in mtype
         mlp_only = cfg.get("mlp_only_layers") or []
         n_experts = cfg.get("num_experts", 0) or cfg.get("num_local_experts", 0) or cfg.get("n_routed_experts", 0) or 0

@@ -19,6 +19,10 @@ from .config import ModelConfig
 
 def to_hf(cfg: ModelConfig, name: str, t: torch.Tensor, expert_offset: int = 0) -> list:
     """One native tensor -> list of (hf_name, tensor view)."""
+    if getattr(cfg, "plan", None) is not None:
+        from .layer_plan import plan_to_checkpoint
+
+        return plan_to_checkpoint(cfg.plan, name, t)
     if name == "embed.weight":
         return [("model.embed_tokens.weight", t)]
     if name == "final_norm.weight":

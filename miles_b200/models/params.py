@@ -16,6 +16,8 @@ Native parameter names::
     layers.i.moe.router.weight [E,H]          layers.i.moe.w1 [E_local,2I,H]   layers.i.moe.w2 [E_local,H,I]
     layers.i.moe.router.bias [E] (sigmoid routers)     layers.i.moe.shared.gate_up.weight [2Is,H]   ...shared.down.weight [H,Is]
 
+Models with a layer plan have the names of ``layer_plan.plan_specs`` instead.
+
 The fused layouts (q|k|v rows, gate|up rows) are what the fused kernels consume; ``hf_mapping`` converts
 to and from HuggingFace names, the role that megatron_to_hf/qwen3moe.py:6-117 plays in the reference.
 """
@@ -60,6 +62,15 @@ def build_specs(cfg: ModelConfig, ep_size: int = 1, layers: Optional[tuple] = No
     H, D = cfg.hidden_size, cfg.head_dim
     lo, hi = layers if layers is not None else (0, cfg.num_layers)
     specs: list[ParamSpec] = []
+    if cfg.plan is not None:
+        from .layer_plan import plan_specs
+
+        specs = [ParamSpec(n, s, "dense", init) for n, s, init in plan_specs(cfg.plan, cfg.vocab_size, H, lo, hi, first, last)]
+        off = 0
+        for s in specs:
+            s.offset = off
+            off += _align(s.numel)
+        return specs
     if first or (last and cfg.tie_embeddings):
         specs.append(ParamSpec("embed.weight", (cfg.vocab_size, H), "dense", "normal"))
     for i in range(lo, hi):
@@ -114,6 +125,8 @@ def tp_local_config(cfg: ModelConfig, tp: int) -> ModelConfig:
     (hidden size, experts, vocabulary) stays. Every shape of the store and of the kernels follows from it."""
     if tp == 1:
         return cfg
+    if cfg.plan is not None:
+        raise NotImplementedError("models with a layer plan are not sharded by tensor parallelism")
     assert cfg.num_q_heads % tp == 0 and cfg.num_kv_heads % tp == 0, "tensor parallel size must divide the head counts"
     assert cfg.is_moe or cfg.ffn_hidden_size % tp == 0
     import copy

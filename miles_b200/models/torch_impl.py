@@ -34,6 +34,12 @@ class InferMeta:
     page_size: int = 16
     cu_list: list = field(default_factory=list)
     prefix: Optional["PrefixInfo"] = None  # prefill only: part of every sequence is already in the KV cache
+    # models with a layer plan: tokens of every sequence that precede the ones of this pass, and the row of the per-sequence
+    # state each sequence owns (device tensors for the kernels, host lists for the launch tables)
+    ctx_lens: Optional[torch.Tensor] = None
+    ctx_list: list = field(default_factory=list)
+    state_slots: Optional[torch.Tensor] = None
+    tables: dict = field(default_factory=dict)  # launch tables built from the lists above, shared by the layers of a pass
 
 
 @dataclass

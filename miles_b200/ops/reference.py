@@ -291,3 +291,50 @@ def fake_int4_quant(x: torch.Tensor, gr: int, gc: int, sym: bool):
         z = (-torch.round(mn / s)).clamp(0, 15)
         q = torch.round(xf / s[..., None, None]) + z[..., None, None]
     return q.permute(0, 2, 1, 3).reshape(rows, cols), s, z
+
+
+# ---------------------------------------------------------------------------------------------- planned layers
+def dynamic_tanh(x, weight, bias, alpha):
+    """Element-wise norm replacement ``tanh(alpha x) * weight + bias`` in fp32."""
+    return torch.tanh(alpha.float() * x.float()) * weight.float() + bias.float()
+
+
+def unit_rms(x, eps: float):
+    return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+
+
+def pair_frequencies(dims: int, base: float, device=None):
+    """fp32 ``base^(-2 k / dims)``, k = 0 .. dims / 2 - 1 (evaluated in fp64)."""
+    k = torch.arange(dims // 2, dtype=torch.float64)
+    return (float(base) ** (-2.0 * k / dims)).to(torch.float32).to(device)
+
+
+def rotate_pairs(x, positions, base: float):
+    """Rotary embedding over interleaved pairs of the last dimension of ``x`` [T, heads, dims]; angles in fp32."""
+    a = positions.float()[:, None, None] * pair_frequencies(x.shape[-1], base, x.device)
+    u, v = x[..., 0::2].float(), x[..., 1::2].float()
+    c, s = torch.cos(a), torch.sin(a)
+    return torch.stack((u * c - v * s, v * c + u * s), -1).flatten(-2).to(x.dtype)
+
+
+def causal_conv_silu(x, weight, bias):
+    """Depthwise causal convolution and silu: ``x`` [T + taps - 1, channels] (the first taps - 1 rows are history)."""
+    taps = weight.shape[1]
+    y = F.conv1d(x.float().t()[None], weight.float()[:, None], bias.float(), groups=x.shape[1])[0].t()
+    assert y.shape[0] == x.shape[0] - taps + 1
+    return F.silu(y).to(x.dtype)
+
+
+def state_space_scan(x, B, C, dt_raw, A_log, D, state):
+    """Selective state space over one sequence: ``x`` [T, H, P], ``B`` / ``C`` [T, G, N], ``dt_raw`` [T, H] before
+    softplus, ``state`` [H, P, N]. Returns (y [T, H, P], state after the last token)."""
+    T, H, _ = x.shape
+    rep = H // B.shape[1]
+    dt = F.softplus(dt_raw, threshold=1e9)
+    decay = torch.exp(-torch.exp(A_log) * dt)
+    B, C = B.repeat_interleave(rep, 1), C.repeat_interleave(rep, 1)
+    ys = []
+    for t in range(T):
+        state = decay[t][:, None, None] * state + (dt[t][:, None] * x[t])[:, :, None] * B[t][:, None, :]
+        ys.append((state * C[t][:, None, :]).sum(-1) + D[:, None] * x[t])
+    return torch.stack(ys), state
