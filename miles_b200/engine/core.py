@@ -21,6 +21,7 @@ from typing import Optional, Sequence
 
 import torch
 
+from ..models.cache_layout import cache_layout
 from ..models.torch_impl import InferMeta
 
 
@@ -68,7 +69,9 @@ class Request:
     slot: int = -1  # row in the running batch
     seed: int = 0
     nodes: list = field(default_factory=list)  # prefix-cache nodes behind the first len(nodes) pages (shared, read only)
-    prefill_cached: int = 0                    # tokens of the current prefill that came from the prefix cache
+    # tokens that precede the current prefill in the cache (from the prefix cache, or earlier portions of the prompt)
+    prefill_cached: int = 0
+    prefilling: bool = False                   # part of the prompt has been computed, more portions follow
     cache_epoch: int = -1
     routes_tokens: int = 0                     # token positions covered by routed_experts so far
     t_submit: float = 0.0
@@ -121,6 +124,12 @@ class Engine:
                  sync=None, ep_decode=None, kv_storage: Optional[torch.Tensor] = None, overlap_decode: bool = True,
                  prefix_cache: bool = False, memory_saver: bool = False):
         self.model = model
+        self.cfg = model.cfg
+        self.store = model.store
+        self.kv_dtype = kv_dtype or self.store.dtype
+        # what the model keeps per token (paged) and per sequence (state): the engine only allocates and hands it out
+        self.layout = cache_layout(self.cfg, self.kv_dtype)
+        self.planned = self.cfg.plan is not None
         # KV cache in the tagged virtual-memory arena (utils/memory_saver.py): releasing it gives the physical memory
         # back but keeps the addresses, so captured decode graphs survive a release / resume cycle
         self._saver = None
@@ -132,7 +141,9 @@ class Engine:
             saver = MemorySaver()
             self._saver = saver if saver.available else None
         self.prefix = None
-        if prefix_cache:
+        # recurrent state exists for the newest token only, so a page boundary inside a cached prefix cannot be resumed
+        # from: models with state run without a prefix cache
+        if prefix_cache and not self.layout.has_state:
             from .prefix_cache import PrefixCache
 
             self.prefix = PrefixCache(page_size)
@@ -145,8 +156,6 @@ class Engine:
         self.ep_decode = ep_decode  # small expert-parallel exchange used by decode steps (graph friendly)
         self.last_mode = 0
         self._graph_pool = None
-        self.cfg = model.cfg
-        self.store = model.store
         self.dev = self.store.device
         self.on_gpu = self.dev.type == "cuda"
         self.page_size = page_size
@@ -155,11 +164,11 @@ class Engine:
         self.max_pages_per_seq = (max_seq_len + page_size - 1) // page_size
         self.max_prefill_tokens = max_prefill_tokens
         self.eos_token_id = eos_token_id
-        self.kv_dtype = kv_dtype or self.store.dtype
-        cfg = self.cfg
-        per_page = 2 * cfg.num_layers * page_size * cfg.num_kv_heads * cfg.head_dim * torch.empty((), dtype=self.kv_dtype).element_size()
+        per_page = max(1, self.layout.bytes_per_slot() * page_size)
         if num_pages is None:
-            if kv_mem_bytes is None:
+            if kv_mem_bytes is not None:
+                kv_mem_bytes -= self.layout.bytes_per_sequence() * (max_running + 1)
+            else:
                 kv_mem_bytes = max_running * max_seq_len * per_page // page_size
             num_pages = max(2, kv_mem_bytes // per_page)
         self.num_pages = int(num_pages)
@@ -168,7 +177,9 @@ class Engine:
         self._alloc_kv()
         self.waiting: deque = deque()
         self.running: list = []
+        self.prefilling: list = []  # admitted requests with portions of their prompt still to come, oldest first
         self.finished: dict = {}
+        self.fed: dict = {}         # sequences whose tokens are given by the caller (feed), by id
         self.paused = False
         self.weight_version = 0
         self._rid = itertools.count()
@@ -185,25 +196,17 @@ class Engine:
 
     # ------------------------------------------------------------------ memory
     def _alloc_kv(self) -> None:
-        cfg = self.cfg
-        slots = self.num_pages * self.page_size
+        slots, sequences = self.num_pages * self.page_size, self.max_running + 1  # the last state row belongs to padding rows
         if self.kv_storage is not None:
             # The buffer is shared in time with another user (the trainer's expert gradients): its contents
             # are undefined whenever a rollout starts, which is fine because every page is written by a
             # prefill or decode step before any position of it is read.
-            per = slots * cfg.num_kv_heads * cfg.head_dim
-            esz = torch.empty((), dtype=self.kv_dtype).element_size()
-            assert self.kv_storage.numel() >= 2 * cfg.num_layers * per * esz, "kv_storage is too small"
-            flat = self.kv_storage[:2 * cfg.num_layers * per * esz].view(self.kv_dtype)
-            views = [flat[i * per:(i + 1) * per].view(slots, cfg.num_kv_heads, cfg.head_dim) for i in range(2 * cfg.num_layers)]
-            self.kv_cache = [(views[2 * i], views[2 * i + 1]) for i in range(cfg.num_layers)]
+            self.kv_cache = self.layout.allocate(slots, sequences, self.dev, self.kv_storage)
             return
         import contextlib
 
         with (self._saver.region(self._kv_tag) if self._saver is not None else contextlib.nullcontext()):
-            self.kv_cache = [(torch.zeros(slots, cfg.num_kv_heads, cfg.head_dim, dtype=self.kv_dtype, device=self.dev),
-                              torch.zeros(slots, cfg.num_kv_heads, cfg.head_dim, dtype=self.kv_dtype, device=self.dev))
-                             for _ in range(cfg.num_layers)]
+            self.kv_cache = self.layout.allocate(slots, sequences, self.dev)
 
     def _alloc_decode_buffers(self) -> None:
         B, dev = self.max_running, self.dev
@@ -219,6 +222,8 @@ class Engine:
         self.d_seeds = torch.zeros(B, dtype=torch.int64, device=dev)
         self.d_step = torch.zeros(B, **i32)
         self.d_active = torch.zeros(B, **i32)
+        self.d_state_slots = torch.full((B,), B, **i32)
+        self.d_logits: Optional[torch.Tensor] = None  # logits of the newest decode step, row by row
         self._rows: list = []
         self._rows_B = 0
         self.d_out_tokens = torch.zeros(B, **i32)
@@ -236,7 +241,7 @@ class Engine:
     def release_memory_occupation(self, tags: Sequence[str] = ("kv_cache", "cuda_graph")) -> None:
         """Free the KV cache and/or captured graphs (weights are shared with the trainer and stay)."""
         self._drain_pending()
-        assert not self.running, "release_memory_occupation with running requests; pause/abort first"
+        assert not self.running and not self.prefilling and not self.fed, "release_memory_occupation with running requests; pause/abort first"
         if "cuda_graph" in tags:
             self._graphs.clear()
         if "kv_cache" in tags:
@@ -263,7 +268,7 @@ class Engine:
             self.pool = PagePool(self.num_pages)
 
     def flush_cache(self) -> bool:
-        if self.running:
+        if self.running or self.prefilling or self.fed:
             if self.prefix is not None:
                 # requests in flight keep the pages they use; everything else is forgotten (weights changed)
                 self.pool.release(self.prefix.clear())
@@ -288,9 +293,13 @@ class Engine:
         ps = self.page_size
         pages = torch.tensor([n.page for n in nodes], dtype=torch.int64, device=self.dev)
         slots = (pages[:, None] * ps + torch.arange(ps, device=self.dev)[None, :]).reshape(-1)
-        kv = torch.stack([torch.stack((kc[slots], vc[slots])) for kc, vc in self.kv_cache])
+        if self.planned:  # rows of every paged tensor (layers that read another layer's rows own none)
+            kv = [rows[slots].cpu() if to_cpu else rows[slots] for rows in self._paged_tensors()]
+        else:
+            kv = torch.stack([torch.stack((kc[slots], vc[slots])) for kc, vc in self.kv_cache])
+            kv = kv.cpu() if to_cpu else kv
         payloads = [n.payload for n in nodes]
-        return {"tokens": [int(t) for t in tokens[:len(nodes) * ps]], "kv": kv.cpu() if to_cpu else kv, "page_size": ps,
+        return {"tokens": [int(t) for t in tokens[:len(nodes) * ps]], "kv": kv, "page_size": ps,
                 "weight_version": self.weight_version,
                 "routed_experts": torch.cat(payloads, 0).cpu() if all(p is not None for p in payloads) else None}
 
@@ -308,7 +317,10 @@ class Engine:
         tokens = [int(t) for t in blob["tokens"]]
         n_pages = len(tokens) // ps
         kv = blob["kv"]
-        assert kv.shape[0] == len(self.kv_cache) and kv.shape[2] >= n_pages * ps, "exported keys / values of another model"
+        if self.planned:
+            assert len(kv) == len(self._paged_tensors()) and all(t.shape[0] >= n_pages * ps for t in kv), "exported rows of another model"
+        else:
+            assert kv.shape[0] == len(self.kv_cache) and kv.shape[2] >= n_pages * ps, "exported keys / values of another model"
         have = self.prefix.match(tokens)
         self.prefix.lock(have)  # an eviction for the new pages must not take the pages we build upon
         try:
@@ -321,10 +333,14 @@ class Engine:
             pg = torch.as_tensor(list(new_pages), dtype=torch.int64, device=self.dev)
             slots = (pg[:, None] * ps + torch.arange(ps, device=self.dev)[None, :]).reshape(-1)
             a = len(have) * ps
-            part = kv[:, :, a:n_pages * ps].to(self.dev)
-            for layer, (kc, vc) in enumerate(self.kv_cache):
-                kc[slots] = part[layer, 0].to(kc.dtype)
-                vc[slots] = part[layer, 1].to(vc.dtype)
+            if self.planned:
+                for rows, src in zip(self._paged_tensors(), kv):
+                    rows[slots] = src[a:n_pages * ps].to(device=self.dev, dtype=rows.dtype)
+            else:
+                part = kv[:, :, a:n_pages * ps].to(self.dev)
+                for layer, (kc, vc) in enumerate(self.kv_cache):
+                    kc[slots] = part[layer, 0].to(kc.dtype)
+                    vc[slots] = part[layer, 1].to(vc.dtype)
             payloads = None
             if blob.get("routed_experts") is not None:
                 re = blob["routed_experts"]
@@ -337,6 +353,9 @@ class Engine:
             freed = self.prefix.unlock(have)
             if freed:
                 self.pool.release(freed)
+
+    def _paged_tensors(self) -> list:
+        return [t for l, ts in zip(self.layout.layers, self.kv_cache) if l.shares is None for t in ts[:len(l.paged)]]
 
     def _alloc(self, n: int):
         """``n`` pages from the pool; when it runs dry, unreferenced prefix-cache pages are evicted first."""
@@ -366,7 +385,7 @@ class Engine:
     def abort_request(self, rid: Optional[str] = None, abort_all: bool = False) -> int:
         self._drain_pending()
         n = 0
-        for req in list(self.running):
+        for req in list(self.running) + list(self.prefilling):
             if abort_all or req.rid == rid:
                 self._finish(req, "abort")
                 n += 1
@@ -386,7 +405,7 @@ class Engine:
         if mode == "abort":
             self.abort_request(abort_all=True)
         elif mode == "retract":
-            for req in list(self.running):
+            for req in list(reversed(self.prefilling)) + list(self.running):
                 self._retract(req)
 
     def continue_generation(self) -> None:
@@ -397,7 +416,7 @@ class Engine:
         return self.weight_version
 
     def has_work(self) -> bool:
-        return bool(self.waiting or self.running or self._pending is not None)
+        return bool(self.waiting or self.running or self.prefilling or self._pending is not None)
 
     def pop_finished(self) -> list:
         out = list(self.finished.values())
@@ -409,10 +428,17 @@ class Engine:
         return (n_tokens + self.page_size - 1) // self.page_size
 
     def _retract(self, req: Request) -> None:
-        self._release(req, offer=True)
-        self.running.remove(req)
+        self._drop(req)
         self.waiting.appendleft(req)
         self.stats["retracted"] += 1
+
+    def _drop(self, req: Request) -> None:
+        """Take the request out of the running set (or out of the middle of its prefill) and give back what it holds."""
+        self._release(req, offer=not req.prefilling)  # a half computed prompt has nothing to offer to the prefix cache
+        for group in (self.running, self.prefilling):
+            if req in group:
+                group.remove(req)
+        req.prefilling, req.prefill_cached = False, 0
 
     def _release(self, req: Request, offer: bool = False) -> None:
         """Give the request's pages back. ``offer``: its full pages (prompt and generated tokens) are offered to the
@@ -449,9 +475,7 @@ class Engine:
 
     def _finish(self, req: Request, reason: str) -> None:
         req.finish_reason = reason
-        self._release(req, offer=True)
-        if req in self.running:
-            self.running.remove(req)
+        self._drop(req)
         self.finished[req.rid] = req
 
     def _check_stop(self, req: Request, tok: int) -> Optional[str]:
@@ -506,11 +530,16 @@ class Engine:
 
     def _admit(self) -> list:
         batch, tokens = [], 0
+        for req in self.prefilling:  # prompts under way come first, in the order they were admitted
+            if tokens >= self.max_prefill_tokens:
+                return batch
+            batch.append(req)
+            tokens += min(req.seq_len - req.prefill_cached, self.max_prefill_tokens - tokens)
         if self.prefix is None:
             while self.waiting and self.slots_free:
                 req = self.waiting[0]
                 n = req.seq_len
-                if batch and tokens + n > self.max_prefill_tokens:
+                if batch and (tokens >= self.max_prefill_tokens if self.planned else tokens + n > self.max_prefill_tokens):
                     break
                 pages = self._alloc(self._pages_needed(n + 1))
                 if pages is None:
@@ -536,7 +565,7 @@ class Engine:
             if any(_common_pages(ids, other, ps, n - 1) > len(nodes) for other in admitted_ids):
                 continue
             new_tokens = n - len(nodes) * ps
-            if batch and tokens + new_tokens > self.max_prefill_tokens:
+            if batch and (tokens >= self.max_prefill_tokens if self.planned else tokens + new_tokens > self.max_prefill_tokens):
                 break
             self.prefix.lock(nodes)  # before allocating: the eviction that may run now must not take them
             pages = self._alloc(self._pages_needed(n + 1) - len(nodes))
@@ -558,59 +587,99 @@ class Engine:
         return batch
 
     # ------------------------------------------------------------------ prefill
-    @torch.no_grad()
-    def _prefill(self, batch: list) -> None:
+    def _stage_rows(self, parts: list):
+        """Device inputs of a pass over new tokens of some sequences. ``parts``: (token ids, tokens already cached, pages,
+        state row) per sequence. Returns (tokens, positions, cu_seqlens on the host and on the device, meta); everything
+        the pass reads from the host travels in one pinned staging buffer."""
         dev, ps = self.dev, self.page_size
-        toks, pos, slots, cu = [], [], [], [0]
-        if not batch:  # lockstep dummy: one token written to the reserved page 0
-            toks, pos, slots, cu = [0], [0], [torch.zeros(1, dtype=torch.int64)], [0, 1]
-        prefix_lens, pre_slots = [], []
-        for req in batch:
-            ids = req.input_ids + req.output_ids
-            n, c = len(ids), req.prefill_cached
-            toks.extend(ids[c:])
+        toks, pos, slots, cu, pre_slots = [], [], [], [0], []
+        for ids, c, pages, _ in parts:
+            n = c + len(ids)
+            toks.extend(ids)
             pos.extend(range(c, n))
-            pg = torch.tensor(req.pages, dtype=torch.int64)
+            pg = torch.tensor(pages, dtype=torch.int64)
             idx = torch.arange(n)
             sl = pg[idx // ps] * ps + idx % ps
             slots.append(sl[c:])
             pre_slots.append(sl[:c])
-            prefix_lens.append(c)
             cu.append(cu[-1] + n - c)
-        # one pinned host staging buffer per prefill: tokens | positions | slot mapping | cu_seqlens, one H2D copy
-        n_tok = len(toks)
-        host = torch.empty(3 * n_tok + len(cu), dtype=torch.int32, pin_memory=self.on_gpu)
+        n_tok, nb = len(toks), len(parts)
+        ctx = [c for _, c, _, _ in parts]
+        width = max(len(pages) for _, _, pages, _ in parts) if self.planned else 0
+        # tokens | positions | slot mapping | cu_seqlens, and for planned layers context lengths | state rows | block table
+        host = torch.empty(3 * n_tok + len(cu) + (2 * nb + nb * width if self.planned else 0), dtype=torch.int32, pin_memory=self.on_gpu)
         host[:n_tok] = torch.tensor(toks, dtype=torch.int32)
         host[n_tok:2 * n_tok] = torch.tensor(pos, dtype=torch.int32)
         host[2 * n_tok:3 * n_tok] = torch.cat(slots).to(torch.int32)
-        host[3 * n_tok:] = torch.tensor(cu, dtype=torch.int32)
+        at = 3 * n_tok + len(cu)
+        host[3 * n_tok:at] = torch.tensor(cu, dtype=torch.int32)
+        if self.planned:
+            host[at:at + nb] = torch.tensor(ctx, dtype=torch.int32)
+            host[at + nb:at + 2 * nb] = torch.tensor([slot for _, _, _, slot in parts], dtype=torch.int32)
+            table = torch.zeros(nb, width, dtype=torch.int32)
+            for b, (_, _, pages, _) in enumerate(parts):
+                table[b, :len(pages)] = torch.tensor(pages, dtype=torch.int32)
+            host[at + 2 * nb:] = table.view(-1)
         staged = host.to(dev, non_blocking=True)
-        tokens, positions, slot_mapping, cu_t = (staged[:n_tok], staged[n_tok:2 * n_tok], staged[2 * n_tok:3 * n_tok],
-                                                 staged[3 * n_tok:])
+        self.h2d_bytes += host.numel() * 4
+        cu_t = staged[3 * n_tok:at]
         max_len = max(b - a for a, b in zip(cu[:-1], cu[1:]))
-        meta = InferMeta(True, cu_t, max_len, slot_mapping, page_size=ps)
-        if any(prefix_lens):
+        meta = InferMeta(True, cu_t, max_len, staged[2 * n_tok:3 * n_tok], page_size=ps)
+        if self.planned:
+            meta.cu_list, meta.ctx_list = cu, ctx
+            meta.ctx_lens, meta.state_slots = staged[at:at + nb], staged[at + nb:at + 2 * nb]
+            meta.block_table = staged[at + 2 * nb:].view(nb, width)
+        elif any(ctx):
             # part of every sequence is already in the KV cache: the attention reads those keys / values from their
             # pages (prefix slots) next to the ones this pass computes
             from ..models.torch_impl import PrefixInfo
 
-            meta.prefix = PrefixInfo.build(prefix_lens, [b - a for a, b in zip(cu[:-1], cu[1:])], torch.cat(pre_slots), dev)
-            self.stats["cached_tokens"] = self.stats.get("cached_tokens", 0) + sum(prefix_lens)
+            meta.prefix = PrefixInfo.build(ctx, [b - a for a, b in zip(cu[:-1], cu[1:])], torch.cat(pre_slots), dev)
+        return staged[:n_tok], staged[n_tok:2 * n_tok], cu, cu_t, meta
+
+    @torch.no_grad()
+    def _prefill(self, batch: list) -> None:
+        dev, ps = self.dev, self.page_size
+        parts, left = [], self.max_prefill_tokens
+        for req in batch:
+            ids, c = req.input_ids + req.output_ids, req.prefill_cached
+            # planned layers compute long prompts in portions of at most max_prefill_tokens per pass
+            n = min(len(ids), c + max(left, 1)) if self.planned else len(ids)
+            left -= n - c
+            parts.append((ids[c:n], c, req.pages, req.slot))
+            if not req.prefilling and c and self.prefix is not None:
+                self.stats["cached_tokens"] = self.stats.get("cached_tokens", 0) + c
+        if not batch:  # lockstep dummy: one token written to the reserved page 0
+            parts = [([0], 0, [0], self.max_running)]
+        tokens, positions, cu, cu_t, meta = self._stage_rows(parts)
+        toks, max_len = tokens, meta.max_seqlen
         want_routes = any(r.return_routed_experts for r in batch) and self.cfg.is_moe
         record = [] if want_routes else None
         kw = {"max_seqlen": max_len} if self.on_gpu and hasattr(self.model, "launches") else {}
         h = self.model.forward_hidden(tokens, positions, cu_t, meta=meta, kv_cache=self.kv_cache, record=record, **kw)
         if not batch:
             return
-        last = torch.tensor([c - 1 for c in cu[1:]], dtype=torch.int64, device=dev)
-        logits = self.model.logits(h[last])
-        tok, lp = self._sample(logits, batch)
-        tok_l, lp_l = tok.tolist(), lp.tolist()
+        done = [c + len(ids) == req.seq_len for req, (ids, c, _, _) in zip(batch, parts)]
+        tok_l, lp_l = [0] * len(batch), [0.0] * len(batch)
+        if any(done):
+            ends = [i for i, d in enumerate(done) if d]
+            logits = self.model.logits(h[torch.tensor([cu[i + 1] - 1 for i in ends], dtype=torch.int64, device=dev)])
+            tok, lp = self._sample(logits, [batch[i] for i in ends])
+            for i, t, l in zip(ends, tok.tolist(), lp.tolist()):
+                tok_l[i], lp_l[i] = t, l
         routes = torch.stack(record, 1).cpu() if want_routes else None  # [T, L, K]
         self.d2h_bytes += 8 * len(batch) + (routes.numel() * 4 if routes is not None else 0)
-        self.h2d_bytes += 12 * len(toks) + 4 * len(cu)
         self.stats["prefill_tokens"] += len(toks)
         for i, req in enumerate(batch):
+            if not done[i]:
+                req.prefill_cached += cu[i + 1] - cu[i]
+                if not req.prefilling:
+                    req.prefilling = True
+                    self.prefilling.append(req)
+                continue
+            if req.prefilling:
+                req.prefilling = False
+                self.prefilling.remove(req)
             if routes is not None and req.return_routed_experts:
                 # this pass covered positions [cached, n): keep what is not recorded yet (after a retraction only the
                 # position of the token that had been sampled but not fed is new)
@@ -698,15 +767,17 @@ class Engine:
     def _upload_rows(self, reqs: list, B: int) -> None:
         """Full refresh of the device-side decode state (only when the batch composition changed)."""
         W = self.max_pages_per_seq
-        h_i = torch.zeros(B, 6 + W, dtype=torch.int32)  # tok, pos, len, top_k, step, active, block_table...
+        h_i = torch.zeros(B, 7 + W, dtype=torch.int32)  # tok, pos, len, top_k, step, active, state row, block_table...
         h_i[:, 2] = 1
+        h_i[:, 6] = self.max_running
         h_f = torch.ones(B, 2, dtype=torch.float32)
         h_s = torch.zeros(B, dtype=torch.int64)
         for i, r in enumerate(reqs):
             L = r.seq_len  # tokens so far; the last one is the input of this step
             h_i[i, 0], h_i[i, 1], h_i[i, 2] = r.output_ids[-1], L - 1, L
             h_i[i, 3], h_i[i, 4], h_i[i, 5] = (r.params.top_k or 0), len(r.output_ids), 1
-            h_i[i, 6:6 + len(r.pages)] = torch.tensor(r.pages, dtype=torch.int32)
+            h_i[i, 6] = r.slot
+            h_i[i, 7:7 + len(r.pages)] = torch.tensor(r.pages, dtype=torch.int32)
             h_f[i, 0], h_f[i, 1] = r.params.temperature, r.params.top_p
             h_s[i] = r.seed
         d_i = h_i.to(self.dev, non_blocking=False)
@@ -716,7 +787,8 @@ class Engine:
         self.d_top_k[:B] = d_i[:, 3]
         self.d_step[:B] = d_i[:, 4]
         self.d_active[:B] = d_i[:, 5]
-        self.d_block_table[:B] = d_i[:, 6:]
+        self.d_state_slots[:B] = d_i[:, 6]
+        self.d_block_table[:B] = d_i[:, 7:]
         d_f = h_f.to(self.dev)
         self.d_temperature[:B] = d_f[:, 0]
         self.d_top_p[:B] = d_f[:, 1]
@@ -916,10 +988,11 @@ class Engine:
         pos = self.d_positions[:B]
         page = self.d_block_table[:B].gather(1, (pos // ps).long()[:, None])[:, 0]
         self.d_slots[:B] = page * ps + pos % ps
-        meta = InferMeta(False, None, 0, self.d_slots[:B], self.d_block_table[:B], self.d_seq_lens[:B], ps)
+        meta = InferMeta(False, None, 0, self.d_slots[:B], self.d_block_table[:B], self.d_seq_lens[:B], ps,
+                         state_slots=self.d_state_slots[:B])
         record = [] if want_routes else None
         h = self.model.forward_hidden(self.d_tokens[:B], pos, None, meta=meta, kv_cache=self.kv_cache, record=record)
-        logits = self.model.logits(h)
+        logits = self.d_logits = self.model.logits(h)
         if self.on_gpu and hasattr(self.model, "C"):
             self.model.C.sample_rows(logits, self.d_temperature[:B], self.d_top_k[:B], self.d_top_p[:B], self.d_seeds[:B],
                                      self.d_step[:B], self.d_out_tokens[:B], self.d_out_logprobs[:B])
@@ -945,6 +1018,8 @@ class Engine:
         if entry is None:
             # warm-up outside capture (first-use attribute setup, allocator growth), then capture
             launches0 = getattr(self.model, "launches", 0)
+            if self.layout.has_state:  # the warm-up must not advance anybody's recurrent state: it works on the padding row
+                self.d_state_slots[:B] = self.max_running
             self._decode_body(B, want_routes)
             torch.cuda.synchronize()
             per_replay = getattr(self.model, "launches", 0) - launches0
@@ -953,17 +1028,80 @@ class Engine:
                 self._graph_pool = torch.cuda.graph_pool_handle()
             with torch.cuda.graph(g, pool=self._graph_pool):
                 out = self._decode_body(B, want_routes)
-            entry = (g, out, per_replay)
+            entry = (g, out, per_replay, self.d_logits)
             self._graphs[key] = entry
             if hasattr(self.model, "launches"):
                 self.model.launches -= 2 * per_replay  # neither the warm-up nor the capture pass produced tokens
             # the warm-up run advanced the device-side decode state; rewind it before the first real replay
             self._upload_rows(list(self._rows), B)
-        g, out, per_replay = entry
+        g, out, per_replay, self.d_logits = entry
         g.replay()
         if hasattr(self.model, "launches"):
             self.model.launches += per_replay
         return out
+
+    # ------------------------------------------------------------------ given tokens
+    @torch.no_grad()
+    def feed(self, entries: Sequence[tuple]) -> list:
+        """One step over given tokens instead of sampled ones. ``entries``: ``(id, token ids, wanted places)`` per sequence;
+        an id's tokens continue what earlier calls brought under it. Single tokens of known sequences run as one decode
+        step (the captured graph included), everything else as one prefill pass. Returns the logits at the wanted places of
+        every entry (``[wanted, vocab]`` fp32). Sequences fed this way share pages and state rows with generation;
+        :meth:`end_feed` gives them back."""
+        self._drain_pending()
+        ps = self.page_size
+        out: list = [None] * len(entries)
+        portions, singles = [], []
+        for k, (rid, toks, want) in enumerate(entries):
+            req = self.fed.get(rid)
+            if req is None:
+                if not self.slots_free:
+                    raise RuntimeError("no free row: max_running sequences are held already")
+                req = self.fed[rid] = Request(rid, [], SamplingParams())
+                req.slot = self.slots_free.pop()
+                self.slot_req[req.slot] = req
+            ctx = len(req.input_ids)
+            if ctx + len(toks) > self.max_seq_len:
+                raise RuntimeError(f"sequence {rid!r} would grow past max_seq_len = {self.max_seq_len}")
+            missing = self._pages_needed(ctx + len(toks)) - len(req.pages)
+            if missing > 0:
+                pages = self._alloc(missing)
+                if pages is None:
+                    raise RuntimeError("out of cache pages")
+                req.pages = list(req.pages) + list(pages)
+            (singles if len(toks) == 1 and ctx > 0 else portions).append((k, req, [int(t) for t in toks], list(want)))
+        if portions:
+            parts = [(toks, len(req.input_ids), req.pages[:self._pages_needed(len(req.input_ids) + len(toks))], req.slot)
+                     for _, req, toks, _ in portions]
+            tokens, positions, cu, cu_t, meta = self._stage_rows(parts)
+            kw = {"max_seqlen": meta.max_seqlen} if self.on_gpu and hasattr(self.model, "launches") else {}
+            h = self.model.forward_hidden(tokens, positions, cu_t, meta=meta, kv_cache=self.kv_cache, **kw)
+            rows = [cu[j] + w for j, (_, _, _, want) in enumerate(portions) for w in want]
+            lg = self.model.logits(h[torch.tensor(rows, dtype=torch.int64, device=self.dev)]) if rows else None
+            at = 0
+            for k, req, toks, want in portions:
+                out[k] = lg[at:at + len(want)] if want else None
+                at += len(want)
+                req.input_ids = req.input_ids + toks
+        for a in range(0, len(singles), self.max_running):
+            group = singles[a:a + self.max_running]
+            B = self._bucket(len(group))
+            for _, req, toks, _ in group:
+                req.output_ids = toks  # the decode step's input is the newest token
+            self._upload_rows([req for _, req, _, _ in group], B)
+            self._run_decode(B, False)
+            lg = self.d_logits[:len(group)].clone()
+            for j, (k, req, toks, want) in enumerate(group):
+                out[k] = lg[j:j + 1] if want else None
+                req.input_ids, req.output_ids = req.input_ids + toks, []
+            self._rows, self._rows_B = [], 0
+        return out
+
+    def end_feed(self, rid: str) -> None:
+        """Give back the pages and the state row of a sequence fed by :meth:`feed`."""
+        req = self.fed.pop(rid, None)
+        if req is not None:
+            self._release(req)
 
     # ------------------------------------------------------------------ scoring
     @torch.no_grad()
