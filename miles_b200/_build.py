@@ -1,4 +1,5 @@
-"""In-tree build of the sm_100a extension ``miles_b200/_C.so``.
+"""In-tree build of the sm_100a extensions ``miles_b200/_C.so`` (training and the uniform decoder families) and
+``miles_b200/_hybrid.so`` (engine kernels of models with a layer plan, with the products and the sampler they share).
 
 Kernels are plain CUDA translation units compiled by nvcc without the PyTorch headers (seconds per
 file); only ``bindings.cpp`` sees ``torch/extension.h``.  Objects are cached under ``csrc/build`` and
@@ -18,6 +19,11 @@ PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 OBJ = CSRC / "build"
 TARGET = PKG / "_C.so"
+# planned-layer models load only this library, so serving one compiles a handful of files
+HYBRID_TARGET = PKG / "_hybrid.so"
+HYBRID_ONLY = {"hybrid_ops.cu", "mamba2.cu", "latent_attention.cu", "latent_prefill.cu", "hybrid_bindings.cpp"}
+HYBRID_SHARED = {"gemm.cu", "decode_small.cu", "decode_stream.cu", "sampling.cu", "serve_bindings.cpp"}
+TARGETS = {"_C": TARGET, "_hybrid": HYBRID_TARGET}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -34,15 +40,18 @@ def _cuda_home() -> Path:
     return Path(_nvcc()).resolve().parent.parent
 
 
-def _newest_header() -> float:
-    hs = list(CSRC.rglob("*.cuh")) + list(CSRC.rglob("*.h")) + list(CSRC.rglob("*.hpp"))
+def _newest_header(hybrid: bool = True) -> float:
+    """Newest header, with or without the ones only planned-layer sources include."""
+    hs = [*CSRC.rglob("*.cuh"), *CSRC.rglob("*.h"), *CSRC.rglob("*.hpp")]
+    hs = [h for h in hs if hybrid or not h.name.startswith("hybrid")]
     return max((h.stat().st_mtime for h in hs), default=0.0)
 
 
-def sources() -> tuple[list[Path], list[Path]]:
+def sources(module: str = "_C") -> tuple[list[Path], list[Path]]:
     cu = sorted(p for p in CSRC.rglob("*.cu") if "build" not in p.parts)
     cpp = sorted(p for p in CSRC.rglob("*.cpp") if "build" not in p.parts and "native" not in p.parts)
-    return cu, cpp
+    keep = (lambda p: p.name in HYBRID_ONLY | HYBRID_SHARED) if module == "_hybrid" else (lambda p: p.name not in HYBRID_ONLY)
+    return [p for p in cu if keep(p)], [p for p in cpp if keep(p)]
 
 
 # ---------------------------------------------------------------------------------------------- host-only module
@@ -72,12 +81,13 @@ def build_native(verbose: bool = False, force: bool = False) -> Path:
     return NATIVE_TARGET
 
 
-def needs_build() -> bool:
-    if not TARGET.exists():
+def needs_build(module: str = "_C") -> bool:
+    target = TARGETS[module]
+    if not target.exists():
         return True
-    t = TARGET.stat().st_mtime
-    cu, cpp = sources()
-    return any(s.stat().st_mtime > t for s in cu + cpp) or _newest_header() > t
+    t = target.stat().st_mtime
+    cu, cpp = sources(module)
+    return any(s.stat().st_mtime > t for s in cu + cpp) or _newest_header(module == "_hybrid") > t
 
 
 def _run(cmd: list[str]) -> None:
@@ -91,10 +101,7 @@ def _obj_for(src: Path) -> Path:
     return OBJ / ("_".join(rel.parts) + ".o")
 
 
-def build(verbose: bool = False, force: bool = False) -> Path:
-    import torch
-    from torch.utils import cpp_extension
-
+def build(verbose: bool = False, force: bool = False, modules: tuple = ("_C", "_hybrid")) -> Path:
     OBJ.mkdir(parents=True, exist_ok=True)
     import fcntl
 
@@ -102,24 +109,29 @@ def build(verbose: bool = False, force: bool = False) -> Path:
     lock = open(OBJ / ".build.lock", "w")
     fcntl.flock(lock, fcntl.LOCK_EX)
     try:
-        return _build_locked(verbose, force)
+        for module in modules:
+            if force or needs_build(module):  # (another process may have built it while this one waited for the lock)
+                _build_locked(module, verbose, force)
+        build_native(verbose=verbose, force=force)
+        return TARGETS[modules[0]]
     finally:
         fcntl.flock(lock, fcntl.LOCK_UN)
         lock.close()
 
 
-def _build_locked(verbose: bool, force: bool) -> Path:
+def _build_locked(module: str, verbose: bool, force: bool) -> None:
     import torch
     from torch.utils import cpp_extension
 
-    cu, cpp = sources()
-    hdr_t = _newest_header()
+    target = TARGETS[module]
+    cu, cpp = sources(module)
+    stale = lambda s, o: force or not o.exists() or o.stat().st_mtime < max(s.stat().st_mtime, _newest_header(s.name in HYBRID_ONLY))
     jobs: list[list[str]] = []
     objs: list[Path] = []
     for s in cu:
         o = _obj_for(s)
         objs.append(o)
-        if force or not o.exists() or o.stat().st_mtime < max(s.stat().st_mtime, hdr_t):
+        if stale(s, o):
             jobs.append([_nvcc(), *NVCC_FLAGS, "-I", str(CSRC), "-c", str(s), "-o", str(o)])
     inc = cpp_extension.include_paths(device_type="cpu") + [str(_cuda_home() / "include"), str(CSRC),
                                                             sysconfig.get_paths()["include"]]
@@ -128,24 +140,22 @@ def _build_locked(verbose: bool, force: bool) -> Path:
     for s in cpp:
         o = _obj_for(s)
         objs.append(o)
-        if force or not o.exists() or o.stat().st_mtime < max(s.stat().st_mtime, hdr_t):
+        if stale(s, o):
             cmd = ["g++", *cxx_flags]
             for i in inc:
                 cmd += ["-isystem", i]
             jobs.append(cmd + ["-c", str(s), "-o", str(o)])
     if verbose:
-        print(f"[miles_b200] compiling {len(jobs)} translation units", file=sys.stderr)
+        print(f"[miles_b200] {module}: compiling {len(jobs)} translation units", file=sys.stderr)
     with ThreadPoolExecutor(max_workers=max(1, min(8, os.cpu_count() or 1))) as ex:
         list(ex.map(_run, jobs))
-    if jobs or not TARGET.exists() or force:
+    if jobs or not target.exists() or force or needs_build(module):
         torch_lib = Path(torch.__file__).parent / "lib"
-        link = ["g++", "-shared", "-o", str(TARGET), *map(str, objs), f"-L{torch_lib}", "-lc10", "-ltorch_cpu",
+        link = ["g++", "-shared", "-o", str(target), *map(str, objs), f"-L{torch_lib}", "-lc10", "-ltorch_cpu",
                 "-ltorch", "-ltorch_python", "-lc10_cuda", "-ltorch_cuda",
                 f"-L{_cuda_home() / 'lib64'}", "-lcudart", f"-Wl,-rpath,{torch_lib}",
                 f"-Wl,-rpath,{_cuda_home() / 'lib64'}"]
         _run(link)
-    build_native(verbose=verbose, force=force)
-    return TARGET
 
 
 if __name__ == "__main__":

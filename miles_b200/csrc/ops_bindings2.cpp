@@ -3,37 +3,12 @@
 #include <c10/cuda/CUDAStream.h>
 #include <torch/extension.h>
 
+#include "binding_helpers.h"
 #include "launchers.h"
 
 namespace {
 
-cudaStream_t cur_stream() { return c10::cuda::getCurrentCUDAStream().stream(); }
-
-#define CHECK_BF16(t) TORCH_CHECK((t).is_cuda() && (t).scalar_type() == at::kBFloat16 && (t).is_contiguous(), #t " must be a contiguous bf16 CUDA tensor")
-#define CHECK_F32(t) TORCH_CHECK((t).is_cuda() && (t).scalar_type() == at::kFloat && (t).is_contiguous(), #t " must be a contiguous fp32 CUDA tensor")
-#define CHECK_I32(t) TORCH_CHECK((t).is_cuda() && (t).scalar_type() == at::kInt && (t).is_contiguous(), #t " must be a contiguous int32 CUDA tensor")
-
-template <typename T>
-T* opt_ptr(const c10::optional<at::Tensor>& t) {
-  return t.has_value() ? static_cast<T*>(t->data_ptr()) : nullptr;
-}
-
-// logits [B, V] (bf16/fp32) -> (token int32 [B], logprob fp32 [B]); per-row parameters are optional tensors.
-void sample_rows(const at::Tensor& logits, const c10::optional<at::Tensor>& temperature,
-                 const c10::optional<at::Tensor>& top_k, const c10::optional<at::Tensor>& top_p,
-                 const c10::optional<at::Tensor>& seeds, const c10::optional<at::Tensor>& step, at::Tensor& out_token,
-                 at::Tensor& out_logprob) {
-  TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.stride(1) == 1, "logits must be 2-D with contiguous rows");
-  const bool fp32 = logits.scalar_type() == at::kFloat;
-  TORCH_CHECK(fp32 || logits.scalar_type() == at::kBFloat16, "logits must be bf16 or fp32");
-  CHECK_I32(out_token); CHECK_F32(out_logprob);
-  if (seeds.has_value()) TORCH_CHECK(seeds->scalar_type() == at::kLong && seeds->is_cuda(), "seeds must be int64 CUDA");
-  const c10::cuda::CUDAGuard guard(logits.device());
-  mb::sample_rows(logits.data_ptr(), fp32, logits.size(0), logits.size(1), logits.stride(0), opt_ptr<float>(temperature),
-                  opt_ptr<int>(top_k), opt_ptr<float>(top_p),
-                  reinterpret_cast<const unsigned long long*>(opt_ptr<int64_t>(seeds)), opt_ptr<int>(step),
-                  out_token.data_ptr<int>(), out_logprob.data_ptr<float>(), cur_stream());
-}
+using namespace mb_bind;
 
 // q [B, Hq, 128]; caches [slots, Hk, 128]; block_table [B, max_pages]; out [B, Hq, 128]; scratch fp32.
 void paged_decode_attention(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache,
@@ -109,23 +84,6 @@ std::vector<at::Tensor> flash_attn_bwd(const at::Tensor& q, const at::Tensor& k,
 }
 
 // ---- small-batch decode kernels (T <= 8)
-void small_gemv(const at::Tensor& x, const c10::optional<at::Tensor>& norm_w, double eps, const at::Tensor& W,
-                const c10::optional<at::Tensor>& residual, at::Tensor& out, const c10::optional<at::Tensor>& status) {
-  CHECK_BF16(x); CHECK_BF16(W);
-  const int T = x.size(0), K = x.size(1), N = W.size(0);
-  TORCH_CHECK(T >= 1 && T <= 64 && W.size(1) == K && K % 32 == 0 && N % 16 == 0, "small_gemv: need 1 <= T <= 64, K % 32 == 0, N % 16 == 0");
-  TORCH_CHECK(T <= 8 || !norm_w.has_value(), "small_gemv: the folded RMSNorm is available for at most 8 rows");
-  TORCH_CHECK(out.is_cuda() && out.is_contiguous() && out.size(0) == T && out.size(1) == N, "small_gemv: bad output shape");
-  const bool f32 = out.scalar_type() == at::kFloat;
-  TORCH_CHECK(f32 || out.scalar_type() == at::kBFloat16, "small_gemv: output must be fp32 or bf16");
-  if (norm_w.has_value()) CHECK_BF16((*norm_w));
-  if (residual.has_value()) { CHECK_BF16((*residual)); TORCH_CHECK(residual->numel() == out.numel(), "small_gemv: residual shape"); }
-  const c10::cuda::CUDAGuard guard(x.device());
-  mb::small_gemv(x.data_ptr(), T, norm_w.has_value() ? norm_w->data_ptr() : nullptr, eps, W.data_ptr(), N, K,
-                 residual.has_value() ? residual->data_ptr() : nullptr, out.data_ptr(), f32,
-                 status.has_value() ? status->data_ptr<int>() : nullptr, cur_stream());
-}
-
 void router_small(const at::Tensor& logits, int64_t K, bool renorm, at::Tensor& ids, at::Tensor& w, at::Tensor& active,
                   at::Tensor& pair_count, at::Tensor& pair_list) {
   CHECK_F32(logits); CHECK_I32(ids); CHECK_F32(w); CHECK_I32(active); CHECK_I32(pair_count); CHECK_I32(pair_list);
@@ -249,13 +207,11 @@ void register_more(pybind11::module_& m) {
   register_mx(m);
   register_ep_ll(m);
   register_weight_push(m);
-  m.def("sample_rows", &sample_rows);
   m.def("paged_decode_attention", &paged_decode_attention, pybind11::arg("q"), pybind11::arg("k_cache"), pybind11::arg("v_cache"),
         pybind11::arg("block_table"), pybind11::arg("seq_lens"), pybind11::arg("out"), pybind11::arg("scratch"),
         pybind11::arg("page_size"), pybind11::arg("num_splits"), pybind11::arg("scale"), pybind11::arg("status") = pybind11::none());
   m.def("flash_attn_fwd", &flash_attn_fwd);
   m.def("flash_attn_bwd", &flash_attn_bwd);
-  m.def("small_gemv", &small_gemv);
   m.def("router_small", &router_small);
   m.def("moe_small_up", &moe_small_up);
   m.def("moe_small_down", &moe_small_down);

@@ -17,7 +17,7 @@ import os
 import sys
 
 
-def build_engine(model_dir: str, dtype: str, max_tokens: int, device: str | None = None, page_size: int = 64, max_running: int = 64):
+def build_engine(model_dir: str, dtype: str, max_tokens: int, device: str = "cuda", page_size: int = 64, max_running: int = 64):
     """The engine that serves a checkpoint directory in ``dtype``, its cache sized for ``max_tokens`` live tokens."""
     import torch
 
@@ -25,7 +25,6 @@ def build_engine(model_dir: str, dtype: str, max_tokens: int, device: str | None
     from ..models import ParamStore, build_model, get_config
     from .core import Engine
 
-    device = device or ("cuda" if torch.cuda.is_available() else "cpu")
     # "float32" means 32-bit products, not a reduced-precision matrix mode
     torch.backends.cuda.matmul.allow_tf32 = False
     torch.backends.cudnn.allow_tf32 = False
@@ -45,15 +44,16 @@ def main(argv=None) -> int:
     ap.add_argument("--dtype", required=True, choices=["bfloat16", "float32"])
     ap.add_argument("--out", required=True, help="directory for the logits files")
     ap.add_argument("--max-tokens", type=int, required=True, help="most tokens that live sequences hold at any time")
+    ap.add_argument("--device", default="cuda", help="cpu: the PyTorch path of the framework's CPU configuration")
     ns = ap.parse_args(argv)
     import torch
 
     from ..models import get_config
 
-    if ns.dtype == "float32" and get_config(ns.model).plan is None and torch.cuda.is_available():
+    if ns.dtype == "float32" and get_config(ns.model).plan is None and ns.device != "cpu":
         print("this model runs in bfloat16 on the GPU", file=sys.stderr)
         return 3
-    engine = build_engine(ns.model, ns.dtype, ns.max_tokens)
+    engine = build_engine(ns.model, ns.dtype, ns.max_tokens, ns.device)
     for line in sys.stdin:
         if not line.strip():
             continue

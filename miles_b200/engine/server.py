@@ -216,7 +216,7 @@ def main(argv=None) -> None:
 
         load_hf(cfg, store, ns.hf_checkpoint)
         tokenizer = load_tokenizer(ns.hf_checkpoint)
-    model = build_model(cfg, store, "b200" if (on_gpu and cfg.head_dim == 128) else "torch")
+    model = build_model(cfg, store, "auto" if cfg.plan is not None else "b200" if (on_gpu and cfg.head_dim == 128) else "torch")
     if ns.quantization != "none" and hasattr(model, "enable_block_scaled"):
         model.enable_block_scaled(ns.quantization)
     kv_bytes = None

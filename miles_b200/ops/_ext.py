@@ -15,12 +15,13 @@ from pathlib import Path
 _LOCK = threading.Lock()
 _MOD = None
 _TRIED = False
+_HYBRID = None
 
 
 def _import_so(path: Path):
     import torch  # noqa: F401  (libtorch symbols must be loaded first)
 
-    spec = importlib.util.spec_from_file_location("miles_b200._C", str(path))
+    spec = importlib.util.spec_from_file_location(f"miles_b200.{path.stem}", str(path))
     mod = importlib.util.module_from_spec(spec)
     spec.loader.exec_module(mod)
     return mod
@@ -47,9 +48,22 @@ def load(required: bool | None = None):
             if _TRIED:
                 raise RuntimeError("miles_b200._C could not be built earlier in this process")
             _TRIED = True
-            _build.build(verbose=True)
+            _build.build(verbose=True, modules=("_C",))
         _MOD = _import_so(_build.TARGET)
         return _MOD
+
+
+def load_hybrid():
+    """The extension behind models with a layer plan (``miles_b200/_hybrid.so``), built first if it is missing or stale."""
+    global _HYBRID
+    with _LOCK:
+        if _HYBRID is None:
+            from .. import _build
+
+            if _build.needs_build("_hybrid"):
+                _build.build(verbose=True, modules=("_hybrid",))
+            _HYBRID = _import_so(_build.HYBRID_TARGET)
+        return _HYBRID
 
 
 def available() -> bool:
