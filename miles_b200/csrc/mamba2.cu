@@ -20,6 +20,18 @@ namespace {
 
 using namespace hy;
 
+// exp(x) S for x <= 0 as fma(c, S, k S). A slow decay multiplies thousands of times, so that a bias of the rounded factor
+// would add up; near 1 the factor is therefore applied as S + (exp(x) - 1) S.
+struct Decay {
+  float c, k;
+  __device__ __forceinline__ explicit Decay(float x) {
+    const bool near_one = x > -0.35f;
+    c = near_one ? expm1f(x) : expf(x);
+    k = near_one ? 1.f : 0.f;
+  }
+  __device__ __forceinline__ float operator()(float s) const { return fmaf(c, s, k * s); }
+};
+
 // ------------------------------------------------------------------------------------------------ convolution (prefill)
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) conv_kernel(const HyMamba a, const int4* __restrict__ tiles, T* __restrict__ xbc) {
@@ -135,7 +147,7 @@ __global__ void __launch_bounds__(256) scan_kernel(const HyMamba a, const T* __r
     const long long r = first + t;
     const T* row = xbc + r * ch;
     const float dt = softplus_f(to_f(dtc[r * a.ld]) + bias);
-    const float decay = expf(A * dt);
+    const Decay decay(A * dt);
     const float x = to_f(row[h * a.P + p]);
     const T *B = row + inner + g * a.N, *C = B + a.groups * a.N;
     float o = 0.f;
@@ -143,7 +155,7 @@ __global__ void __launch_bounds__(256) scan_kernel(const HyMamba a, const T* __r
     for (int i = 0; i < NR; ++i) {
       const int k = lane + 32 * i;
       if (k < a.N) {
-        S[i] = decay * S[i] + dt * to_f(B[k]) * x;
+        S[i] = decay(S[i]) + dt * to_f(B[k]) * x;
         o += S[i] * to_f(C[k]);
       }
     }
@@ -187,7 +199,7 @@ __global__ void __launch_bounds__(256) step_kernel(const HyMamba a, const int* _
   __syncthreads();
   const float A = -expf(to_f(static_cast<const T*>(a.A_log)[h])), D = to_f(static_cast<const T*>(a.D)[h]);
   const float dt = softplus_f(to_f(pr[inner + ch + h]) + to_f(static_cast<const T*>(a.dt_bias)[h]));
-  const float decay = expf(A * dt);
+  const Decay decay(A * dt);
   const float *x = sm, *B = sm + P, *C = B + N;
   float* st = a.state + (slot * a.heads + h) * static_cast<long long>(P) * N;
   T* out = y + static_cast<long long>(b) * inner + h * P;
@@ -209,10 +221,10 @@ __global__ void __launch_bounds__(256) step_kernel(const HyMamba a, const int* _
         for (int u = 0; u < U; ++u) {
           if (p0 + u >= P) break;
           const float xp = x[p0 + u];
-          s[u].x = decay * s[u].x + dt * bv.x * xp;
-          s[u].y = decay * s[u].y + dt * bv.y * xp;
-          s[u].z = decay * s[u].z + dt * bv.z * xp;
-          s[u].w = decay * s[u].w + dt * bv.w * xp;
+          s[u].x = decay(s[u].x) + dt * bv.x * xp;
+          s[u].y = decay(s[u].y) + dt * bv.y * xp;
+          s[u].z = decay(s[u].z) + dt * bv.z * xp;
+          s[u].w = decay(s[u].w) + dt * bv.w * xp;
           o[u] += s[u].x * cv.x + s[u].y * cv.y + s[u].z * cv.z + s[u].w * cv.w;
           *reinterpret_cast<float4*>(st + static_cast<long long>(p0 + u) * N + k) = s[u];
         }
@@ -228,7 +240,7 @@ __global__ void __launch_bounds__(256) step_kernel(const HyMamba a, const int* _
       float o = 0.f;
       float* row = st + static_cast<long long>(p) * N;
       for (int k = lane; k < N; k += 32) {
-        const float s = decay * (fresh ? 0.f : row[k]) + dt * B[k] * x[p];
+        const float s = decay(fresh ? 0.f : row[k]) + dt * B[k] * x[p];
         row[k] = s;
         o += s * C[k];
       }
