@@ -30,7 +30,10 @@ SIZES = {
 }
 
 
-def rokivik_config(s: dict, window: int = 2048) -> dict:
+WINDOW = 2048
+
+
+def rokivik_config(s: dict, window: int = WINDOW) -> dict:
     def mamba():
         return {"type": "mamba2", "mixer": {"heads": s["mheads"], "vdim": 64, "state": 128, "groups": s["groups"], "conv": 4,
                                             "norm_groups": s["groups"]}, "mlp": {"kind": "dense", "ff": s["ff"]}}
@@ -125,15 +128,18 @@ def floors(cfg, kind: str, s: dict, T: int, ctx: int, prefill: bool) -> dict:
     inner, ch = hd * P, hd * P + 2 * G * N
     f = {}
     if kind == "rokivik":
-        R, W, h, L = 512, 576, s["heads"], sum(range(1, ctx + 1)) if prefill else ctx
+        # (mean over the three attention layers: two windows and one whole context)
+        R, W, h = 512, 576, s["heads"]
+        seen = [min(i, WINDOW) for i in range(1, ctx + 1)]
+        L = (2 * sum(seen) + sum(range(1, ctx + 1))) / 3 if prefill else (2 * seen[-1] + ctx) / 3
         if prefill:
             n = T // ctx
             c = 128
             chunks = n * ((ctx + c - 1) // c)
             st = chunks * hd * P * N * 4
-            f["conv4_pair"] = (T * ch * 2 * 2, 0)
+            f["conv4_vec"] = (T * ch * 2 * 2, 0)
             f["chunk_state"] = (T * (inner + G * N) * 2 + st, 2 * T * hd * P * N)
-            f["chunk_pass"] = (2 * st, 0)
+            f["chunk_pass"] = (2 * st, 0)  # (fp32 in, two bf16 planes out)
             f["chunk_out"] = (T * (2 * inner + 2 * G * N) * 2 + st, 2 * T * hd * (P * N + (c + 1) / 2 * (N + P)))
             f["mamba_tail"] = (T * (3 * inner + 3 * s["ff"]) * 2, 0)
             f["latent_in"] = (T * (2 * (s["q_rank"] + W) + 3 * s["ff"]) * 2, 0)
@@ -148,7 +154,7 @@ def floors(cfg, kind: str, s: dict, T: int, ctx: int, prefill: bool) -> dict:
             f["step_kernel"] = (T * (hd * P * N * 8 + ch * 2 * 5 + inner * 2), 0)
             f["mamba_tail"] = (T * (3 * inner + 3 * s["ff"]) * 2, 0)
             f["latent_in"] = (T * (2 * (s["q_rank"] + W) + 3 * s["ff"]) * 2, 0)
-            f["latent_decode"] = (T * ctx * W * 2 + T * h * (W * 2 + R * 4), 2 * T * ctx * h * (W + R))
+            f["latent_decode"] = (T * L * W * 2 + T * h * (W * 2 + R * 4), 2 * T * L * h * (W + R))
             f["absorb_q"] = (h * 128 * R * 2 + T * h * (192 + W) * 2, 2 * T * h * 128 * R)
             f["latent_up"] = (h * 128 * R * 2 + T * h * (R * 4 + 128 * 2), 2 * T * h * 128 * R)
             f["side_fused"] = (2 * s["side"] * H * 2 + T * H * (4 + 4 + 4 + 2), 4 * T * s["side"] * H)

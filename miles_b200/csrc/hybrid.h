@@ -80,11 +80,12 @@ int hy_conv(bool f32, const HyMamba& a, const int* tiles, int n_tiles, void* xbc
 // Sequential scan (any sizes, exact fp32): y [T, heads * P]
 int hy_scan(bool f32, const HyMamba& a, const void* xbc, void* y, cudaStream_t s);
 // Chunked scan on the tensor cores (bf16). `chunks` int32 [n][4] = {sequence, first row, rows, chunk index in sequence},
-// sequence by sequence; `first_chunk` [nseq + 1]; work: fp32 [n, heads, P, N], decay: fp32 [n, heads].
+// sequence by sequence; `first_chunk` [nseq + 1]; work: fp32 [n, heads, P, N], decay: fp32 [n, heads], before: bf16
+// [n, heads, 2, P, N].
 bool hy_chunk_scan_supported(int P, int N, int heads, int groups);
 constexpr int HY_CHUNK = 128;
 int hy_chunk_scan(const HyMamba& a, const void* xbc, const int* chunks, int n_chunks, const int* first_chunk, float* work,
-                  float* decay, void* y, cudaStream_t s);
+                  float* decay, void* before, void* y, cudaStream_t s);
 // One token per sequence: convolution, state update and output in one kernel. positions[b] = 0 starts from a zero state.
 int hy_mamba_step(bool f32, const HyMamba& a, const int* positions, int B, void* y, cudaStream_t s);
 

@@ -191,8 +191,9 @@ void mamba_prefill(MAMBA_ARGS, const at::Tensor& cu, const at::Tensor& ctx, cons
     const int64_t n = chunks->size(0);
     TORCH_CHECK(chunks->size(1) == 4 && first_chunk->numel() == ctx.numel() + 1, "mamba_prefill: chunk tables");
     at::Tensor work = at::empty({n * heads * P * N}, state.options()), decay = at::empty({n * heads}, state.options());
+    at::Tensor before = at::empty({n * heads * 2 * P * N}, proj.options());
     RUN(mb::hy_chunk_scan(a, xbc.data_ptr(), chunks->data_ptr<int>(), n, first_chunk->data_ptr<int>(), work.data_ptr<float>(),
-                          decay.data_ptr<float>(), y.data_ptr(), cur_stream()));
+                          decay.data_ptr<float>(), before.data_ptr(), y.data_ptr(), cur_stream()));
   } else {
     RUN(mb::hy_scan(f, a, xbc.data_ptr(), y.data_ptr(), cur_stream()));
   }

@@ -81,14 +81,14 @@ __device__ __forceinline__ void cat_ff(const HyCat& c, long long t, bool vec) {
 
 // Grid (T, 2): y = 0 the mixer part, y = 1 the feed-forward part of a row.
 template <typename T>
-__global__ void __launch_bounds__(256) mamba_tail_kernel(const T* __restrict__ y, const T* __restrict__ w, int inner, int ng, float eps,
+__global__ void __launch_bounds__(1024) mamba_tail_kernel(const T* __restrict__ y, const T* __restrict__ w, int inner, int ng, float eps,
                                                          const HyCat c, bool ff_vec, bool mix_vec) {
   const long long t = blockIdx.x;
   if (blockIdx.y == 1) {
     cat_ff<T>(c, t, ff_vec);
     return;
   }
-  extern __shared__ float sm[];  // [inner] gated values, then [8] partial sums
+  extern __shared__ float sm[];  // [inner] gated values, then [32] partial sums
   float* part = sm + inner;
   const T* yr = y + t * inner;
   const T* z = static_cast<const T*>(c.proj) + t * c.ld;
@@ -106,11 +106,11 @@ __global__ void __launch_bounds__(256) mamba_tail_kernel(const T* __restrict__ y
     for (int i = threadIdx.x; i < inner; i += blockDim.x) sm[i] = to_f(yr[i]) * silu_f(to_f(z[i]));
   }
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, size = inner / ng;
-  const int wpg = ng >= 8 ? 1 : 8 / ng;  // warps per group
-  for (int g0 = 0; g0 < ng; g0 += 8 / wpg) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, size = inner / ng, nw = blockDim.x >> 5;
+  const int wpg = ng >= nw ? 1 : nw / ng;  // warps per group
+  for (int g0 = 0; g0 < ng; g0 += nw / wpg) {
     const int g = g0 + warp / wpg;
-    const bool live = g < ng && warp < (8 / wpg) * wpg;
+    const bool live = g < ng && warp < (nw / wpg) * wpg;
     float s = 0.f;
     if (live)
       for (int i = (warp % wpg) * 32 + lane; i < size; i += wpg * 32) {
@@ -133,7 +133,7 @@ __global__ void __launch_bounds__(256) mamba_tail_kernel(const T* __restrict__ y
 
 // Grid (T, 2): y = 0 the latents of a row, y = 1 its feed-forward part.
 template <typename T>
-__global__ void __launch_bounds__(256) latent_in_kernel(const HyLatentIn a, const HyCat c, bool ff_vec) {
+__global__ void __launch_bounds__(1024) latent_in_kernel(const HyLatentIn a, const HyCat c, bool ff_vec) {
   __shared__ float red[33];
   const long long t = blockIdx.x;
   if (blockIdx.y == 1) {
@@ -179,22 +179,40 @@ __global__ void __launch_bounds__(256) latent_in_kernel(const HyLatentIn a, cons
 
 // ------------------------------------------------------------------------------------------------ per-layer token input
 constexpr int CS = 8;    // CTAs per cluster: each owns an eighth of the gate rows and of the output columns
-constexpr int STHREADS = 256;
+constexpr int STHREADS = 1024;
+constexpr int LPR = 4;   // lanes per row of the projection
+constexpr int PF = 8;    // 16-byte pieces of a projection row a lane fetches ahead (rows of up to LPR * PF * 8 bf16 values)
 
-// TB tokens per cluster.
+// TB tokens per cluster. The weights do not depend on anything computed here, so their loads are issued first: the gate rows of
+// the warps, and the first projection row of every group of LPR lanes.
 template <typename T, int TB>
 __global__ void __launch_bounds__(STHREADS) side_fused_kernel(const HySide a, int n_tok, bool vec_h, bool vec_s) {
-  extern __shared__ float sm[];
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float wred[STHREADS / 32][TB];
+  constexpr int N = Vec<T>::N;
   cg::cluster_group cl = cg::this_cluster();
   const int rank = static_cast<int>(cl.block_rank());
   const int t0 = static_cast<int>(blockIdx.x / CS) * TB;
   const int H = a.H, sd = a.sd;
-  float* xs = sm;                       // [TB][H] residual with delta
-  float* gs = xs + TB * H;              // [TB][sd]
-  float* ss = gs + TB * sd;             // [TB][CS] partial sums of squares
+  const int Hp = (H + 3) & ~3, sp = (sd + 3) & ~3;
+  float* xs = sm;                       // [TB][Hp] residual with delta
+  float* gs = xs + TB * Hp;             // [TB][sp]
+  float* ss = gs + TB * sp;             // [TB][CS] partial sums of squares
   const int cols = (H + CS - 1) / CS, c0 = rank * cols, c1 = min(H, c0 + cols);
   float* ys = ss + TB * CS;             // [TB][cols]
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = STHREADS / 32;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = threadIdx.x & (LPR - 1);
+  const int row_of = threadIdx.x / LPR;
+  const bool ahead = vec_s && sd <= LPR * PF * N;
+  uint4 pw[PF];
+  if (ahead) {
+    const int c = c0 + row_of;
+#pragma unroll
+    for (int i = 0; i < PF; ++i) {
+      const int k = (i * LPR + sub) * N;
+      pw[i] = make_uint4(0u, 0u, 0u, 0u);
+      if (c < c1 && k < sd) pw[i] = *reinterpret_cast<const uint4*>(static_cast<const T*>(a.proj) + static_cast<long long>(c) * sd + k);
+    }
+  }
   for (int b = 0; b < TB; ++b) {
     const int t = t0 + b;
     for (int i = threadIdx.x; i < H; i += STHREADS) {
@@ -203,32 +221,35 @@ __global__ void __launch_bounds__(STHREADS) side_fused_kernel(const HySide a, in
         v = a.x[static_cast<long long>(t) * H + i];
         if (a.delta) v += a.delta[static_cast<long long>(t) * H + i];
       }
-      xs[b * H + i] = v;
+      xs[b * Hp + i] = v;
     }
   }
   cl.sync();  // every CTA of the cluster runs before its shared memory is written from another
   // gate products of this CTA's rows, sent to every CTA of the cluster
   const int dims = (sd + CS - 1) / CS, d0 = rank * dims, d1 = min(sd, d0 + dims);
-  for (int d = d0 + warp; d < d1; d += nw) {
+  for (int d = d0 + warp; d < d1; d += STHREADS / 32) {
     const T* w = static_cast<const T*>(a.gate) + static_cast<long long>(d) * H;
     float s[TB];
 #pragma unroll
     for (int b = 0; b < TB; ++b) s[b] = 0.f;
     if (vec_h) {
-      constexpr int N = Vec<T>::N;
+#pragma unroll 4
       for (int i = lane * N; i < H; i += 32 * N) {
         float v[N];
         Vec<T>::load(w + i, v);
 #pragma unroll
         for (int b = 0; b < TB; ++b)
 #pragma unroll
-          for (int k = 0; k < N; ++k) s[b] += v[k] * xs[b * H + i + k];
+          for (int k = 0; k < N; k += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(xs + b * Hp + i + k);
+            s[b] += v[k] * x.x + v[k + 1] * x.y + v[k + 2] * x.z + v[k + 3] * x.w;
+          }
       }
     } else {
       for (int i = lane; i < H; i += 32) {
         const float v = to_f(w[i]);
 #pragma unroll
-        for (int b = 0; b < TB; ++b) s[b] += v * xs[b * H + i];
+        for (int b = 0; b < TB; ++b) s[b] += v * xs[b * Hp + i];
       }
     }
 #pragma unroll
@@ -243,61 +264,73 @@ __global__ void __launch_bounds__(STHREADS) side_fused_kernel(const HySide a, in
           tok = 0;
         }
         const float e = to_f(static_cast<const T*>(a.embed)[static_cast<long long>(tok) * a.embed_ld + a.embed_col + d]);
-        g = gelu_tanh_f(s[b]) * e;
-        g = to_f(from_f<T>(g));
+        g = to_f(from_f<T>(gelu_tanh_f(s[b]) * e));
       }
-      if (lane < CS) *cl.map_shared_rank(gs + b * sd + d, lane) = g;
+      if (lane < CS) *cl.map_shared_rank(gs + b * sp + d, lane) = g;
     }
   }
   cl.sync();
-  // this CTA's output columns: 8 lanes per row of the projection
-  {
-    float sq[TB];
+  // this CTA's output columns: LPR lanes per row of the projection
+  float sq[TB];
 #pragma unroll
-    for (int b = 0; b < TB; ++b) sq[b] = 0.f;
-    const int sub = threadIdx.x & 7;
-    for (int base = c0; base < c1; base += STHREADS / 8) {
-      const int c = base + (threadIdx.x >> 3);
-      float s[TB];
+  for (int b = 0; b < TB; ++b) sq[b] = 0.f;
+  for (int base = c0; base < c1; base += STHREADS / LPR) {
+    const int c = base + row_of;
+    const T* w = static_cast<const T*>(a.proj) + static_cast<long long>(c) * sd;
+    float s[TB];
 #pragma unroll
-      for (int b = 0; b < TB; ++b) s[b] = 0.f;
-      if (c < c1) {
-        const T* w = static_cast<const T*>(a.proj) + static_cast<long long>(c) * sd;
-        if (vec_s) {
-          constexpr int N = Vec<T>::N;
-          for (int i = sub * N; i < sd; i += 8 * N) {
-            float v[N];
-            Vec<T>::load(w + i, v);
+    for (int b = 0; b < TB; ++b) s[b] = 0.f;
+    auto dot = [&](const uint4& raw, int k) {
+      float v[N];
+      Vec<T>::load(reinterpret_cast<const T*>(&raw), v);
 #pragma unroll
-            for (int b = 0; b < TB; ++b)
+      for (int b = 0; b < TB; ++b)
 #pragma unroll
-              for (int k = 0; k < N; ++k) s[b] += v[k] * gs[b * sd + i + k];
-          }
-        } else {
-          for (int i = sub; i < sd; i += 8) {
-            const float v = to_f(w[i]);
-#pragma unroll
-            for (int b = 0; b < TB; ++b) s[b] += v * gs[b * sd + i];
-          }
+        for (int j = 0; j < N; j += 4) {
+          const float4 g = *reinterpret_cast<const float4*>(gs + b * sp + k + j);
+          s[b] += v[j] * g.x + v[j + 1] * g.y + v[j + 2] * g.z + v[j + 3] * g.w;
         }
-      }
+    };
+    if (ahead) {
 #pragma unroll
-      for (int b = 0; b < TB; ++b) {
-        s[b] += __shfl_xor_sync(0xffffffffu, s[b], 1);
-        s[b] += __shfl_xor_sync(0xffffffffu, s[b], 2);
-        s[b] += __shfl_xor_sync(0xffffffffu, s[b], 4);
-        if (c < c1 && sub == 0) {
-          ys[b * cols + c - c0] = s[b];
-          sq[b] += s[b] * s[b];
+      for (int i = 0; i < PF; ++i)
+        if ((i * LPR + sub) * N < sd) dot(pw[i], (i * LPR + sub) * N);
+      const int cn = c + STHREADS / LPR;  // the next row of this lane
+#pragma unroll
+      for (int i = 0; i < PF; ++i) {
+        const int k = (i * LPR + sub) * N;
+        if (cn < c1 && k < sd) pw[i] = *reinterpret_cast<const uint4*>(static_cast<const T*>(a.proj) + static_cast<long long>(cn) * sd + k);
+      }
+    } else if (c < c1) {
+      if (vec_s) {
+        for (int k = sub * N; k < sd; k += LPR * N) dot(*reinterpret_cast<const uint4*>(w + k), k);
+      } else {
+        for (int i = sub; i < sd; i += LPR) {
+          const float v = to_f(w[i]);
+#pragma unroll
+          for (int b = 0; b < TB; ++b) s[b] += v * gs[b * sp + i];
         }
       }
     }
-    __shared__ float red[33];
 #pragma unroll
     for (int b = 0; b < TB; ++b) {
-      const float tot = block_sum(sq[b], red);
-      if (threadIdx.x < CS) *cl.map_shared_rank(ss + b * CS + rank, threadIdx.x) = tot;
+      s[b] += __shfl_xor_sync(0xffffffffu, s[b], 1);
+      s[b] += __shfl_xor_sync(0xffffffffu, s[b], 2);
+      if (c < c1 && sub == 0) {
+        ys[b * cols + c - c0] = s[b];
+        sq[b] += s[b] * s[b];
+      }
     }
+  }
+#pragma unroll
+  for (int b = 0; b < TB; ++b) {
+    sq[b] = warp_sum(sq[b]);
+    if (lane == 0) wred[warp][b] = sq[b];
+  }
+  __syncthreads();
+  if (warp < TB) {
+    const float tot = warp_sum(wred[lane][warp]);
+    if (lane < CS) *cl.map_shared_rank(ss + warp * CS + rank, lane) = tot;
   }
   cl.sync();
   const float al = to_f(static_cast<const T*>(a.na)[0]);
@@ -309,7 +342,7 @@ __global__ void __launch_bounds__(STHREADS) side_fused_kernel(const HySide a, in
     for (int k = 0; k < CS; ++k) tot += ss[b * CS + k];
     const float r = 1.f / sqrtf(tot / static_cast<float>(H) + a.eps);
     for (int c = c0 + threadIdx.x; c < c1; c += STHREADS) {
-      const float v = xs[b * H + c] + ys[b * cols + c - c0] * r * to_f(static_cast<const T*>(a.norm)[c]);
+      const float v = xs[b * Hp + c] + ys[b * cols + c - c0] * r * to_f(static_cast<const T*>(a.norm)[c]);
       a.x[static_cast<long long>(t) * H + c] = v;
       static_cast<T*>(a.h)[static_cast<long long>(t) * H + c] =
           from_f<T>(tanhf(al * v) * to_f(static_cast<const T*>(a.nw)[c]) + to_f(static_cast<const T*>(a.nb)[c]));
@@ -328,9 +361,10 @@ __global__ void __launch_bounds__(256) cast_rows_kernel(const float* __restrict_
   }
 }
 
-template <typename T>
+// V values per thread (V = 1: any width)
+template <typename T, int V>
 __global__ void __launch_bounds__(256) side_gate_kernel(const float* __restrict__ z, const HySide a, T* __restrict__ g, long long n) {
-  const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  const long long i = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) * V;
   if (i >= n) return;
   const long long t = i / a.sd;
   const int d = static_cast<int>(i - t * a.sd);
@@ -339,8 +373,22 @@ __global__ void __launch_bounds__(256) side_gate_kernel(const float* __restrict_
     if (a.status) atomicCAS(a.status, 0, 10);
     tok = 0;
   }
-  const float e = to_f(static_cast<const T*>(a.embed)[static_cast<long long>(tok) * a.embed_ld + a.embed_col + d]);
-  g[i] = from_f<T>(gelu_tanh_f(z[i]) * e);
+  const T* e = static_cast<const T*>(a.embed) + static_cast<long long>(tok) * a.embed_ld + a.embed_col + d;
+  if constexpr (V > 1) {
+    float ev[V], o[V];
+    Vec<T>::load(e, ev);
+#pragma unroll
+    for (int k = 0; k < V; k += 4) {
+      const float4 v = *reinterpret_cast<const float4*>(z + i + k);
+      o[k] = gelu_tanh_f(v.x) * ev[k];
+      o[k + 1] = gelu_tanh_f(v.y) * ev[k + 1];
+      o[k + 2] = gelu_tanh_f(v.z) * ev[k + 2];
+      o[k + 3] = gelu_tanh_f(v.w) * ev[k + 3];
+    }
+    Vec<T>::store(g + i, o);
+  } else {
+    g[i] = from_f<T>(gelu_tanh_f(z[i]) * to_f(e[0]));
+  }
 }
 
 template <typename T>
@@ -397,7 +445,7 @@ __global__ void __launch_bounds__(256) side_finish_kernel(const float* __restric
 template <typename T, int TB>
 int launch_side(const HySide& a, int n_tok, cudaStream_t s) {
   const int cols = (a.H + CS - 1) / CS;
-  const size_t smem = sizeof(float) * (static_cast<size_t>(TB) * (a.H + a.sd + CS + cols));
+  const size_t smem = sizeof(float) * (static_cast<size_t>(TB) * (((a.H + 3) & ~3) + ((a.sd + 3) & ~3) + CS + cols));
   auto kern = side_fused_kernel<T, TB>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
@@ -434,12 +482,13 @@ int embed_norm_t(const int* tokens, int T_, const void* table, int V, int H, con
 
 template <typename T>
 int mamba_tail_t(const void* y, const void* w, int inner, int ng, float eps, const HyCat& c, int T_, cudaStream_t s) {
-  const size_t smem = sizeof(float) * (static_cast<size_t>(inner) + 8);
+  const size_t smem = sizeof(float) * (static_cast<size_t>(inner) + 32);
   auto kern = mamba_tail_kernel<T>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   const bool mv = inner % Vec<T>::N == 0 && aligned16<T>(y, inner) && aligned16<T>(c.proj, c.ld);
-  kern<<<dim3(T_, 2), 256, smem, s>>>(static_cast<const T*>(y), static_cast<const T*>(w), inner, ng, eps, c, ff_vec_ok<T>(c), mv);
+  // few rows: latency counts, so every load of a row is in flight at once
+  kern<<<dim3(T_, 2), T_ <= 148 ? 1024 : 256, smem, s>>>(static_cast<const T*>(y), static_cast<const T*>(w), inner, ng, eps, c, ff_vec_ok<T>(c), mv);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -458,15 +507,15 @@ int hy_mamba_tail(bool f32, const void* y, const void* w, int inner, int norm_gr
 
 int hy_latent_in(bool f32, const HyLatentIn& a, const HyCat& c, int T, cudaStream_t s) {
   if (f32)
-    latent_in_kernel<float><<<dim3(T, 2), 256, 0, s>>>(a, c, ff_vec_ok<float>(c));
+    latent_in_kernel<float><<<dim3(T, 2), T <= 148 ? 1024 : 256, 0, s>>>(a, c, ff_vec_ok<float>(c));
   else
-    latent_in_kernel<bf16><<<dim3(T, 2), 256, 0, s>>>(a, c, ff_vec_ok<bf16>(c));
+    latent_in_kernel<bf16><<<dim3(T, 2), T <= 148 ? 1024 : 256, 0, s>>>(a, c, ff_vec_ok<bf16>(c));
   return static_cast<int>(cudaGetLastError());
 }
 
 int hy_side_fused(bool f32, const HySide& a, int T, cudaStream_t s) {
   // tokens share the weight reads of their cluster; few rows are spread over more clusters, and wide rows bound the memory
-  const bool four = T > 32 && static_cast<long long>(a.H) * 4 * 4 * 9 / 8 + a.sd * 16 < 200 * 1024;
+  const bool four = T > 16 && static_cast<long long>(a.H) * 4 * 4 * 9 / 8 + a.sd * 16 < 200 * 1024;
   if (f32) return four ? launch_side<float, 4>(a, T, s) : launch_side<float, 1>(a, T, s);
   return four ? launch_side<bf16, 4>(a, T, s) : launch_side<bf16, 1>(a, T, s);
 }
@@ -477,14 +526,19 @@ int hy_cast_rows(const float* x, void* out, long long n, cudaStream_t s) {
   return static_cast<int>(cudaGetLastError());
 }
 
-int hy_side_gate(bool f32, const float* z, const HySide& a, void* g, int T, cudaStream_t s) {
-  const long long n = static_cast<long long>(T) * a.sd;
-  const unsigned blocks = static_cast<unsigned>((n + 255) / 256);
-  if (f32)
-    side_gate_kernel<float><<<blocks, 256, 0, s>>>(z, a, static_cast<float*>(g), n);
+template <typename T>
+static int side_gate_t(const float* z, const HySide& a, void* g, int rows, cudaStream_t s) {
+  const long long n = static_cast<long long>(rows) * a.sd;
+  constexpr int V = hy::Vec<T>::N;
+  if (a.sd % V == 0 && a.embed_ld % V == 0)
+    side_gate_kernel<T, V><<<static_cast<unsigned>((n / V + 255) / 256), 256, 0, s>>>(z, a, static_cast<T*>(g), n);
   else
-    side_gate_kernel<bf16><<<blocks, 256, 0, s>>>(z, a, static_cast<bf16*>(g), n);
+    side_gate_kernel<T, 1><<<static_cast<unsigned>((n + 255) / 256), 256, 0, s>>>(z, a, static_cast<T*>(g), n);
   return static_cast<int>(cudaGetLastError());
+}
+
+int hy_side_gate(bool f32, const float* z, const HySide& a, void* g, int T, cudaStream_t s) {
+  return f32 ? side_gate_t<float>(z, a, g, T, s) : side_gate_t<bf16>(z, a, g, T, s);
 }
 
 int hy_side_finish(bool f32, const float* y, const HySide& a, int T, cudaStream_t s) {

@@ -30,120 +30,248 @@ __device__ __forceinline__ long long row_slot(const HyLatent& a, int seq, int po
 }
 
 // ------------------------------------------------------------------------------------------------ projections
-// Block (x, head, row tile): x < nr: 128 latent columns; x == nr: the rotated part and the padding.
+// Rotated part and padding of row t, head h (all threads of the block, rows t0 .. t0 + TT).
 template <typename T, typename O>
-__global__ void __launch_bounds__(128) absorb_q_kernel(const HyLatent a, const T* __restrict__ q, const int* __restrict__ positions,
+__device__ __forceinline__ void absorb_rotated(const HyLatent& a, const T* __restrict__ q, const int* __restrict__ positions, int n_rows,
+                                               O* __restrict__ ql, int qld, int h, int t0) {
+  const int tail = qld - a.rank;
+  for (int i = threadIdx.x; i < TT * tail; i += blockDim.x) {
+    const int b = i / tail, c = i - b * tail, t = t0 + b;
+    if (t >= n_rows) break;
+    float v = 0.f;
+    if (c < a.rot) {
+      const T* src = q + (static_cast<long long>(t) * a.heads + h) * (a.dim + a.rot) + a.dim;
+      float sn, cs;
+      sincosf(static_cast<float>(positions[t]) * a.freq[c >> 1], &sn, &cs);
+      const float u = to_f(src[c & ~1]), w = to_f(src[c | 1]);
+      v = (c & 1) ? w * cs + u * sn : u * cs - w * sn;
+    }
+    ql[(static_cast<long long>(t) * a.heads + h) * qld + a.rank + c] = from_f<O>(v);
+  }
+}
+
+// Block (x, head, row tile): x < nr: 128 latent columns; x == nr: the rotated part and the padding. VEC: 16 lanes cover the
+// columns (16 bytes each), the block's 16 half-warps split the head's dimensions so that all weight loads are in flight at
+// once; the partial sums meet in shared memory.
+template <typename T, typename O, bool VEC>
+__global__ void __launch_bounds__(256) absorb_q_kernel(const HyLatent a, const T* __restrict__ q, const int* __restrict__ positions,
                                                        int n_rows, O* __restrict__ ql, int qld, int nr) {
-  extern __shared__ float qs[];  // [TT][dim]
+  extern __shared__ float qs[];  // [TT][dim], VEC: then [8][TT][128] partial sums
   const int h = blockIdx.y, t0 = blockIdx.z * TT, qd = a.dim + a.rot;
   if (static_cast<int>(blockIdx.x) == nr) {
-    for (int i = threadIdx.x; i < TT * (qld - a.rank); i += blockDim.x) {
-      const int b = i / (qld - a.rank), c = i - b * (qld - a.rank), t = t0 + b;
-      if (t >= n_rows) break;
-      float v = 0.f;
-      if (c < a.rot) {
-        const T* src = q + (static_cast<long long>(t) * a.heads + h) * qd + a.dim;
-        float sn, cs;
-        sincosf(static_cast<float>(positions[t]) * a.freq[c >> 1], &sn, &cs);
-        const float u = to_f(src[c & ~1]), w = to_f(src[c | 1]);
-        v = (c & 1) ? w * cs + u * sn : u * cs - w * sn;
-      }
-      ql[(static_cast<long long>(t) * a.heads + h) * qld + a.rank + c] = from_f<O>(v);
-    }
+    absorb_rotated<T, O>(a, q, positions, n_rows, ql, qld, h, t0);
     return;
   }
   for (int i = threadIdx.x; i < TT * a.dim; i += blockDim.x) {
     const int b = i / a.dim, d = i - b * a.dim;
     qs[i] = t0 + b < n_rows ? to_f(q[(static_cast<long long>(t0 + b) * a.heads + h) * qd + d]) : 0.f;
   }
-  __syncthreads();
-  const int r = blockIdx.x * 128 + threadIdx.x;
-  if (r >= a.rank) return;
-  const T* w = static_cast<const T*>(a.ukv) + static_cast<long long>(h) * a.dim * a.rank + r;
-  float acc[TT];
+  const T* w = static_cast<const T*>(a.ukv) + static_cast<long long>(h) * a.dim * a.rank;
+  if constexpr (VEC) {
+    float* part = qs + TT * a.dim;
+    const int lane16 = threadIdx.x & 15, slice = threadIdx.x >> 4;  // 16 slices of the dimensions
+    const int r = blockIdx.x * 128 + lane16 * 8;
+    float acc[TT][8];
 #pragma unroll
-  for (int b = 0; b < TT; ++b) acc[b] = 0.f;
-#pragma unroll 8
-  for (int d = 0; d < a.dim; ++d) {
-    const float v = to_f(w[static_cast<long long>(d) * a.rank]);
+    for (int b = 0; b < TT; ++b)
 #pragma unroll
-    for (int b = 0; b < TT; ++b) acc[b] += v * qs[b * a.dim + d];
-  }
-#pragma unroll
-  for (int b = 0; b < TT; ++b)
-    if (t0 + b < n_rows) ql[(static_cast<long long>(t0 + b) * a.heads + h) * qld + r] = from_f<O>(acc[b]);
-}
-
-// Block (x, head, row tile): 32 output values of a head. o is [T, heads, splits, rank] with (max, sum) per split when ml is
-// given (unnormalised partial outputs), else normalised and splits = 1.
-template <typename T>
-__global__ void __launch_bounds__(128) latent_up_kernel(const HyLatent a, const float* __restrict__ o, const float* __restrict__ ml,
-                                                        int splits, int n_rows, T* __restrict__ cat, int ldc, bool vec) {
-  extern __shared__ float os[];  // [TT][rank]
-  __shared__ float coef[TT][64];
-  const int h = blockIdx.y, t0 = blockIdx.z * TT;
-  const int rows = min(TT, n_rows - t0);
-  if (ml) {
-    if (static_cast<int>(threadIdx.x) < rows) {
-      const float* p = ml + (static_cast<long long>(t0 + threadIdx.x) * a.heads + h) * splits * 2;
-      float m = -FLT_MAX, l = 0.f;
-      for (int s = 0; s < splits; ++s) m = fmaxf(m, p[2 * s]);
-      for (int s = 0; s < splits; ++s) {
-        const float c = p[2 * s] == -FLT_MAX ? 0.f : exp2f(p[2 * s] - m);
-        coef[threadIdx.x][s] = c;
-        l += c * p[2 * s + 1];
-      }
-      const float inv = l > 0.f ? 1.f / l : 0.f;
-      for (int s = 0; s < splits; ++s) coef[threadIdx.x][s] *= inv;
-    }
+      for (int k = 0; k < 8; ++k) acc[b][k] = 0.f;
+    constexpr int U = 4;
     __syncthreads();
-  }
-  for (int i = threadIdx.x; i < TT * a.rank; i += blockDim.x) {
-    const int b = i / a.rank, r = i - b * a.rank;
-    float v = 0.f;
-    if (b < rows) {
-      const float* p = o + (static_cast<long long>(t0 + b) * a.heads + h) * splits * a.rank + r;
-      if (ml) {
-        for (int s = 0; s < splits; ++s)
-          if (coef[b][s] != 0.f) v += coef[b][s] * p[static_cast<long long>(s) * a.rank];
-      } else {
-        v = p[0];
+    if (r < a.rank) {
+      for (int d0 = slice; d0 < a.dim; d0 += 16 * U) {
+        uint4 raw[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+          if (d0 + 16 * u < a.dim) raw[u] = *reinterpret_cast<const uint4*>(w + static_cast<long long>(d0 + 16 * u) * a.rank + r);
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int d = d0 + 16 * u;
+          if (d >= a.dim) break;
+          const uint32_t x4[4] = {raw[u].x, raw[u].y, raw[u].z, raw[u].w};
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&x4[k]));
+#pragma unroll
+            for (int b = 0; b < TT; ++b) {
+              const float qv = qs[b * a.dim + d];
+              acc[b][2 * k] += f.x * qv;
+              acc[b][2 * k + 1] += f.y * qv;
+            }
+          }
+        }
       }
     }
-    os[i] = v;
-  }
-  __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const T* wv = static_cast<const T*>(a.ukv) + static_cast<long long>(a.heads) * a.dim * a.rank;
-  const int v_end = min(a.vdim, static_cast<int>(blockIdx.x) * 32 + 32);
-  for (int v = blockIdx.x * 32 + warp; v < v_end; v += 4) {
-    const T* w = wv + (static_cast<long long>(h) * a.vdim + v) * a.rank;
+    const int warp = threadIdx.x >> 5;
+#pragma unroll
+    for (int b = 0; b < TT; ++b)
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const float v = acc[b][k] + __shfl_xor_sync(0xffffffffu, acc[b][k], 16);
+        if ((threadIdx.x & 16) == 0) part[(warp * TT + b) * 128 + lane16 * 8 + k] = v;
+      }
+    __syncthreads();
+    for (int i = threadIdx.x; i < TT * 128; i += blockDim.x) {
+      const int b = i >> 7, c = i & 127, rr = blockIdx.x * 128 + c;
+      if (t0 + b >= n_rows || rr >= a.rank) continue;
+      float v = 0.f;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v += part[(k * TT + b) * 128 + c];
+      ql[(static_cast<long long>(t0 + b) * a.heads + h) * qld + rr] = from_f<O>(v);
+    }
+  } else {
+    __syncthreads();
+    const int r = blockIdx.x * 128 + threadIdx.x;
+    if (threadIdx.x >= 128 || r >= a.rank) return;
     float acc[TT];
 #pragma unroll
     for (int b = 0; b < TT; ++b) acc[b] = 0.f;
-    if (vec) {
-      constexpr int N = Vec<T>::N;
-      for (int r = lane * N; r < a.rank; r += 32 * N) {
-        float x[N];
-        Vec<T>::load(w + r, x);
+#pragma unroll 8
+    for (int d = 0; d < a.dim; ++d) {
+      const float v = to_f(w[static_cast<long long>(d) * a.rank + r]);
 #pragma unroll
-        for (int b = 0; b < TT; ++b)
-#pragma unroll
-          for (int k = 0; k < N; ++k) acc[b] += x[k] * os[b * a.rank + r + k];
-      }
-    } else {
-      for (int r = lane; r < a.rank; r += 32) {
-        const float x = to_f(w[r]);
-#pragma unroll
-        for (int b = 0; b < TT; ++b) acc[b] += x * os[b * a.rank + r];
-      }
+      for (int b = 0; b < TT; ++b) acc[b] += v * qs[b * a.dim + d];
     }
 #pragma unroll
-    for (int b = 0; b < TT; ++b) {
-      acc[b] = warp_sum(acc[b]);
-      if (lane == 0 && b < rows) cat[static_cast<long long>(t0 + b) * ldc + h * a.vdim + v] = from_f<T>(acc[b]);
+    for (int b = 0; b < TT; ++b)
+      if (t0 + b < n_rows) ql[(static_cast<long long>(t0 + b) * a.heads + h) * qld + r] = from_f<O>(acc[b]);
+  }
+}
+
+// Block (x, head, row tile): 32 output values of a head. o is [T, heads, splits, rank] with (max, sum) per split when ml is
+// given (unnormalised partial outputs), else normalised and splits = 1. RT rows per block.
+template <typename T, int RT>
+__global__ void __launch_bounds__(256) latent_up_kernel(const HyLatent a, const float* __restrict__ o, const float* __restrict__ ml,
+                                                        int splits, int n_rows, T* __restrict__ cat, int ldc, bool vec) {
+  extern __shared__ float os[];  // [RT][rank]
+  __shared__ float coef[RT][64];
+  const int h = blockIdx.y, t0 = blockIdx.z * RT;
+  const int rows = min(RT, n_rows - t0);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* wv = static_cast<const T*>(a.ukv) + (static_cast<long long>(a.heads) * a.dim + h * a.vdim) * a.rank;
+  constexpr int N = Vec<T>::N, VB = 4, WC = 2;  // a warp's four output values; chunks of their weights fetched ahead
+  const int v0 = blockIdx.x * 32 + warp * VB;
+  float w[VB][WC][N];
+  auto fetch = [&](int base) {
+#pragma unroll
+    for (int i = 0; i < VB; ++i)
+#pragma unroll
+      for (int k = 0; k < WC; ++k) {
+        const int r = base + (k * 32 + lane) * N;
+        if (v0 + i < a.vdim && r < a.rank) {
+          Vec<T>::load(wv + static_cast<long long>(v0 + i) * a.rank + r, w[i][k]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < N; ++j) w[i][k][j] = 0.f;
+        }
+      }
+  };
+  if (vec) fetch(0);  // (does not depend on the attention's result)
+  if (ml) {  // a warp per row: coefficients of the splits
+    for (int b = warp; b < rows; b += 8) {
+      const float* p = ml + (static_cast<long long>(t0 + b) * a.heads + h) * splits * 2;
+      float mv[2], lv[2], m = -FLT_MAX;
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const int s = lane + 32 * k;
+        mv[k] = s < splits ? p[2 * s] : -FLT_MAX;
+        lv[k] = s < splits ? p[2 * s + 1] : 0.f;
+        m = fmaxf(m, mv[k]);
+      }
+#pragma unroll
+      for (int off = 16; off > 0; off >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, off));
+      float l = 0.f, c[2];
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        c[k] = mv[k] == -FLT_MAX ? 0.f : exp2f(mv[k] - m);
+        l += c[k] * lv[k];
+      }
+      l = warp_sum(l);
+      const float inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+      for (int k = 0; k < 2; ++k)
+        if (lane + 32 * k < splits) coef[b][lane + 32 * k] = c[k] * inv;
+    }
+    __syncthreads();
+  }
+  if ((a.rank & 3) == 0) {
+    for (int i = threadIdx.x * 4; i < RT * a.rank; i += blockDim.x * 4) {
+      const int b = i / a.rank, r = i - b * a.rank;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (b < rows) {
+        const float* p = o + (static_cast<long long>(t0 + b) * a.heads + h) * splits * a.rank + r;
+        if (ml) {
+#pragma unroll 4
+          for (int s = 0; s < splits; ++s) {
+            const float c = coef[b][s];
+            const float4 u = *reinterpret_cast<const float4*>(p + static_cast<long long>(s) * a.rank);
+            v.x += c * u.x; v.y += c * u.y; v.z += c * u.z; v.w += c * u.w;
+          }
+        } else {
+          v = *reinterpret_cast<const float4*>(p);
+        }
+      }
+      *reinterpret_cast<float4*>(os + i) = v;
+    }
+  } else {
+    for (int i = threadIdx.x; i < RT * a.rank; i += blockDim.x) {
+      const int b = i / a.rank, r = i - b * a.rank;
+      float v = 0.f;
+      if (b < rows) {
+        const float* p = o + (static_cast<long long>(t0 + b) * a.heads + h) * splits * a.rank + r;
+        if (ml) {
+          for (int s = 0; s < splits; ++s) v += coef[b][s] * p[static_cast<long long>(s) * a.rank];
+        } else {
+          v = p[0];
+        }
+      }
+      os[i] = v;
     }
   }
+  __syncthreads();
+  float acc[VB][RT];
+#pragma unroll
+  for (int i = 0; i < VB; ++i)
+#pragma unroll
+    for (int b = 0; b < RT; ++b) acc[i][b] = 0.f;
+  if (vec) {
+    for (int base = 0; base < a.rank; base += WC * 32 * N) {
+      if (base > 0) fetch(base);
+#pragma unroll
+      for (int k = 0; k < WC; ++k) {
+        const int r = base + (k * 32 + lane) * N;
+        if (r >= a.rank) continue;
+#pragma unroll
+        for (int b = 0; b < RT; ++b) {
+          float x[N];
+#pragma unroll
+          for (int j = 0; j < N; j += 4) {
+            const float4 u = *reinterpret_cast<const float4*>(os + b * a.rank + r + j);
+            x[j] = u.x; x[j + 1] = u.y; x[j + 2] = u.z; x[j + 3] = u.w;
+          }
+#pragma unroll
+          for (int i = 0; i < VB; ++i)
+#pragma unroll
+            for (int j = 0; j < N; ++j) acc[i][b] += w[i][k][j] * x[j];
+        }
+      }
+    }
+  } else {
+    for (int r = lane; r < a.rank; r += 32)
+#pragma unroll
+      for (int i = 0; i < VB; ++i) {
+        const float x = v0 + i < a.vdim ? to_f(wv[static_cast<long long>(v0 + i) * a.rank + r]) : 0.f;
+#pragma unroll
+        for (int b = 0; b < RT; ++b) acc[i][b] += x * os[b * a.rank + r];
+      }
+  }
+#pragma unroll
+  for (int i = 0; i < VB; ++i)
+#pragma unroll
+    for (int b = 0; b < RT; ++b) {
+      const float v = warp_sum(acc[i][b]);
+      if (lane == 0 && b < rows && v0 + i < a.vdim) cat[static_cast<long long>(t0 + b) * ldc + h * a.vdim + v0 + i] = from_f<T>(v);
+    }
 }
 
 // ------------------------------------------------------------------------------------------------ plain attention
@@ -236,21 +364,28 @@ __device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint3
 
 __host__ __device__ inline int decode_k(int rank, int rot) { return (rank + rot + 31) / 32 * 32; }
 
-// CTA = (sequence, group of MT * 16 heads, split). Scores: a warp owns 8 of the stage's 64 tokens; outputs: a warp owns an
-// eighth of the latent columns. Rows of a stage are read from the cache once for all heads of the group.
+// CTA = (sequence, group of MT * 16 heads, split). Warp (wm, wt): head tile wm; scores of the wt-th token group, outputs of the
+// wt-th group of latent columns. Rows of a stage are read from the cache once for all heads of the group; queries stay in
+// registers (as far as they fit: the first QI chunks of 32), so that shared memory carries little more than the rows.
 template <int MT>
 __global__ void __launch_bounds__(DW * 32) latent_decode_kernel(const HyLatent a, const bf16* __restrict__ ql, int qld,
                                                                 const int* __restrict__ seq_lens, int splits,
                                                                 float* __restrict__ po, float* __restrict__ pml) {
+  constexpr int NG = DW / MT;           // token groups, column groups
+  constexpr int KI = 18;                // 32-wide chunks of a query at most (576 values)
+  constexpr int QI = MT == 1 ? 18 : 10; // of which in registers
+  constexpr int NTM = 8 * MT;           // 8-wide output tiles per warp at most (512 columns over NG warps)
   extern __shared__ __align__(16) unsigned char raw[];
+  __shared__ int slot_s[2][TOK];
   const int KP = decode_k(a.rank, a.rot), ld = KP + 8;
   bf16* Ks = reinterpret_cast<bf16*>(raw);             // [2][TOK][ld]
   bf16* Qs = Ks + 2 * TOK * ld;                        // [MT * 16][ld]
   bf16* Ps = Qs + MT * 16 * ld;                        // [MT * 16][PLD]
-  float* wmax = reinterpret_cast<float*>(Ps + MT * 16 * PLD);  // [DW][MT * 16]
-  float* wsum = wmax + DW * MT * 16;                   // [DW][MT * 16]
+  float* wmax = reinterpret_cast<float*>(Ps + MT * 16 * PLD);  // [NG][MT * 16]
+  float* wsum = wmax + DW * MT * 16;                   // [NG][MT * 16]
   const int b = blockIdx.x, h0 = blockIdx.y * MT * 16, split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int wm = warp % MT, wt = warp / MT;
   int len = seq_lens[b];
   const long long cap = static_cast<long long>(a.max_pages) * a.page_size;
   if (len < 0 || len > cap) {
@@ -264,38 +399,55 @@ __global__ void __launch_bounds__(DW * 32) latent_decode_kernel(const HyLatent a
   const int n_ch = (t_hi - t_lo + TOK - 1) / TOK;
   const int chunks = KP / 8, wchunks = a.width / 8;
 
+  auto find_slots = [&](int ch) {  // by the first TOK threads, a barrier before they are used
+    if (threadIdx.x >= TOK || ch >= n_ch) return;
+    const int t = t_lo + ch * TOK + static_cast<int>(threadIdx.x);
+    long long slot = -1;
+    if (t < t_hi) {
+      slot = row_slot(a, b, t);
+      if (slot < 0 && a.status) atomicCAS(a.status, 0, 9);
+    }
+    slot_s[ch & 1][threadIdx.x] = static_cast<int>(slot);
+  };
   auto issue = [&](int ch, int stage) {
-    for (int i = threadIdx.x; i < TOK * chunks; i += DW * 32) {
-      const int r = i / chunks, c = i - r * chunks, t = t_lo + ch * TOK + r;
-      long long slot = -1;
-      if (t < t_hi) {
-        slot = row_slot(a, b, t);
-        if (slot < 0 && c == 0 && a.status) atomicCAS(a.status, 0, 9);
+#pragma unroll 2
+    for (int r = warp; r < TOK; r += DW) {
+      const int slot = slot_s[ch & 1][r];
+      const bf16* src = static_cast<const bf16*>(a.rows) + static_cast<long long>(slot < 0 ? 0 : slot) * a.width;
+      const uint32_t dst = s_u32(Ks + (stage * TOK + r) * ld);
+      for (int c = lane; c < chunks; c += 32) {
+        const bool ok = slot >= 0 && c < wchunks;
+        cp_async16(dst + c * 16, src + (ok ? c * 8 : 0), ok ? 16 : 0);
       }
-      const bool ok = slot >= 0 && c < wchunks;
-      cp_async16(s_u32(Ks + (stage * TOK + r) * ld + c * 8), static_cast<const bf16*>(a.rows) + (ok ? slot * a.width + c * 8 : 0), ok ? 16 : 0);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
+  find_slots(0);
+  for (int r = warp; r < MT * 16; r += DW)
+    for (int c = lane * 8; c < KP; c += 256) {
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (h0 + r < a.heads && c < qld) v = *reinterpret_cast<const uint4*>(ql + (static_cast<long long>(b) * a.heads + h0 + r) * qld + c);
+      *reinterpret_cast<uint4*>(Qs + r * ld + c) = v;
+    }
+  __syncthreads();
   if (n_ch > 0) issue(0, 0);
-  for (int i = threadIdx.x; i < MT * 16 * chunks; i += DW * 32) {
-    const int r = i / chunks, c = (i - r * chunks) * 8;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (h0 + r < a.heads && c < qld) v = *reinterpret_cast<const uint4*>(ql + (static_cast<long long>(b) * a.heads + h0 + r) * qld + c);
-    *reinterpret_cast<uint4*>(Qs + r * ld + c) = v;
-  }
+  find_slots(1);
+  const uint32_t qaddr = s_u32(Qs + (wm * 16 + (lane & 15)) * ld + ((lane >> 4) << 3));
+  uint32_t qa[QI][2][4];
+#pragma unroll
+  for (int i = 0; i < QI; ++i)
+    if (i * 32 < KP) {
+      ldsm4(qaddr + i * 64, qa[i][0]);
+      ldsm4(qaddr + i * 64 + 32, qa[i][1]);
+    }
   const float sl2 = a.scale * 1.4426950408889634f;
-  float m_run[MT][2], l_run[MT][2], o[MT][8][4];
+  float m_run[2] = {-FLT_MAX, -FLT_MAX}, l_run[2] = {0.f, 0.f}, o[NTM][4];
 #pragma unroll
-  for (int mt = 0; mt < MT; ++mt) {
-    m_run[mt][0] = m_run[mt][1] = -FLT_MAX;
-    l_run[mt][0] = l_run[mt][1] = 0.f;
-#pragma unroll
-    for (int j = 0; j < 8; ++j) o[mt][j][0] = o[mt][j][1] = o[mt][j][2] = o[mt][j][3] = 0.f;
-  }
-  const int NT = (a.rank + 63) / 64;      // 8-wide column tiles per warp
-  const int col0 = warp * NT * 8;
+  for (int j = 0; j < NTM; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  const int NT = (a.rank + 8 * NG - 1) / (8 * NG);  // 8-wide column tiles per warp
+  const int col0 = wt * NT * 8;
   const int r0 = lane >> 2;
+  __syncthreads();  // slots of the second stage
   for (int ch = 0; ch < n_ch; ++ch) {
     const int stage = ch & 1;
     if (ch + 1 < n_ch) {
@@ -305,114 +457,120 @@ __global__ void __launch_bounds__(DW * 32) latent_decode_kernel(const HyLatent a
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
+    find_slots(ch + 2);  // (the ones of chunk ch have been used)
     const bf16* Kst = Ks + stage * TOK * ld;
     float sc[MT][4];
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt) sc[mt][0] = sc[mt][1] = sc[mt][2] = sc[mt][3] = 0.f;
-    const uint32_t kaddr = s_u32(Kst + (warp * 8 + (lane & 7)) * ld + (lane >> 3) * 8);
-    const uint32_t qaddr = s_u32(Qs + (lane & 15) * ld + ((lane >> 4) << 3));
-#pragma unroll 2
-    for (int k0 = 0; k0 < KP; k0 += 32) {
-      uint32_t kb[4];
-      ldsm4(kaddr + k0 * 2, kb);
+    for (int nt = 0; nt < MT; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
+    const uint32_t kaddr = s_u32(Kst + (wt * 8 * MT + (lane & 7)) * ld + (lane >> 3) * 8);
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) {
-        uint32_t qa[4];
-        ldsm4(qaddr + (mt * 16 * ld + k0) * 2, qa);
-        mma(sc[mt], qa, kb[0], kb[1]);
-        ldsm4(qaddr + (mt * 16 * ld + k0 + 16) * 2, qa);
-        mma(sc[mt], qa, kb[2], kb[3]);
+    for (int i = 0; i < KI; ++i) {
+      if (i * 32 >= KP) break;
+      uint32_t q0[4], q1[4];
+      if (i < QI) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          q0[k] = qa[i < QI ? i : 0][0][k];
+          q1[k] = qa[i < QI ? i : 0][1][k];
+        }
+      } else {
+        ldsm4(qaddr + i * 64, q0);
+        ldsm4(qaddr + i * 64 + 32, q1);
+      }
+#pragma unroll
+      for (int nt = 0; nt < MT; ++nt) {
+        uint32_t kb[4];
+        ldsm4(kaddr + (nt * 8 * ld + i * 32) * 2, kb);
+        mma(sc[nt], q0, kb[0], kb[1]);
+        mma(sc[nt], q1, kb[2], kb[3]);
       }
     }
-    const int tok = t_lo + ch * TOK + warp * 8 + (lane & 3) * 2;
+    const int tok = t_lo + ch * TOK + wt * 8 * MT + (lane & 3) * 2;
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt) {
+    for (int r = 0; r < 2; ++r) {
+      float mx = -FLT_MAX;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) sc[mt][e] = tok + (e & 1) < t_hi ? sc[mt][e] * sl2 : -FLT_MAX;
+      for (int nt = 0; nt < MT; ++nt)
 #pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        float mx = fmaxf(sc[mt][2 * r], sc[mt][2 * r + 1]);
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-        if ((lane & 3) == 0) wmax[warp * MT * 16 + mt * 16 + r0 + 8 * r] = mx;
+        for (int e = 0; e < 2; ++e) {
+          float& v = sc[nt][2 * r + e];
+          v = tok + nt * 8 + e < t_hi ? v * sl2 : -FLT_MAX;
+          mx = fmaxf(mx, v);
+        }
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+      if ((lane & 3) == 0) wmax[wt * MT * 16 + wm * 16 + r0 + 8 * r] = mx;
+    }
+    __syncthreads();
+    float corr[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int row = wm * 16 + r0 + 8 * r;
+      float mn = m_run[r];
+#pragma unroll
+      for (int w = 0; w < NG; ++w) mn = fmaxf(mn, wmax[w * MT * 16 + row]);
+      corr[r] = m_run[r] == -FLT_MAX ? 0.f : exp2f(m_run[r] - mn);
+      m_run[r] = mn;
+      l_run[r] *= corr[r];
+#pragma unroll
+      for (int nt = 0; nt < MT; ++nt) {
+        const float p0 = sc[nt][2 * r] == -FLT_MAX ? 0.f : exp2f(sc[nt][2 * r] - mn);
+        const float p1 = sc[nt][2 * r + 1] == -FLT_MAX ? 0.f : exp2f(sc[nt][2 * r + 1] - mn);
+        l_run[r] += p0 + p1;
+        *reinterpret_cast<__nv_bfloat162*>(Ps + row * PLD + (wt * MT + nt) * 8 + (lane & 3) * 2) = __floats2bfloat162_rn(p0, p1);
       }
     }
     __syncthreads();
-    float corr[MT][2];
+    if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-      for (int r = 0; r < 2; ++r) {
-        const int row = mt * 16 + r0 + 8 * r;
-        float mn = m_run[mt][r];
-#pragma unroll
-        for (int w = 0; w < DW; ++w) mn = fmaxf(mn, wmax[w * MT * 16 + row]);
-        corr[mt][r] = m_run[mt][r] == -FLT_MAX ? 0.f : exp2f(m_run[mt][r] - mn);
-        m_run[mt][r] = mn;
-        const float p0 = sc[mt][2 * r] == -FLT_MAX ? 0.f : exp2f(sc[mt][2 * r] - mn);
-        const float p1 = sc[mt][2 * r + 1] == -FLT_MAX ? 0.f : exp2f(sc[mt][2 * r + 1] - mn);
-        l_run[mt][r] = l_run[mt][r] * corr[mt][r] + p0 + p1;
-        *reinterpret_cast<__nv_bfloat162*>(Ps + row * PLD + warp * 8 + (lane & 3) * 2) = __floats2bfloat162_rn(p0, p1);
+      for (int j = 0; j < NTM; ++j) {
+        o[j][0] *= corr[0]; o[j][1] *= corr[0];
+        o[j][2] *= corr[1]; o[j][3] *= corr[1];
       }
-    __syncthreads();
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        o[mt][j][0] *= corr[mt][0]; o[mt][j][1] *= corr[mt][0];
-        o[mt][j][2] *= corr[mt][1]; o[mt][j][3] *= corr[mt][1];
-      }
+    }
 #pragma unroll
     for (int k0 = 0; k0 < TOK; k0 += 16) {
-      uint32_t pa[MT][4];
+      uint32_t pa[4];
+      ldsm4(s_u32(Ps + (wm * 16 + (lane & 15)) * PLD + k0 + ((lane >> 4) << 3)), pa);
+      const uint32_t vrow = s_u32(Kst + (k0 + (lane & 7) + (((lane >> 3) & 1) << 3)) * ld);
 #pragma unroll
-      for (int mt = 0; mt < MT; ++mt) ldsm4(s_u32(Ps + (mt * 16 + (lane & 15)) * PLD + k0 + ((lane >> 4) << 3)), pa[mt]);
-      const bf16* vrow = Kst + (k0 + (lane & 7) + (((lane >> 3) & 1) << 3)) * ld;
-#pragma unroll
-      for (int jp = 0; jp < 4; ++jp) {
+      for (int jp = 0; jp < NTM / 2; ++jp) {
         if (2 * jp >= NT) break;
         const int c = col0 + jp * 16 + ((lane >> 4) << 3);
         uint32_t vb[4];
-        ldsm4t(s_u32(vrow + min(c, KP - 8)), vb);  // (columns past the row end belong to tiles that are not stored)
-#pragma unroll
-        for (int mt = 0; mt < MT; ++mt) {
-          mma(o[mt][2 * jp], pa[mt], vb[0], vb[1]);
-          mma(o[mt][2 * jp + 1], pa[mt], vb[2], vb[3]);
-        }
+        ldsm4t(vrow + min(c, KP - 8) * 2, vb);  // (columns past the row end belong to tiles that are not stored)
+        mma(o[2 * jp], pa, vb[0], vb[1]);
+        mma(o[2 * jp + 1], pa, vb[2], vb[3]);
       }
     }
     __syncthreads();  // the stage is refilled next
   }
-  // sums over the warps
+  // sums over the token groups
 #pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      float l = l_run[mt][r];
-      l += __shfl_xor_sync(0xffffffffu, l, 1);
-      l += __shfl_xor_sync(0xffffffffu, l, 2);
-      if ((lane & 3) == 0) wsum[warp * MT * 16 + mt * 16 + r0 + 8 * r] = l;
-    }
+  for (int r = 0; r < 2; ++r) {
+    float l = l_run[r];
+    l += __shfl_xor_sync(0xffffffffu, l, 1);
+    l += __shfl_xor_sync(0xffffffffu, l, 2);
+    if ((lane & 3) == 0) wsum[wt * MT * 16 + wm * 16 + r0 + 8 * r] = l;
+  }
   __syncthreads();
 #pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int row = mt * 16 + r0 + 8 * r, h = h0 + row;
-      if (h >= a.heads) continue;
-      const long long base = (static_cast<long long>(b) * a.heads + h) * splits + split;
-      if (warp == 0 && (lane & 3) == 0) {
-        float l = 0.f;
-        for (int w = 0; w < DW; ++w) l += wsum[w * MT * 16 + row];
-        pml[base * 2] = m_run[mt][r];
-        pml[base * 2 + 1] = l;
-      }
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const int c = col0 + j * 8 + (lane & 3) * 2;
-        if (j < NT && c < a.rank) *reinterpret_cast<float2*>(po + base * a.rank + c) = make_float2(o[mt][j][2 * r], o[mt][j][2 * r + 1]);
-      }
+  for (int r = 0; r < 2; ++r) {
+    const int row = wm * 16 + r0 + 8 * r, h = h0 + row;
+    if (h >= a.heads) continue;
+    const long long base = (static_cast<long long>(b) * a.heads + h) * splits + split;
+    if (wt == 0 && (lane & 3) == 0) {
+      float l = 0.f;
+      for (int w = 0; w < NG; ++w) l += wsum[w * MT * 16 + row];
+      pml[base * 2] = m_run[r];
+      pml[base * 2 + 1] = l;
     }
+#pragma unroll
+    for (int j = 0; j < NTM; ++j) {
+      const int c = col0 + j * 8 + (lane & 3) * 2;
+      if (j < NT && c < a.rank) *reinterpret_cast<float2*>(po + base * a.rank + c) = make_float2(o[j][2 * r], o[j][2 * r + 1]);
+    }
+  }
 }
 
 size_t decode_smem(int MT, int rank, int rot) {
@@ -470,23 +628,31 @@ __global__ void __launch_bounds__(256) pad_q_kernel(const HyLatent a, const bf16
 template <typename T, typename O>
 int absorb_t(const HyLatent& a, const void* q, const int* positions, int n, void* ql, int qld, cudaStream_t s) {
   const int nr = (a.rank + 127) / 128;
-  const size_t smem = sizeof(float) * TT * a.dim;
-  auto kern = absorb_q_kernel<T, O>;
+  auto go = [&](auto kern, size_t smem) -> int {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+    kern<<<dim3(nr + 1, a.heads, (n + TT - 1) / TT), 256, smem, s>>>(a, static_cast<const T*>(q), positions, n, static_cast<O*>(ql), qld, nr);
+    return static_cast<int>(cudaGetLastError());
+  };
+  if constexpr (sizeof(T) == 2)
+    if (a.rank % 8 == 0 && aligned16<T>(a.ukv, a.rank)) return go(absorb_q_kernel<T, O, true>, sizeof(float) * (TT * a.dim + 8 * TT * 128));
+  return go(absorb_q_kernel<T, O, false>, sizeof(float) * TT * a.dim);
+}
+
+template <typename T, int RT>
+int up_rt(const HyLatent& a, const float* o, const float* ml, int splits, int n, void* cat, int ldc, cudaStream_t s) {
+  const size_t smem = sizeof(float) * RT * a.rank;
+  auto kern = latent_up_kernel<T, RT>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
-  kern<<<dim3(nr + 1, a.heads, (n + TT - 1) / TT), 128, smem, s>>>(a, static_cast<const T*>(q), positions, n, static_cast<O*>(ql), qld, nr);
+  kern<<<dim3((a.vdim + 31) / 32, a.heads, (n + RT - 1) / RT), 256, smem, s>>>(a, o, ml, splits, n, static_cast<T*>(cat), ldc,
+                                                                              a.rank % Vec<T>::N == 0 && aligned16<T>(a.ukv, a.rank));
   return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T>
 int up_t(const HyLatent& a, const float* o, const float* ml, int splits, int n, void* cat, int ldc, cudaStream_t s) {
-  const size_t smem = sizeof(float) * TT * a.rank;
-  auto kern = latent_up_kernel<T>;
-  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-  if (e != cudaSuccess) return static_cast<int>(e);
-  kern<<<dim3((a.vdim + 31) / 32, a.heads, (n + TT - 1) / TT), 128, smem, s>>>(a, o, ml, splits, n, static_cast<T*>(cat), ldc,
-                                                                              a.rank % Vec<T>::N == 0);
-  return static_cast<int>(cudaGetLastError());
+  return n <= 2 ? up_rt<T, 1>(a, o, ml, splits, n, cat, ldc, s) : up_rt<T, 4>(a, o, ml, splits, n, cat, ldc, s);
 }
 
 template <typename T>
@@ -537,12 +703,12 @@ int hy_latent_up(bool f32, const HyLatent& a, const float* o, const float* ml, i
 }
 
 bool hy_latent_decode_supported(int heads, int rank, int rot, int width) {
-  return heads >= 1 && rank % 8 == 0 && rank >= 8 && rank <= 512 && width % 8 == 0 && decode_smem(heads > 16 ? 2 : 1, rank, rot) <= 227 * 1024;
+  return heads >= 1 && rank % 8 == 0 && rank >= 8 && rank <= 512 && decode_k(rank, rot) <= 576 && width % 8 == 0 && decode_smem(heads > 16 ? 2 : 1, rank, rot) <= 227 * 1024;
 }
 
 int hy_latent_decode(const HyLatent& a, const void* ql, int qld, const int* seq_lens, int B, int splits, float* o, float* ml,
                      cudaStream_t s) {
-  if (!hy_latent_decode_supported(a.heads, a.rank, a.rot, a.width) || qld % 8 != 0 || splits < 1 || splits > 64)
+  if (!hy_latent_decode_supported(a.heads, a.rank, a.rot, a.width) || qld % 8 != 0 || splits < 1 || splits > 64 || a.num_slots > 0x7fffffffll)
     return static_cast<int>(cudaErrorInvalidValue);
   const bf16* q = static_cast<const bf16*>(ql);
   return a.heads > 16 ? decode_t<2>(a, q, qld, seq_lens, B, splits, o, ml, s) : decode_t<1>(a, q, qld, seq_lens, B, splits, o, ml, s);

@@ -79,38 +79,62 @@ __global__ void __launch_bounds__(128) conv_kernel(const HyMamba a, const int4* 
   }
 }
 
-// Two channels per thread for bf16 rows whose columns start on even offsets, four taps.
-__global__ void __launch_bounds__(128) conv4_pair_kernel(const HyMamba a, const int4* __restrict__ tiles, bf16* __restrict__ xbc) {
+// Eight channels per thread for bf16 rows whose columns start on 16-byte boundaries, four taps.
+__global__ void __launch_bounds__(128) conv4_vec_kernel(const HyMamba a, const int4* __restrict__ tiles, bf16* __restrict__ xbc) {
   const int4 tl = tiles[blockIdx.x];
   const int inner = a.heads * a.P, ch = inner + 2 * a.groups * a.N;
-  const int c = (blockIdx.y * 128 + threadIdx.x) * 2;
+  const int c = (blockIdx.y * 128 + threadIdx.x) * 8;
   if (c >= ch) return;
   const int seq = tl.x, row0 = tl.y, n = tl.z;
   const int first = a.cu[seq], ctx = a.ctx[seq];
   const bf16* in = static_cast<const bf16*>(a.proj) + inner + c;
   const bf16* ring = static_cast<const bf16*>(a.ring) + static_cast<long long>(a.slots[seq]) * 4 * ch + c;
-  auto ld2 = [](const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); };
-  auto input = [&](int r, int back) -> float2 {
-    const int q = r - back;
-    if (q >= first) return ld2(in + static_cast<long long>(q) * a.ld);
-    const int p = ctx + q - first;
-    return p < 0 ? make_float2(0.f, 0.f) : ld2(ring + static_cast<long long>(p & 3) * ch);
-  };
-  const bf16* w = static_cast<const bf16*>(a.conv_w) + static_cast<long long>(c) * 4;
-  float2 wv[4], h0 = input(row0, 3), h1 = input(row0, 2), h2 = input(row0, 1);
+  float w[4][8], bias[8], h[3][8];
+  {
+    const bf16* wp = static_cast<const bf16*>(a.conv_w) + static_cast<long long>(c) * 4;  // [channel][tap]
 #pragma unroll
-  for (int k = 0; k < 4; ++k) wv[k] = make_float2(to_f(w[k]), to_f(w[4 + k]));
-  const float2 bias = ld2(static_cast<const bf16*>(a.conv_b) + c);
-#pragma unroll 4
-  for (int t = 0; t < n; ++t) {
-    const float2 h3 = ld2(in + static_cast<long long>(row0 + t) * a.ld);
-    float x = bias.x, y = bias.y;
-    x += wv[0].x * h0.x; y += wv[0].y * h0.y;
-    x += wv[1].x * h1.x; y += wv[1].y * h1.y;
-    x += wv[2].x * h2.x; y += wv[2].y * h2.y;
-    x += wv[3].x * h3.x; y += wv[3].y * h3.y;
-    h0 = h1; h1 = h2; h2 = h3;
-    *reinterpret_cast<__nv_bfloat162*>(xbc + static_cast<long long>(row0 + t) * ch + c) = __floats2bfloat162_rn(silu_f(x), silu_f(y));
+    for (int k = 0; k < 4; ++k) {
+      float t[8];
+      Vec<bf16>::load(wp + k * 8, t);  // channels 2k, 2k + 1
+#pragma unroll
+      for (int j = 0; j < 8; ++j) w[j & 3][2 * k + (j >> 2)] = t[j];
+    }
+  }
+  Vec<bf16>::load(static_cast<const bf16*>(a.conv_b) + c, bias);
+#pragma unroll
+  for (int k = 0; k < 3; ++k) {  // inputs of the three tokens before the tile
+    const int q = row0 - 3 + k, p = ctx + q - first;
+    if (q >= first)
+      Vec<bf16>::load(in + static_cast<long long>(q) * a.ld, h[k]);
+    else if (p >= 0)
+      Vec<bf16>::load(ring + static_cast<long long>(p & 3) * ch, h[k]);
+    else
+#pragma unroll
+      for (int j = 0; j < 8; ++j) h[k][j] = 0.f;
+  }
+  constexpr int U = 4;  // tokens whose loads are in flight
+  for (int t0 = 0; t0 < n; t0 += U) {
+    uint4 raw[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (t0 + u < n) raw[u] = *reinterpret_cast<const uint4*>(in + static_cast<long long>(row0 + t0 + u) * a.ld);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (t0 + u >= n) break;
+      const uint32_t r[4] = {raw[u].x, raw[u].y, raw[u].z, raw[u].w};
+      float o[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r[j >> 1]));
+        const float x = (j & 1) ? f.y : f.x;
+        const float v = bias[j] + w[0][j] * h[0][j] + w[1][j] * h[1][j] + w[2][j] * h[2][j] + w[3][j] * x;
+        h[0][j] = h[1][j];
+        h[1][j] = h[2][j];
+        h[2][j] = x;
+        o[j] = __fdividef(v, 1.f + __expf(-v));
+      }
+      Vec<bf16>::store(xbc + static_cast<long long>(row0 + t0 + u) * ch + c, o);
+    }
   }
 }
 
@@ -276,280 +300,386 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
   lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
-// dt and the running sum of -exp(A_log) dt over the chunk: smem dt[Q], acum[Q] (zeros past n keep the sum flat)
-__device__ __forceinline__ void chunk_decay(const HyMamba& a, int h, int row0, int n, float* dts, float* acum) {
-  const int inner = a.heads * a.P, ch = inner + 2 * a.groups * a.N;
-  if (threadIdx.x < Q) {
-    float dt = 0.f;
-    if (static_cast<int>(threadIdx.x) < n)
-      dt = softplus_f(to_f(static_cast<const bf16*>(a.proj)[static_cast<long long>(row0 + threadIdx.x) * a.ld + inner + ch + h]) +
-                      to_f(static_cast<const bf16*>(a.dt_bias)[h]));
-    dts[threadIdx.x] = dt;
-    float v = -expf(to_f(static_cast<const bf16*>(a.A_log)[h])) * dt;
-    const int lane = threadIdx.x & 31;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const float u = __shfl_up_sync(0xffffffffu, v, o);
-      if (lane >= o) v += u;
-    }
-    acum[threadIdx.x] = v;
-  }
-  __syncthreads();
-  float base = 0.f;
-  if (threadIdx.x < Q)
-    for (int w = 0; w < static_cast<int>(threadIdx.x >> 5); ++w) base += acum[w * 32 + 31];
-  __syncthreads();
-  if (threadIdx.x < Q) acum[threadIdx.x] += base;
-  __syncthreads();
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src, int bytes) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void cp_wait_all() {
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
 }
 
-// rows [n, w] of xbc starting at column c0 into smem [Q][ld], zero filled to wp columns and Q rows
-__device__ __forceinline__ void load_tile(const bf16* __restrict__ xbc, long long ch, int row0, int n, int c0, int w, int wp,
-                                          bf16* dst, int ld, bool vec) {
+constexpr float LOG2E = 1.4426950408889634f;
+constexpr int MAX_HB = 8;        // heads of one group a CTA works on (a warp computes the decays of each)
+
+// Warp w: step sizes of head h0 + w over the chunk and the running sum of -exp(A_log) dt in units of log2. Tokens past n get
+// dt = 0, so the sum stays flat.
+__device__ __forceinline__ void chunk_decays(const HyMamba& a, int h0, int nh, int row0, int n, float* dts, float* acum) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (warp >= nh) return;
+  const int h = h0 + warp, inner = a.heads * a.P, ch = inner + 2 * a.groups * a.N;
+  const bf16* col = static_cast<const bf16*>(a.proj) + inner + ch + h;
+  const float bias = to_f(static_cast<const bf16*>(a.dt_bias)[h]), A = -expf(to_f(static_cast<const bf16*>(a.A_log)[h])) * LOG2E;
+  float dt[Q / 32], v[Q / 32], run = 0.f;
+#pragma unroll
+  for (int i = 0; i < Q / 32; ++i) {
+    const int t = lane * (Q / 32) + i;
+    dt[i] = t < n ? softplus_f(to_f(col[static_cast<long long>(row0 + t) * a.ld]) + bias) : 0.f;
+    run += A * dt[i];
+    v[i] = run;
+  }
+  float base = run;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float u = __shfl_up_sync(0xffffffffu, base, o);
+    if (lane >= o) base += u;
+  }
+  base -= run;
+#pragma unroll
+  for (int i = 0; i < Q / 32; ++i) {
+    dts[warp * Q + lane * (Q / 32) + i] = dt[i];
+    acum[warp * Q + lane * (Q / 32) + i] = base + v[i];
+  }
+}
+
+// rows [n, w] of a row-major bf16 matrix (pitch `pitch`) into smem [rows][ld], zero filled to wp columns; vec: by 16-byte
+// asynchronous copies the caller waits for
+__device__ __forceinline__ void load_tile(const bf16* __restrict__ src, long long pitch, int n, int w, int rows, int wp, bf16* dst,
+                                          int ld, bool vec) {
   if (vec) {
     const int per = wp / 8;
-    for (int i = threadIdx.x; i < Q * per; i += CW * 32) {
+    for (int i = threadIdx.x; i < rows * per; i += CW * 32) {
       const int r = i / per, c = (i - r * per) * 8;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (r < n && c < w) v = *reinterpret_cast<const uint4*>(xbc + (row0 + r) * ch + c0 + c);
-      *reinterpret_cast<uint4*>(dst + r * ld + c) = v;
+      const bool ok = r < n && c < w;
+      cp16(s_u32(dst + r * ld + c), src + (ok ? r * pitch + c : 0), ok ? 16 : 0);
     }
   } else {
-    for (int i = threadIdx.x; i < Q * wp; i += CW * 32) {
+    for (int i = threadIdx.x; i < rows * wp; i += CW * 32) {
       const int r = i / wp, c = i - r * wp;
-      dst[r * ld + c] = (r < n && c < w) ? xbc[(row0 + r) * ch + c0 + c] : __float2bfloat16(0.f);
+      dst[r * ld + c] = (r < n && c < w) ? src[r * pitch + c] : __float2bfloat16(0.f);
     }
   }
 }
 
-// (1) work[chunk, h, p, n] = sum_t exp(acum_end - acum_t) dt_t x_t[p] B_t[n];  decay[chunk, h] = exp(acum_end)
-__global__ void __launch_bounds__(CW * 32) chunk_state_kernel(const HyMamba a, const bf16* __restrict__ xbc,
-                                                              const int4* __restrict__ chunks, float* __restrict__ work,
-                                                              float* __restrict__ decay, bool vec) {
+// (1) work[chunk, h, p, n] = sum_t exp(acum_end - acum_t) dt_t x_t[p] B_t[n];  decay[chunk, h] = exp(acum_end). A CTA takes
+// several heads of a group: their B is the same tile.
+template <int PT>
+__global__ void __launch_bounds__(CW * 32, 2) chunk_state_kernel(const HyMamba a, const bf16* __restrict__ xbc,
+                                                                 const int4* __restrict__ chunks, int hb, float* __restrict__ work,
+                                                                 float* __restrict__ decay, bool vec) {
   extern __shared__ __align__(16) unsigned char raw[];
   const int4 ck = chunks[blockIdx.x];
-  const int h = blockIdx.y, row0 = ck.y, n = ck.z;
-  const int P = a.P, N = a.N, PP = (P + 15) / 16 * 16, NP = (N + 63) / 64 * 64;
-  const int inner = a.heads * P, ch = inner + 2 * a.groups * N, g = h / (a.heads / a.groups);
-  const int ldx = PP + LDX_PAD, ldb = NP + LDX_PAD;
+  const int row0 = ck.y, n = ck.z;
+  const int P = a.P, N = a.N, NP = (N + 63) / 64 * 64, hpg = a.heads / a.groups;
+  constexpr int PP = PT * 16, ldx = PP + LDX_PAD, XV = PP * Q / 8 / (CW * 32);
+  const int inner = a.heads * P, ch = inner + 2 * a.groups * N;
+  const int per_group = (hpg + hb - 1) / hb, g = blockIdx.y / per_group;
+  const int h0 = g * hpg + (blockIdx.y - g * per_group) * hb, nh = min(hb, (g + 1) * hpg - h0);
+  const int ldb = NP + LDX_PAD;
   bf16* xh = reinterpret_cast<bf16*>(raw);   // [Q][ldx] weighted x, high part
   bf16* xl = xh + Q * ldx;                   // low part
   bf16* Bs = xl + Q * ldx;                   // [Q][ldb]
-  float* dts = reinterpret_cast<float*>(Bs + Q * ldb);
-  float* acum = dts + Q;
-  chunk_decay(a, h, row0, n, dts, acum);
-  load_tile(xbc, ch, row0, n, inner + g * N, N, NP, Bs, ldb, vec);
-  const float end = acum[Q - 1];
-  for (int i = threadIdx.x; i < Q * (PP / 2); i += CW * 32) {
-    const int r = i / (PP / 2), c = (i - r * (PP / 2)) * 2;
-    float u = 0.f, v = 0.f;
-    if (r < n) {
-      const float w = expf(end - acum[r]) * dts[r];
+  float* dts = reinterpret_cast<float*>(Bs + Q * ldb);  // [MAX_HB][Q]
+  float* acum = dts + MAX_HB * Q;
+  load_tile(xbc + static_cast<long long>(row0) * ch + inner + g * N, ch, n, N, Q, NP, Bs, ldb, vec);
+  uint4 xr[XV];
+  auto fetch = [&](int h) {
+#pragma unroll
+    for (int i = 0; i < XV; ++i) {
+      const int k = threadIdx.x + i * CW * 32, r = k / (PP / 8), c = (k - r * (PP / 8)) * 8;
+      xr[i] = make_uint4(0u, 0u, 0u, 0u);
+      if (r >= n || c >= P) continue;
       const bf16* src = xbc + static_cast<long long>(row0 + r) * ch + h * P + c;
-      if (c < P) u = w * to_f(src[0]);
-      if (c + 1 < P) v = w * to_f(src[1]);
+      if (vec) {
+        xr[i] = *reinterpret_cast<const uint4*>(src);
+      } else {
+        bf16 t[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) t[j] = c + j < P ? src[j] : __float2bfloat16(0.f);
+        xr[i] = *reinterpret_cast<const uint4*>(t);
+      }
     }
-    uint32_t hi, lo;
-    split2(u, v, hi, lo);
-    *reinterpret_cast<uint32_t*>(xh + r * ldx + c) = hi;
-    *reinterpret_cast<uint32_t*>(xl + r * ldx + c) = lo;
-  }
-  if (threadIdx.x == 0) decay[static_cast<long long>(blockIdx.x) * a.heads + h] = expf(end);
+  };
+  fetch(h0);
+  chunk_decays(a, h0, nh, row0, n, dts, acum);
+  cp_wait_all();
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  float* out = work + (static_cast<long long>(blockIdx.x) * a.heads + h) * P * N;
-  const int mt = PP / 16, nt = NP / 64;
-  for (int unit = warp; unit < mt * nt; unit += CW) {
-    const int m0 = (unit % mt) * 16, n0 = (unit / mt) * 64;
-    float acc[8][4];
+  const int nt = NP / 64;
+  for (int hi = 0; hi < nh; ++hi) {
+    const int h = h0 + hi;
+    const float* ac = acum + hi * Q;
+    const float* dt = dts + hi * Q;
+    const float end = ac[Q - 1];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
-    for (int k0 = 0; k0 < Q; k0 += 16) {
-      if (k0 >= n) break;
-      uint32_t ah[4], al[4];
-      // A = (weighted x)^T: rows p, contraction t; stored [t][p], so transpose while loading
-      const int ar = k0 + (lane & 7) + ((lane >> 4) << 3), ac = m0 + (((lane >> 3) & 1) << 3);
-      ldsm4t(s_u32(xh + ar * ldx + ac), ah);
-      ldsm4t(s_u32(xl + ar * ldx + ac), al);
+    for (int i = 0; i < XV; ++i) {
+      const int k = threadIdx.x + i * CW * 32, r = k / (PP / 8), c = (k - r * (PP / 8)) * 8;
+      const float w = ex2(end - ac[r]) * dt[r];
+      const uint32_t* q = reinterpret_cast<const uint32_t*>(&xr[i]);
+      uint32_t hi4[4], lo4[4];
 #pragma unroll
-      for (int jp = 0; jp < 4; ++jp) {
-        uint32_t b[4];
-        const int br = k0 + (lane & 7) + (((lane >> 3) & 1) << 3), bc = n0 + jp * 16 + ((lane >> 4) << 3);
-        ldsm4t(s_u32(Bs + br * ldb + bc), b);
-        mma(acc[2 * jp], ah, b[0], b[1]);
-        mma(acc[2 * jp], al, b[0], b[1]);
-        mma(acc[2 * jp + 1], ah, b[2], b[3]);
-        mma(acc[2 * jp + 1], al, b[2], b[3]);
+      for (int j = 0; j < 4; ++j) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q[j]));
+        split2(w * f.x, w * f.y, hi4[j], lo4[j]);
+      }
+      *reinterpret_cast<uint4*>(xh + r * ldx + c) = make_uint4(hi4[0], hi4[1], hi4[2], hi4[3]);
+      *reinterpret_cast<uint4*>(xl + r * ldx + c) = make_uint4(lo4[0], lo4[1], lo4[2], lo4[3]);
+    }
+    if (hi + 1 < nh) fetch(h + 1);
+    if (threadIdx.x == 0) decay[static_cast<long long>(blockIdx.x) * a.heads + h] = ex2(end);
+    __syncthreads();
+    float* out = work + (static_cast<long long>(blockIdx.x) * a.heads + h) * P * N;
+    for (int unit = warp; unit < PT * nt; unit += CW) {
+      const int m0 = (unit % PT) * 16, n0 = (unit / PT) * 64;
+      float acc[8][4];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+#pragma unroll 2
+      for (int k0 = 0; k0 < n; k0 += 16) {
+        uint32_t ah[4], al[4];
+        // A = (weighted x)^T: rows p, contraction t; stored [t][p], so transpose while loading
+        const int ar = k0 + (lane & 7) + ((lane >> 4) << 3), acol = m0 + (((lane >> 3) & 1) << 3);
+        ldsm4t(s_u32(xh + ar * ldx + acol), ah);
+        ldsm4t(s_u32(xl + ar * ldx + acol), al);
+#pragma unroll
+        for (int jp = 0; jp < 4; ++jp) {
+          uint32_t b[4];
+          const int br = k0 + (lane & 7) + (((lane >> 3) & 1) << 3), bc = n0 + jp * 16 + ((lane >> 4) << 3);
+          ldsm4t(s_u32(Bs + br * ldb + bc), b);
+          mma(acc[2 * jp], ah, b[0], b[1]);
+          mma(acc[2 * jp], al, b[0], b[1]);
+          mma(acc[2 * jp + 1], ah, b[2], b[3]);
+          mma(acc[2 * jp + 1], al, b[2], b[3]);
+        }
+      }
+      const int p0 = m0 + (lane >> 2);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const int c = n0 + j * 8 + (lane & 3) * 2;
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int p = p0 + e * 8;
+          if (p >= P) continue;
+          float* dst = out + static_cast<long long>(p) * N + c;
+          if ((N & 1) == 0) {
+            if (c < N) *reinterpret_cast<float2*>(dst) = make_float2(acc[j][2 * e], acc[j][2 * e + 1]);
+          } else {
+            if (c < N) dst[0] = acc[j][2 * e];
+            if (c + 1 < N) dst[1] = acc[j][2 * e + 1];
+          }
+        }
       }
     }
-    const int p0 = m0 + (lane >> 2);
-#pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      const int c = n0 + j * 8 + (lane & 3) * 2;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int p = p0 + (e >> 1) * 8, cc = c + (e & 1);
-        if (p < P && cc < N) out[static_cast<long long>(p) * N + cc] = acc[j][e];
-      }
-    }
+    __syncthreads();
   }
 }
 
-// (2) replace every chunk's contribution by the state before the chunk; leave the state after the last in the slot
+// (2) the state before every chunk, as two bf16 planes (high part, low part) [chunk, h, 2, P, N]; the state after the last chunk
+// goes to the sequence's row
+template <int V>
 __global__ void __launch_bounds__(256) chunk_pass_kernel(const HyMamba a, const int* __restrict__ first_chunk,
-                                                         const float* __restrict__ decay, float* __restrict__ work) {
+                                                         const float* __restrict__ decay, const float* __restrict__ work,
+                                                         bf16* __restrict__ before) {
   const int h = blockIdx.y, seq = blockIdx.z;
   const long long size = static_cast<long long>(a.P) * a.N;
-  const long long i = static_cast<long long>(blockIdx.x) * 256 + threadIdx.x;
+  const long long i = (static_cast<long long>(blockIdx.x) * 256 + threadIdx.x) * V;
   if (i >= size) return;
   float* st = a.state + (static_cast<long long>(a.slots[seq]) * a.heads + h) * size + i;
-  float s = a.ctx[seq] > 0 ? *st : 0.f;
-  const int c1 = first_chunk[seq + 1];
-  int c = first_chunk[seq];
-  constexpr int U = 8;
-  for (; c + U <= c1; c += U) {  // loads of several chunks in flight
-    float v[U], d[U];
+  float s[V];
+  const bool cont = a.ctx[seq] > 0;
+  auto load = [](const float* p, float (&v)[V]) {
+    if constexpr (V == 4) {
+      const float4 t = *reinterpret_cast<const float4*>(p);
+      v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+    } else {
+      v[0] = p[0];
+    }
+  };
+#pragma unroll
+  for (int k = 0; k < V; ++k) s[k] = 0.f;
+  if (cont) load(st, s);
+  const int c0 = first_chunk[seq], c1 = first_chunk[seq + 1];
+  constexpr int U = 8;  // loads of several chunks in flight
+  for (int c = c0; c < c1; c += U) {
+    float v[U][V], d[U];
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-      v[u] = work[(static_cast<long long>(c + u) * a.heads + h) * size + i];
+      if (c + u >= c1) break;
+      load(work + (static_cast<long long>(c + u) * a.heads + h) * size + i, v[u]);
       d[u] = decay[static_cast<long long>(c + u) * a.heads + h];
     }
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-      work[(static_cast<long long>(c + u) * a.heads + h) * size + i] = s;
-      s = d[u] * s + v[u];
+      if (c + u >= c1) break;
+      bf16* dst = before + (static_cast<long long>(c + u) * a.heads + h) * 2 * size + i;
+      if constexpr (V == 4) {
+        uint32_t hi[2], lo[2];
+        split2(s[0], s[1], hi[0], lo[0]);
+        split2(s[2], s[3], hi[1], lo[1]);
+        *reinterpret_cast<uint2*>(dst) = make_uint2(hi[0], hi[1]);
+        *reinterpret_cast<uint2*>(dst + size) = make_uint2(lo[0], lo[1]);
+      } else {
+        dst[0] = __float2bfloat16(s[0]);
+        dst[size] = __float2bfloat16(s[0] - to_f(dst[0]));
+      }
+#pragma unroll
+      for (int k = 0; k < V; ++k) s[k] = d[u] * s[k] + v[u][k];
     }
   }
-  for (; c < c1; ++c) {
-    float* w = work + (static_cast<long long>(c) * a.heads + h) * size + i;
-    const float v = *w;
-    *w = s;
-    s = decay[static_cast<long long>(c) * a.heads + h] * s + v;
-  }
-  *st = s;
+  if constexpr (V == 4)
+    *reinterpret_cast<float4*>(st) = make_float4(s[0], s[1], s[2], s[3]);
+  else
+    *st = s[0];
 }
 
 // (3) y[t] = exp(acum_t) C_t S_before + sum_{s <= t} (C_t . B_s) exp(acum_t - acum_s) dt_s x_s + D x_t
-template <int PT>  // 16-wide tiles of P
-__global__ void __launch_bounds__(CW * 32) chunk_out_kernel(const HyMamba a, const bf16* __restrict__ xbc,
-                                                            const int4* __restrict__ chunks, const float* __restrict__ work,
-                                                            bf16* __restrict__ y, bool vec) {
+//
+// A CTA takes several heads of a group: the products C B^T of the chunk are the same for all of them and stay in registers. The
+// lower triangle has 36 blocks of 16 x 16 tokens; four warps take the row tiles (w, 7 - w), nine blocks each, and two such sets
+// split the columns p.
+template <int PH>  // 16-wide tiles of P per half
+__global__ void __launch_bounds__(CW * 32, PH <= 2 ? 2 : 1)
+chunk_out_kernel(const HyMamba a, const bf16* __restrict__ xbc, const int4* __restrict__ chunks, int hb,
+                 const bf16* __restrict__ before, bf16* __restrict__ y, bool vec) {
   extern __shared__ __align__(16) unsigned char raw[];
   const int4 ck = chunks[blockIdx.x];
-  const int h = blockIdx.y, seq = ck.x, row0 = ck.y, n = ck.z;
-  const int P = a.P, N = a.N, NP = (N + 15) / 16 * 16;
-  const int inner = a.heads * P, ch = inner + 2 * a.groups * N, g = h / (a.heads / a.groups);
-  constexpr int PP = PT * 16;
+  const int seq = ck.x, row0 = ck.y, n = ck.z;
+  const int P = a.P, N = a.N, NP = (N + 15) / 16 * 16, hpg = a.heads / a.groups;
+  const int inner = a.heads * P, ch = inner + 2 * a.groups * N;
+  const int per_group = (hpg + hb - 1) / hb, g = blockIdx.y / per_group;
+  const int h0 = g * hpg + (blockIdx.y - g * per_group) * hb, nh = min(hb, (g + 1) * hpg - h0);
+  constexpr int PP = PH * 32;
   constexpr int ldx = PP + LDX_PAD;
   const int ldn = NP + LDX_PAD;
   bf16* Cs = reinterpret_cast<bf16*>(raw);  // [Q][ldn]
-  bf16* Bs = Cs + Q * ldn;                  // [Q][ldn]
-  bf16* xs = Bs + Q * ldn;                  // [Q][ldx]
-  bf16* Sh = xs + Q * ldx;                  // [PP][ldn] carried state, high part
-  bf16* Sl = Sh + PP * ldn;                 // low part
-  float* dts = reinterpret_cast<float*>(Sl + PP * ldn);
-  float* acum = dts + Q;
+  bf16* xs = Cs + Q * ldn;                  // [Q][ldx]
+  bf16* Bs = xs + Q * ldx;                  // [Q][ldn], later the carried state: [2][PP][ldn]
+  bf16* Ss = Bs;
+  float* dts = reinterpret_cast<float*>(Bs + (Q > 2 * PP ? Q : 2 * PP) * ldn);  // [MAX_HB][Q]
+  float* acum = dts + MAX_HB * Q;
   const bool carried = ck.w > 0 || a.ctx[seq] > 0;
-  load_tile(xbc, ch, row0, n, inner + a.groups * N + g * N, N, NP, Cs, ldn, vec);
-  load_tile(xbc, ch, row0, n, inner + g * N, N, NP, Bs, ldn, vec);
-  load_tile(xbc, ch, row0, n, h * P, P, PP, xs, ldx, vec);
-  if (carried) {
-    const float* src = work + (static_cast<long long>(blockIdx.x) * a.heads + h) * P * N;
-    for (int i = threadIdx.x; i < PP * (NP / 2); i += CW * 32) {
-      const int p = i / (NP / 2), c = (i - p * (NP / 2)) * 2;
-      float u = 0.f, v = 0.f;
-      if (p < P) {
-        if (c < N) u = src[static_cast<long long>(p) * N + c];
-        if (c + 1 < N) v = src[static_cast<long long>(p) * N + c + 1];
-      }
-      uint32_t hi, lo;
-      split2(u, v, hi, lo);
-      *reinterpret_cast<uint32_t*>(Sh + p * ldn + c) = hi;
-      *reinterpret_cast<uint32_t*>(Sl + p * ldn + c) = lo;
-    }
-  }
-  chunk_decay(a, h, row0, n, dts, acum);  // ends with a block barrier
+  const bf16* rows = xbc + static_cast<long long>(row0) * ch;
+  load_tile(rows + inner + a.groups * N + g * N, ch, n, N, Q, NP, Cs, ldn, vec);
+  load_tile(rows + inner + g * N, ch, n, N, Q, NP, Bs, ldn, vec);
+  chunk_decays(a, h0, nh, row0, n, dts, acum);
+  cp_wait_all();
+  __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t0 = warp * 16;
-  if (t0 >= n) return;
-  const int r0 = t0 + (lane >> 2);  // this lane's rows: r0 and r0 + 8
-  float o[2 * PT][4];
+  const int half = warp >> 2, ta = warp & 3, tb = 7 - ta;   // this warp's row tiles
+  const int a_row = lane & 15, a_col = (lane >> 4) << 3;
+  const int b_row = (lane & 7) + ((lane >> 4) << 3), b_col = ((lane >> 3) & 1) << 3;    // [n][k] operands
+  const int v_row = (lane & 7) + (((lane >> 3) & 1) << 3), v_col = (lane >> 4) << 3;    // [k][n] operands
+  float gm[9][2][4];
 #pragma unroll
-  for (int j = 0; j < 2 * PT; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-  const int a_row = t0 + (lane & 15), a_col = (lane >> 4) << 3;
-  if (carried) {
-    for (int k0 = 0; k0 < NP; k0 += 16) {
-      uint32_t cf[4];
-      ldsm4(s_u32(Cs + a_row * ldn + k0 + a_col), cf);
+  for (int i = 0; i < 9; ++i) {
+    const int tile = i <= ta ? ta : tb, s = i <= ta ? i : i - ta - 1;
 #pragma unroll
-      for (int jp = 0; jp < PT; ++jp) {
-        uint32_t b[4];
-        const int br = jp * 16 + (lane & 7) + ((lane >> 4) << 3), bc = k0 + (((lane >> 3) & 1) << 3);
-        ldsm4(s_u32(Sh + br * ldn + bc), b);
-        mma(o[2 * jp], cf, b[0], b[1]);
-        mma(o[2 * jp + 1], cf, b[2], b[3]);
-        ldsm4(s_u32(Sl + br * ldn + bc), b);
-        mma(o[2 * jp], cf, b[0], b[1]);
-        mma(o[2 * jp + 1], cf, b[2], b[3]);
-      }
-    }
-    const float e0 = expf(acum[r0]), e1 = expf(acum[r0 + 8]);
-#pragma unroll
-    for (int j = 0; j < 2 * PT; ++j) {
-      o[j][0] *= e0; o[j][1] *= e0;
-      o[j][2] *= e1; o[j][3] *= e1;
-    }
-  }
-  const float ac0 = acum[r0], ac1 = acum[r0 + 8];
-  for (int s0 = 0; s0 <= t0; s0 += 16) {  // blocks of 16 earlier tokens
-    float sc[2][4];
-    sc[0][0] = sc[0][1] = sc[0][2] = sc[0][3] = 0.f;
-    sc[1][0] = sc[1][1] = sc[1][2] = sc[1][3] = 0.f;
+    for (int e = 0; e < 4; ++e) gm[i][0][e] = gm[i][1][e] = 0.f;
+    const uint32_t ca = s_u32(Cs + (tile * 16 + a_row) * ldn + a_col), ba = s_u32(Bs + (s * 16 + b_row) * ldn + b_col);
+#pragma unroll 2
     for (int k0 = 0; k0 < NP; k0 += 16) {
       uint32_t cf[4], b[4];
-      ldsm4(s_u32(Cs + a_row * ldn + k0 + a_col), cf);
-      ldsm4(s_u32(Bs + (s0 + (lane & 7) + ((lane >> 4) << 3)) * ldn + k0 + (((lane >> 3) & 1) << 3)), b);
-      mma(sc[0], cf, b[0], b[1]);
-      mma(sc[1], cf, b[2], b[3]);
-    }
-    // scores -> decay-weighted coefficients, split in two bf16 terms; accumulator layout = A-operand layout
-    uint32_t wh[4], wl[4];
-#pragma unroll
-    for (int nt = 0; nt < 2; ++nt) {
-      float w[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int s = s0 + nt * 8 + (lane & 3) * 2 + (e & 1), t = r0 + (e >> 1) * 8;
-        w[e] = s <= t ? sc[nt][e] * expf((e >> 1 ? ac1 : ac0) - acum[s]) * dts[s] : 0.f;
-      }
-      split2(w[0], w[1], wh[nt * 2], wl[nt * 2]);
-      split2(w[2], w[3], wh[nt * 2 + 1], wl[nt * 2 + 1]);
-    }
-#pragma unroll
-    for (int jp = 0; jp < PT; ++jp) {
-      uint32_t b[4];
-      ldsm4t(s_u32(xs + (s0 + (lane & 7) + (((lane >> 3) & 1) << 3)) * ldx + jp * 16 + ((lane >> 4) << 3)), b);
-      mma(o[2 * jp], wh, b[0], b[1]);
-      mma(o[2 * jp], wl, b[0], b[1]);
-      mma(o[2 * jp + 1], wh, b[2], b[3]);
-      mma(o[2 * jp + 1], wl, b[2], b[3]);
+      ldsm4(ca + k0 * 2, cf);
+      ldsm4(ba + k0 * 2, b);
+      mma(gm[i][0], cf, b[0], b[1]);
+      mma(gm[i][1], cf, b[2], b[3]);
     }
   }
-  const float D = to_f(static_cast<const bf16*>(a.D)[h]);
+  const int pc0 = half * PH * 16;  // first column of this warp
+  for (int hi = 0; hi < nh; ++hi) {
+    const int h = h0 + hi;
+    __syncthreads();  // B, or the previous head's tiles, have been read
+    load_tile(rows + h * P, ch, n, P, Q, PP, xs, ldx, vec);
+    if (carried) {
+      const bf16* src = before + (static_cast<long long>(blockIdx.x) * a.heads + h) * 2 * P * N;
+      load_tile(src, N, P, N, PP, NP, Ss, ldn, vec);
+      load_tile(src + static_cast<long long>(P) * N, N, P, N, PP, NP, Ss + PP * ldn, ldn, vec);
+    }
+    cp_wait_all();
+    __syncthreads();
+    const float* ac = acum + hi * Q;
+    const float* dt = dts + hi * Q;
+    const float D = to_f(static_cast<const bf16*>(a.D)[h]);
+    float o[2 * PH][4];
 #pragma unroll
-  for (int j = 0; j < 2 * PT; ++j) {
-    const int p = j * 8 + (lane & 3) * 2;
+    for (int i = 0; i < 9; ++i) {
+      const int tile = i <= ta ? ta : tb, s0 = (i <= ta ? i : i - ta - 1) * 16;
+      const int r0 = tile * 16 + (lane >> 2);
+      const float ac0 = ac[r0], ac1 = ac[r0 + 8];
+      if (i == 0 || i == ta + 1) {  // a row tile begins: what the carried state gives
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int t = r0 + e * 8;
-      if (t >= n) continue;
-      bf16* dst = y + static_cast<long long>(row0 + t) * inner + h * P + p;
-      const float u = o[j][2 * e] + D * to_f(xs[t * ldx + p]), v = o[j][2 * e + 1] + D * to_f(xs[t * ldx + p + 1]);
-      if (p + 1 < P && (P & 1) == 0) {
-        *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(u, v);
-      } else {
-        if (p < P) dst[0] = __float2bfloat16(u);
-        if (p + 1 < P) dst[1] = __float2bfloat16(v);
+        for (int j = 0; j < 2 * PH; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+        if (carried) {
+          const uint32_t ca = s_u32(Cs + (tile * 16 + a_row) * ldn + a_col), sa = s_u32(Ss + (pc0 + b_row) * ldn + b_col);
+#pragma unroll 1
+          for (int k0 = 0; k0 < NP; k0 += 16) {
+            uint32_t cf[4];
+            ldsm4(ca + k0 * 2, cf);
+#pragma unroll
+            for (int jp = 0; jp < PH; ++jp) {
+              uint32_t b[4];
+              ldsm4(sa + (jp * 16 * ldn + k0) * 2, b);
+              mma(o[2 * jp], cf, b[0], b[1]);
+              mma(o[2 * jp + 1], cf, b[2], b[3]);
+              ldsm4(sa + ((PP + jp * 16) * ldn + k0) * 2, b);
+              mma(o[2 * jp], cf, b[0], b[1]);
+              mma(o[2 * jp + 1], cf, b[2], b[3]);
+            }
+          }
+          const float e0 = ex2(ac0), e1 = ex2(ac1);
+#pragma unroll
+          for (int j = 0; j < 2 * PH; ++j) {
+            o[j][0] *= e0; o[j][1] *= e0;
+            o[j][2] *= e1; o[j][3] *= e1;
+          }
+        }
+      }
+      // scores -> decay-weighted coefficients, split in two bf16 terms; accumulator layout = A-operand layout
+      uint32_t wh[4], wl[4];
+#pragma unroll
+      for (int nt = 0; nt < 2; ++nt) {
+        const int s = s0 + nt * 8 + (lane & 3) * 2;
+        const float2 as = *reinterpret_cast<const float2*>(ac + s), ds = *reinterpret_cast<const float2*>(dt + s);
+        float w[4];
+        w[0] = s <= r0 ? gm[i][nt][0] * ex2(ac0 - as.x) * ds.x : 0.f;
+        w[1] = s + 1 <= r0 ? gm[i][nt][1] * ex2(ac0 - as.y) * ds.y : 0.f;
+        w[2] = s <= r0 + 8 ? gm[i][nt][2] * ex2(ac1 - as.x) * ds.x : 0.f;
+        w[3] = s + 1 <= r0 + 8 ? gm[i][nt][3] * ex2(ac1 - as.y) * ds.y : 0.f;
+        split2(w[0], w[1], wh[nt * 2], wl[nt * 2]);
+        split2(w[2], w[3], wh[nt * 2 + 1], wl[nt * 2 + 1]);
+      }
+      const uint32_t xa = s_u32(xs + (s0 + v_row) * ldx + pc0 + v_col);
+#pragma unroll
+      for (int jp = 0; jp < PH; ++jp) {
+        uint32_t b[4];
+        ldsm4t(xa + jp * 32, b);
+        mma(o[2 * jp], wh, b[0], b[1]);
+        mma(o[2 * jp], wl, b[0], b[1]);
+        mma(o[2 * jp + 1], wh, b[2], b[3]);
+        mma(o[2 * jp + 1], wl, b[2], b[3]);
+      }
+      if (i == ta || i == 8) {  // the row tile is complete
+#pragma unroll
+        for (int j = 0; j < 2 * PH; ++j) {
+          const int p = pc0 + j * 8 + (lane & 3) * 2;
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int t = r0 + e * 8;
+            if (t >= n) continue;
+            bf16* dst = y + static_cast<long long>(row0 + t) * inner + h * P + p;
+            const float u = o[j][2 * e] + D * to_f(xs[t * ldx + p]), v = o[j][2 * e + 1] + D * to_f(xs[t * ldx + p + 1]);
+            if ((P & 1) == 0) {
+              if (p < P) *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(u, v);
+            } else {
+              if (p < P) dst[0] = __float2bfloat16(u);
+              if (p + 1 < P) dst[1] = __float2bfloat16(v);
+            }
+          }
+        }
       }
     }
   }
@@ -563,8 +693,9 @@ int conv_t(const HyMamba& a, const int* tiles, int n_tiles, void* xbc, cudaStrea
   T* out = static_cast<T*>(xbc);
   bool done = false;
   if constexpr (sizeof(T) == 2) {
-    if (a.taps == 4 && (a.heads * a.P) % 2 == 0 && ch % 2 == 0 && a.ld % 2 == 0) {
-      conv4_pair_kernel<<<dim3(n_tiles, (ch + 255) / 256), 128, 0, s>>>(a, tl, out);
+    if (a.taps == 4 && (a.heads * a.P) % 8 == 0 && ch % 8 == 0 && aligned16<T>(a.proj, a.ld) && aligned16<T>(a.ring, ch) &&
+        aligned16<T>(a.conv_w, 8) && aligned16<T>(a.conv_b, 8)) {
+      conv4_vec_kernel<<<dim3(n_tiles, (ch / 8 + 127) / 128), 128, 0, s>>>(a, tl, out);
       done = true;
     }
   }
@@ -605,26 +736,44 @@ int step_t(const HyMamba& a, const int* positions, int B, void* y, cudaStream_t 
   return static_cast<int>(cudaGetLastError());
 }
 
-size_t state_smem(int P, int N) {
-  const int PP = (P + 15) / 16 * 16, NP = (N + 63) / 64 * 64;
-  return static_cast<size_t>(2) * (2 * Q * (PP + LDX_PAD) + Q * (NP + LDX_PAD)) + 2 * Q * sizeof(float);
+size_t state_smem(int PT, int N) {
+  const int NP = (N + 63) / 64 * 64;
+  return static_cast<size_t>(2) * (2 * Q * (PT * 16 + LDX_PAD) + Q * (NP + LDX_PAD)) + 2 * MAX_HB * Q * sizeof(float);
 }
-size_t out_smem(int PP, int N) {
-  const int NP = (N + 15) / 16 * 16;
-  return static_cast<size_t>(2) * (2 * Q * (NP + LDX_PAD) + Q * (PP + LDX_PAD) + 2 * PP * (NP + LDX_PAD)) + 2 * Q * sizeof(float);
+size_t out_smem(int PH, int N) {
+  const int NP = (N + 15) / 16 * 16, PP = PH * 32;
+  return static_cast<size_t>(2) * (Q * (NP + LDX_PAD) + Q * (PP + LDX_PAD) + (Q > 2 * PP ? Q : 2 * PP) * (NP + LDX_PAD)) +
+         2 * MAX_HB * Q * sizeof(float);
 }
-int out_tiles(int P) {
-  const int t = (P + 15) / 16;
-  return t <= 2 ? 2 : (t <= 3 ? 3 : (t <= 4 ? 4 : (t <= 6 ? 6 : 8)));
+int half_tiles(int P) { return (P + 31) / 32; }
+
+// heads per CTA: as many as leave the device a few waves of CTAs
+int heads_per_cta(int n_chunks, int heads, int groups) {
+  const int hpg = heads / groups;
+  int hb = hpg < MAX_HB ? hpg : MAX_HB;
+  while (hb > 1 && static_cast<long long>(n_chunks) * groups * ((hpg + hb - 1) / hb) < 3 * 2 * 148) hb = (hb + 1) / 2;
+  return hb;
 }
 
 template <int PT>
-int launch_out(const HyMamba& a, const bf16* xbc, const int4* ck, int n_chunks, const float* work, bf16* y, bool vec, cudaStream_t s) {
-  const size_t smem = out_smem(PT * 16, a.N);
-  auto kern = chunk_out_kernel<PT>;
+int launch_state(const HyMamba& a, const bf16* xbc, const int4* ck, int n_chunks, int hb, float* work, float* decay, bool vec, cudaStream_t s) {
+  const size_t smem = state_smem(PT, a.N);
+  auto kern = chunk_state_kernel<PT>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
-  kern<<<dim3(n_chunks, a.heads), CW * 32, smem, s>>>(a, xbc, ck, work, y, vec);
+  const int hpg = a.heads / a.groups;
+  kern<<<dim3(n_chunks, a.groups * ((hpg + hb - 1) / hb)), CW * 32, smem, s>>>(a, xbc, ck, hb, work, decay, vec);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <int PH>
+int launch_out(const HyMamba& a, const bf16* xbc, const int4* ck, int n_chunks, int hb, const bf16* before, bf16* y, bool vec, cudaStream_t s) {
+  const size_t smem = out_smem(PH, a.N);
+  auto kern = chunk_out_kernel<PH>;
+  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+  if (e != cudaSuccess) return static_cast<int>(e);
+  const int hpg = a.heads / a.groups;
+  kern<<<dim3(n_chunks, a.groups * ((hpg + hb - 1) / hb)), CW * 32, smem, s>>>(a, xbc, ck, hb, before, y, vec);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -642,30 +791,38 @@ int hy_mamba_step(bool f32, const HyMamba& a, const int* positions, int B, void*
 
 bool hy_chunk_scan_supported(int P, int N, int, int) {
   if (P < 1 || P > 128 || N < 1 || N > 256) return false;
-  return state_smem(P, N) <= 227 * 1024 && out_smem(out_tiles(P) * 16, N) <= 227 * 1024;
+  const int ph = half_tiles(P);
+  return state_smem(2 * ph, N) <= 227 * 1024 && out_smem(ph, N) <= 227 * 1024;
 }
 
 int hy_chunk_scan(const HyMamba& a, const void* xbc_, const int* chunks, int n_chunks, const int* first_chunk, float* work,
-                  float* decay, void* y_, cudaStream_t s) {
+                  float* decay, void* before_, void* y_, cudaStream_t s) {
   if (!hy_chunk_scan_supported(a.P, a.N, a.heads, a.groups)) return static_cast<int>(cudaErrorInvalidValue);
   const bf16* xbc = static_cast<const bf16*>(xbc_);
-  bf16* y = static_cast<bf16*>(y_);
+  bf16 *y = static_cast<bf16*>(y_), *before = static_cast<bf16*>(before_);
   const int4* ck = reinterpret_cast<const int4*>(chunks);
   const bool vec = a.P % 8 == 0 && a.N % 8 == 0 && (reinterpret_cast<uintptr_t>(xbc) & 15) == 0;
-  const size_t sm1 = state_smem(a.P, a.N);
-  cudaError_t e = cudaFuncSetAttribute(chunk_state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(sm1));
-  if (e != cudaSuccess) return static_cast<int>(e);
-  chunk_state_kernel<<<dim3(n_chunks, a.heads), CW * 32, sm1, s>>>(a, xbc, ck, work, decay, vec);
+  const int ph = half_tiles(a.P), hb = heads_per_cta(n_chunks, a.heads, a.groups);
+  int rc = 0;
+  switch (ph) {
+    case 1: rc = launch_state<2>(a, xbc, ck, n_chunks, hb, work, decay, vec, s); break;
+    case 2: rc = launch_state<4>(a, xbc, ck, n_chunks, hb, work, decay, vec, s); break;
+    case 3: rc = launch_state<6>(a, xbc, ck, n_chunks, hb, work, decay, vec, s); break;
+    default: rc = launch_state<8>(a, xbc, ck, n_chunks, hb, work, decay, vec, s); break;
+  }
+  if (rc != 0) return rc;
   const long long size = static_cast<long long>(a.P) * a.N;
-  chunk_pass_kernel<<<dim3(static_cast<unsigned>((size + 255) / 256), a.heads, a.nseq), 256, 0, s>>>(a, first_chunk, decay, work);
-  e = cudaGetLastError();
+  if (size % 4 == 0)
+    chunk_pass_kernel<4><<<dim3(static_cast<unsigned>((size / 4 + 255) / 256), a.heads, a.nseq), 256, 0, s>>>(a, first_chunk, decay, work, before);
+  else
+    chunk_pass_kernel<1><<<dim3(static_cast<unsigned>((size + 255) / 256), a.heads, a.nseq), 256, 0, s>>>(a, first_chunk, decay, work, before);
+  const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return static_cast<int>(e);
-  switch (out_tiles(a.P)) {
-    case 2: return launch_out<2>(a, xbc, ck, n_chunks, work, y, vec, s);
-    case 3: return launch_out<3>(a, xbc, ck, n_chunks, work, y, vec, s);
-    case 4: return launch_out<4>(a, xbc, ck, n_chunks, work, y, vec, s);
-    case 6: return launch_out<6>(a, xbc, ck, n_chunks, work, y, vec, s);
-    default: return launch_out<8>(a, xbc, ck, n_chunks, work, y, vec, s);
+  switch (ph) {
+    case 1: return launch_out<1>(a, xbc, ck, n_chunks, hb, before, y, vec, s);
+    case 2: return launch_out<2>(a, xbc, ck, n_chunks, hb, before, y, vec, s);
+    case 3: return launch_out<3>(a, xbc, ck, n_chunks, hb, before, y, vec, s);
+    default: return launch_out<4>(a, xbc, ck, n_chunks, hb, before, y, vec, s);
   }
 }
 

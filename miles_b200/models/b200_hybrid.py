@@ -60,7 +60,7 @@ class B200Hybrid(TorchHybrid):
             return F.linear(x, w).to(out_dtype)
         out = torch.empty(T, N, dtype=out_dtype, device=x.device)
         self.launches += 1
-        if T <= SMALL_T and N % 16 == 0 and K % 32 == 0 and N * K * 2 < (48 << 20) and x.is_contiguous():
+        if T <= SMALL_T and N % 16 == 0 and K % 32 == 0 and (T <= 8 or N * K * 2 < (48 << 20)) and x.is_contiguous():
             self.C.small_gemv(x, None, 0.0, w, None, out, self.status)
         else:
             self.C.gemm(x, w, out, False, False, False, 0, self.status)

@@ -192,7 +192,7 @@ def latent_case(m, lens, news, seed, dtype, page=8, peak=4.0):
         rows[torch.tensor(own)[at // page] * page + at % page] = torch.cat([c, kr, torch.zeros(n, width - R - r)], 1)
         qq = q(torch.randn(k, H, d + r, generator=g) * peak)   # sharp: single keys stand out
         for off, h in ((m["mask"]["size"], 0), (m["mask"]["size"] - 1, H - 1)):  # just outside and just inside the last query's window:
-            if 0 <= n - 1 - off < n:                                             # keys that would take all of one head's weight
+            if 0 <= n - 1 - off < n and (H > 1 or off == m["mask"]["size"]):                                             # keys that would take all of one head's weight
                 v = ukv[h * d:(h + 1) * d].T @ qq[-1, h, :d]
                 c[n - 1 - off] = q(3 * v / v.norm() * R ** 0.5)
         own_rows = torch.tensor(own)[at // page] * page + at % page
