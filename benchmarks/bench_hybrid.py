@@ -192,7 +192,7 @@ def run(sizes: list, steps: int, warmup: int, kernels: bool, prompts: list, batc
     pk = peaks()
     for size in sizes:
         for kind in ("rokivik", "qwen3"):
-            cfg, model, eng = build(kind, size, max(batches), max(ctx + 1024, max(prompts)), max(16384, max(prompts)))
+            cfg, model, eng = build(kind, size, max(max(batches), 8192 // min(prompts) + 1), max(ctx + 1024, max(prompts)), max(16384, max(prompts)))
             name = cfg.name if kind == "rokivik" else f"{SIZES[size]['like']} layers x 6"
             base = {"model": name, "params_m": round(cfg.num_params() / 1e6), "layers": cfg.num_layers, "dtype": "bf16", "data": "random tokens and weights",
                     "l2": "weights larger than L2"}

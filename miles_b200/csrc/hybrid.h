@@ -57,8 +57,9 @@ struct HySide {
   int* status;
 };
 int hy_side_fused(bool f32, const HySide& a, int T, cudaStream_t s);
-// The same in pieces around tensor-core products, for many rows: cast x, then g from the gate product, then the rest.
-int hy_cast_rows(const float* x, void* out_bf16, long long n, cudaStream_t s);
+// The same in pieces around tensor-core products, for many rows: x += delta (may be null) and its bf16 copy, then g from the gate
+// product, then the rest.
+int hy_cast_rows(float* x, const float* delta, void* out_bf16, long long n, cudaStream_t s);
 int hy_side_gate(bool f32, const float* z, const HySide& a, void* g, int T, cudaStream_t s);
 int hy_side_finish(bool f32, const float* y, const HySide& a, int T, cudaStream_t s);
 

@@ -133,11 +133,12 @@ void side_finish(SIDE_ARGS, const at::Tensor& y) {
   const c10::cuda::CUDAGuard guard(x.device());
   RUN(mb::hy_side_finish(is_f32(gate), y.data_ptr<float>(), a, x.size(0), cur_stream()));
 }
-void cast_rows(const at::Tensor& x, at::Tensor& out) {
+void cast_rows(at::Tensor& x, const OptT& delta, at::Tensor& out) {
   CHECK_F32(x); CHECK_BF16(out);
   TORCH_CHECK(x.numel() == out.numel(), "cast_rows: shapes");
+  if (delta.has_value()) { CHECK_F32((*delta)); TORCH_CHECK(delta->numel() == x.numel(), "cast_rows: delta"); }
   const c10::cuda::CUDAGuard guard(x.device());
-  RUN(mb::hy_cast_rows(x.data_ptr<float>(), out.data_ptr(), x.numel(), cur_stream()));
+  RUN(mb::hy_cast_rows(x.data_ptr<float>(), opt_ptr<float>(delta), out.data_ptr(), x.numel(), cur_stream()));
 }
 
 // ------------------------------------------------------------------------------------------------ Mamba-2

@@ -350,14 +350,25 @@ __global__ void __launch_bounds__(STHREADS) side_fused_kernel(const HySide a, in
   }
 }
 
-__global__ void __launch_bounds__(256) cast_rows_kernel(const float* __restrict__ x, bf16* __restrict__ o, long long n) {
+__global__ void __launch_bounds__(256) cast_rows_kernel(float* __restrict__ x, const float* __restrict__ delta, bf16* __restrict__ o,
+                                                        long long n) {
   const long long i = (static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x) * 8;
   if (i + 8 <= n) {
-    const float4 a = *reinterpret_cast<const float4*>(x + i), b = *reinterpret_cast<const float4*>(x + i + 4);
+    float4 a = *reinterpret_cast<const float4*>(x + i), b = *reinterpret_cast<const float4*>(x + i + 4);
+    if (delta) {
+      const float4 u = *reinterpret_cast<const float4*>(delta + i), v = *reinterpret_cast<const float4*>(delta + i + 4);
+      a.x += u.x; a.y += u.y; a.z += u.z; a.w += u.w;
+      b.x += v.x; b.y += v.y; b.z += v.z; b.w += v.w;
+      *reinterpret_cast<float4*>(x + i) = a;
+      *reinterpret_cast<float4*>(x + i + 4) = b;
+    }
     const float v[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
     Vec<bf16>::store(o + i, v);
   } else {
-    for (long long k = i; k < n; ++k) o[k] = __float2bfloat16(x[k]);
+    for (long long k = i; k < n; ++k) {
+      if (delta) x[k] += delta[k];
+      o[k] = __float2bfloat16(x[k]);
+    }
   }
 }
 
@@ -520,9 +531,9 @@ int hy_side_fused(bool f32, const HySide& a, int T, cudaStream_t s) {
   return four ? launch_side<bf16, 4>(a, T, s) : launch_side<bf16, 1>(a, T, s);
 }
 
-int hy_cast_rows(const float* x, void* out, long long n, cudaStream_t s) {
+int hy_cast_rows(float* x, const float* delta, void* out, long long n, cudaStream_t s) {
   const long long blocks = (n + 2047) / 2048;
-  cast_rows_kernel<<<static_cast<unsigned>(blocks), 256, 0, s>>>(x, static_cast<bf16*>(out), n);
+  cast_rows_kernel<<<static_cast<unsigned>(blocks), 256, 0, s>>>(x, delta, static_cast<bf16*>(out), n);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -32,6 +32,15 @@ struct Decay {
   __device__ __forceinline__ float operator()(float s) const { return fmaf(c, s, k * s); }
 };
 
+// State row of a sequence; one outside the cache is reported and not followed (-1: the sequence starts from nothing and its state
+// is not kept).
+__device__ __forceinline__ long long state_row(const HyMamba& a, int seq) {
+  const int slot = a.slots[seq];
+  if (slot >= 0 && slot < a.sequences) return slot;
+  if (a.status) atomicCAS(a.status, 0, 11);
+  return -1;
+}
+
 // ------------------------------------------------------------------------------------------------ convolution (prefill)
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) conv_kernel(const HyMamba a, const int4* __restrict__ tiles, T* __restrict__ xbc) {
@@ -42,9 +51,9 @@ __global__ void __launch_bounds__(128) conv_kernel(const HyMamba a, const int4* 
   const int taps = TAPS > 0 ? TAPS : a.taps;
   const int seq = tl.x, row0 = tl.y, n = tl.z;
   const int first = a.cu[seq], ctx = a.ctx[seq];
-  const long long slot = a.slots[seq];
+  const long long slot = state_row(a, seq);
   const T* in = static_cast<const T*>(a.proj) + inner + c;
-  const T* ring = static_cast<const T*>(a.ring) + slot * taps * ch + c;
+  const T* ring = static_cast<const T*>(a.ring) + (slot < 0 ? 0 : slot) * taps * ch + c;
   const T* w = static_cast<const T*>(a.conv_w) + static_cast<long long>(c) * taps;
   const float bias = to_f(static_cast<const T*>(a.conv_b)[c]);
   // input of the token `back` rows before row r
@@ -52,7 +61,7 @@ __global__ void __launch_bounds__(128) conv_kernel(const HyMamba a, const int4* 
     const int q = r - back;
     if (q >= first) return to_f(in[static_cast<long long>(q) * a.ld]);
     const int p = ctx + q - first;
-    return p < 0 ? 0.f : to_f(ring[static_cast<long long>(p % taps) * ch]);
+    return p < 0 || slot < 0 ? 0.f : to_f(ring[static_cast<long long>(p % taps) * ch]);
   };
   if constexpr (TAPS > 0) {
     float wv[TAPS], hist[TAPS];
@@ -88,7 +97,8 @@ __global__ void __launch_bounds__(128) conv4_vec_kernel(const HyMamba a, const i
   const int seq = tl.x, row0 = tl.y, n = tl.z;
   const int first = a.cu[seq], ctx = a.ctx[seq];
   const bf16* in = static_cast<const bf16*>(a.proj) + inner + c;
-  const bf16* ring = static_cast<const bf16*>(a.ring) + static_cast<long long>(a.slots[seq]) * 4 * ch + c;
+  const long long slot = state_row(a, seq);
+  const bf16* ring = static_cast<const bf16*>(a.ring) + (slot < 0 ? 0 : slot) * 4 * ch + c;
   float w[4][8], bias[8], h[3][8];
   {
     const bf16* wp = static_cast<const bf16*>(a.conv_w) + static_cast<long long>(c) * 4;  // [channel][tap]
@@ -106,7 +116,7 @@ __global__ void __launch_bounds__(128) conv4_vec_kernel(const HyMamba a, const i
     const int q = row0 - 3 + k, p = ctx + q - first;
     if (q >= first)
       Vec<bf16>::load(in + static_cast<long long>(q) * a.ld, h[k]);
-    else if (p >= 0)
+    else if (p >= 0 && slot >= 0)
       Vec<bf16>::load(ring + static_cast<long long>(p & 3) * ch, h[k]);
     else
 #pragma unroll
@@ -146,7 +156,9 @@ __global__ void __launch_bounds__(256) ring_kernel(const HyMamba a) {
   if (c >= ch) return;
   const int first = a.cu[seq], n = a.cu[seq + 1] - first, ctx = a.ctx[seq];
   const T* in = static_cast<const T*>(a.proj) + inner + c;
-  T* ring = static_cast<T*>(a.ring) + static_cast<long long>(a.slots[seq]) * a.taps * ch + c;
+  const long long slot = state_row(a, seq);
+  if (slot < 0) return;
+  T* ring = static_cast<T*>(a.ring) + slot * a.taps * ch + c;
   for (int q = max(0, n - a.taps); q < n; ++q)
     ring[static_cast<long long>((ctx + q) % a.taps) * ch] = in[static_cast<long long>(first + q) * a.ld];
 }
@@ -160,10 +172,11 @@ __global__ void __launch_bounds__(256) scan_kernel(const HyMamba a, const T* __r
   if (p >= a.P) return;
   const int inner = a.heads * a.P, ch = inner + 2 * a.groups * a.N, g = h / (a.heads / a.groups);
   const int first = a.cu[seq], n = a.cu[seq + 1] - first;
-  float* st = a.state + ((static_cast<long long>(a.slots[seq]) * a.heads + h) * a.P + p) * a.N;
+  const long long slot = state_row(a, seq);
+  float* st = a.state + (((slot < 0 ? 0 : slot) * a.heads + h) * a.P + p) * a.N;
   float S[NR];
 #pragma unroll
-  for (int i = 0; i < NR; ++i) S[i] = (a.ctx[seq] > 0 && lane + 32 * i < a.N) ? st[lane + 32 * i] : 0.f;
+  for (int i = 0; i < NR; ++i) S[i] = (slot >= 0 && a.ctx[seq] > 0 && lane + 32 * i < a.N) ? st[lane + 32 * i] : 0.f;
   const float A = -expf(to_f(static_cast<const T*>(a.A_log)[h])), D = to_f(static_cast<const T*>(a.D)[h]);
   const float bias = to_f(static_cast<const T*>(a.dt_bias)[h]);
   const T* dtc = static_cast<const T*>(a.proj) + inner + ch + h;
@@ -186,6 +199,7 @@ __global__ void __launch_bounds__(256) scan_kernel(const HyMamba a, const T* __r
     o = warp_sum(o);
     if (lane == 0) y[r * inner + h * a.P + p] = from_f<T>(o + D * x);
   }
+  if (slot < 0) return;
 #pragma unroll
   for (int i = 0; i < NR; ++i)
     if (lane + 32 * i < a.N) st[lane + 32 * i] = S[i];
@@ -316,9 +330,9 @@ __device__ __forceinline__ void cp_wait_all() {
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr int MAX_HB = 8;        // heads of one group a CTA works on (a warp computes the decays of each)
 
-// Warp w: step sizes of head h0 + w over the chunk and the running sum of -exp(A_log) dt in units of log2. Tokens past n get
-// dt = 0, so the sum stays flat.
-__device__ __forceinline__ void chunk_decays(const HyMamba& a, int h0, int nh, int row0, int n, float* dts, float* acum) {
+// Warp w, head h0 + w, in units of log2: acum = running sum of -exp(A_log) dt over the chunk, src = acum - log2(dt), so that what
+// token s hands to token t is exp2(acum_t - src_s) = exp(..) dt_s. Tokens past n get dt = 0: the sum stays flat, src = +inf.
+__device__ __forceinline__ void chunk_decays(const HyMamba& a, int h0, int nh, int row0, int n, float* src, float* acum) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (warp >= nh) return;
   const int h = h0 + warp, inner = a.heads * a.P, ch = inner + 2 * a.groups * a.N;
@@ -341,24 +355,37 @@ __device__ __forceinline__ void chunk_decays(const HyMamba& a, int h0, int nh, i
   base -= run;
 #pragma unroll
   for (int i = 0; i < Q / 32; ++i) {
-    dts[warp * Q + lane * (Q / 32) + i] = dt[i];
+    src[warp * Q + lane * (Q / 32) + i] = base + v[i] - log2f(dt[i]);
     acum[warp * Q + lane * (Q / 32) + i] = base + v[i];
   }
 }
 
 // rows [n, w] of a row-major bf16 matrix (pitch `pitch`) into smem [rows][ld], zero filled to wp columns; vec: by 16-byte
 // asynchronous copies the caller waits for
+template <int THREADS>
 __device__ __forceinline__ void load_tile(const bf16* __restrict__ src, long long pitch, int n, int w, int rows, int wp, bf16* dst,
                                           int ld, bool vec) {
   if (vec) {
     const int per = wp / 8;
-    for (int i = threadIdx.x; i < rows * per; i += CW * 32) {
+    if ((THREADS) % per == 0) {  // every thread keeps its column
+      const int step = THREADS / per, r0 = threadIdx.x / per, c = (threadIdx.x - r0 * per) * 8;
+      const bool col = c < w;
+      const bf16* p = src + r0 * pitch + c;
+      uint32_t d = s_u32(dst + r0 * ld + c);
+#pragma unroll 4
+      for (int r = r0; r < rows; r += step, p += step * pitch, d += step * ld * 2) {
+        const bool ok = col && r < n;
+        cp16(d, ok ? p : src, ok ? 16 : 0);
+      }
+      return;
+    }
+    for (int i = threadIdx.x; i < rows * per; i += THREADS) {
       const int r = i / per, c = (i - r * per) * 8;
       const bool ok = r < n && c < w;
       cp16(s_u32(dst + r * ld + c), src + (ok ? r * pitch + c : 0), ok ? 16 : 0);
     }
   } else {
-    for (int i = threadIdx.x; i < rows * wp; i += CW * 32) {
+    for (int i = threadIdx.x; i < rows * wp; i += THREADS) {
       const int r = i / wp, c = i - r * wp;
       dst[r * ld + c] = (r < n && c < w) ? src[r * pitch + c] : __float2bfloat16(0.f);
     }
@@ -383,9 +410,9 @@ __global__ void __launch_bounds__(CW * 32, 2) chunk_state_kernel(const HyMamba a
   bf16* xh = reinterpret_cast<bf16*>(raw);   // [Q][ldx] weighted x, high part
   bf16* xl = xh + Q * ldx;                   // low part
   bf16* Bs = xl + Q * ldx;                   // [Q][ldb]
-  float* dts = reinterpret_cast<float*>(Bs + Q * ldb);  // [MAX_HB][Q]
-  float* acum = dts + MAX_HB * Q;
-  load_tile(xbc + static_cast<long long>(row0) * ch + inner + g * N, ch, n, N, Q, NP, Bs, ldb, vec);
+  float* srcs = reinterpret_cast<float*>(Bs + Q * ldb);  // [MAX_HB][Q]
+  float* acum = srcs + MAX_HB * Q;
+  load_tile<CW * 32>(xbc + static_cast<long long>(row0) * ch + inner + g * N, ch, n, N, Q, NP, Bs, ldb, vec);
   uint4 xr[XV];
   auto fetch = [&](int h) {
 #pragma unroll
@@ -405,20 +432,19 @@ __global__ void __launch_bounds__(CW * 32, 2) chunk_state_kernel(const HyMamba a
     }
   };
   fetch(h0);
-  chunk_decays(a, h0, nh, row0, n, dts, acum);
+  chunk_decays(a, h0, nh, row0, n, srcs, acum);
   cp_wait_all();
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int nt = NP / 64;
   for (int hi = 0; hi < nh; ++hi) {
     const int h = h0 + hi;
-    const float* ac = acum + hi * Q;
-    const float* dt = dts + hi * Q;
-    const float end = ac[Q - 1];
+    const float* from = srcs + hi * Q;
+    const float end = acum[hi * Q + Q - 1];
 #pragma unroll
     for (int i = 0; i < XV; ++i) {
       const int k = threadIdx.x + i * CW * 32, r = k / (PP / 8), c = (k - r * (PP / 8)) * 8;
-      const float w = ex2(end - ac[r]) * dt[r];
+      const float w = ex2(end - from[r]);
       const uint32_t* q = reinterpret_cast<const uint32_t*>(&xr[i]);
       uint32_t hi4[4], lo4[4];
 #pragma unroll
@@ -488,9 +514,10 @@ __global__ void __launch_bounds__(256) chunk_pass_kernel(const HyMamba a, const 
   const long long size = static_cast<long long>(a.P) * a.N;
   const long long i = (static_cast<long long>(blockIdx.x) * 256 + threadIdx.x) * V;
   if (i >= size) return;
-  float* st = a.state + (static_cast<long long>(a.slots[seq]) * a.heads + h) * size + i;
+  const long long slot = state_row(a, seq);
+  float* st = a.state + ((slot < 0 ? 0 : slot) * a.heads + h) * size + i;
   float s[V];
-  const bool cont = a.ctx[seq] > 0;
+  const bool cont = slot >= 0 && a.ctx[seq] > 0;
   auto load = [](const float* p, float (&v)[V]) {
     if constexpr (V == 4) {
       const float4 t = *reinterpret_cast<const float4*>(p);
@@ -530,6 +557,7 @@ __global__ void __launch_bounds__(256) chunk_pass_kernel(const HyMamba a, const 
       for (int k = 0; k < V; ++k) s[k] = d[u] * s[k] + v[u][k];
     }
   }
+  if (slot < 0) return;
   if constexpr (V == 4)
     *reinterpret_cast<float4*>(st) = make_float4(s[0], s[1], s[2], s[3]);
   else
@@ -538,11 +566,13 @@ __global__ void __launch_bounds__(256) chunk_pass_kernel(const HyMamba a, const 
 
 // (3) y[t] = exp(acum_t) C_t S_before + sum_{s <= t} (C_t . B_s) exp(acum_t - acum_s) dt_s x_s + D x_t
 //
-// A CTA takes several heads of a group: the products C B^T of the chunk are the same for all of them and stay in registers. The
-// lower triangle has 36 blocks of 16 x 16 tokens; four warps take the row tiles (w, 7 - w), nine blocks each, and two such sets
-// split the columns p.
-template <int PH>  // 16-wide tiles of P per half
-__global__ void __launch_bounds__(CW * 32, PH <= 2 ? 2 : 1)
+// A CTA takes several heads of a group: the products C B^T of the chunk are the same for all of them and are kept in shared
+// memory, fragment by fragment. The lower triangle has 36 blocks of 16 x 16 tokens; a warp takes the row tiles (w, 7 - w), nine
+// blocks, and 16 * PH columns p. With NBUF = 2 the next head's x and carried state arrive while this one computes.
+constexpr int OW = 16;  // warps
+
+template <int PH, int NBUF>
+__global__ void __launch_bounds__(OW * 32, 1)
 chunk_out_kernel(const HyMamba a, const bf16* __restrict__ xbc, const int4* __restrict__ chunks, int hb,
                  const bf16* __restrict__ before, bf16* __restrict__ y, bool vec) {
   extern __shared__ __align__(16) unsigned char raw[];
@@ -552,117 +582,144 @@ chunk_out_kernel(const HyMamba a, const bf16* __restrict__ xbc, const int4* __re
   const int inner = a.heads * P, ch = inner + 2 * a.groups * N;
   const int per_group = (hpg + hb - 1) / hb, g = blockIdx.y / per_group;
   const int h0 = g * hpg + (blockIdx.y - g * per_group) * hb, nh = min(hb, (g + 1) * hpg - h0);
-  constexpr int PP = PH * 32;
+  constexpr int PP = PH * 64;
   constexpr int ldx = PP + LDX_PAD;
   const int ldn = NP + LDX_PAD;
-  bf16* Cs = reinterpret_cast<bf16*>(raw);  // [Q][ldn]
-  bf16* xs = Cs + Q * ldn;                  // [Q][ldx]
-  bf16* Bs = xs + Q * ldx;                  // [Q][ldn], later the carried state: [2][PP][ldn]
-  bf16* Ss = Bs;
-  float* dts = reinterpret_cast<float*>(Bs + (Q > 2 * PP ? Q : 2 * PP) * ldn);  // [MAX_HB][Q]
-  float* acum = dts + MAX_HB * Q;
+  float* Gs = reinterpret_cast<float*>(raw);             // [36][32 lanes][8]
+  float* srcs = Gs + 36 * 256;                           // [MAX_HB][Q]
+  float* acum = srcs + MAX_HB * Q;
+  bf16* Cs = reinterpret_cast<bf16*>(acum + MAX_HB * Q); // [Q][ldn]
+  bf16* xs = Cs + Q * ldn;                               // [NBUF][Q][ldx]
+  bf16* Ss = xs + NBUF * Q * ldx;                        // [NBUF][2][PP][ldn]; the first one holds B before that
   const bool carried = ck.w > 0 || a.ctx[seq] > 0;
   const bf16* rows = xbc + static_cast<long long>(row0) * ch;
-  load_tile(rows + inner + a.groups * N + g * N, ch, n, N, Q, NP, Cs, ldn, vec);
-  load_tile(rows + inner + g * N, ch, n, N, Q, NP, Bs, ldn, vec);
-  chunk_decays(a, h0, nh, row0, n, dts, acum);
+  load_tile<OW * 32>(rows + inner + a.groups * N + g * N, ch, n, N, Q, NP, Cs, ldn, vec);
+  load_tile<OW * 32>(rows + inner + g * N, ch, n, N, Q, NP, Ss, ldn, vec);
+  chunk_decays(a, h0, nh, row0, n, srcs, acum);
   cp_wait_all();
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int half = warp >> 2, ta = warp & 3, tb = 7 - ta;   // this warp's row tiles
+  const int pg = warp >> 2, ta = warp & 3, tb = 7 - ta;     // column group, row tiles
   const int a_row = lane & 15, a_col = (lane >> 4) << 3;
   const int b_row = (lane & 7) + ((lane >> 4) << 3), b_col = ((lane >> 3) & 1) << 3;    // [n][k] operands
   const int v_row = (lane & 7) + (((lane >> 3) & 1) << 3), v_col = (lane >> 4) << 3;    // [k][n] operands
-  float gm[9][2][4];
-#pragma unroll
-  for (int i = 0; i < 9; ++i) {
-    const int tile = i <= ta ? ta : tb, s = i <= ta ? i : i - ta - 1;
-#pragma unroll
-    for (int e = 0; e < 4; ++e) gm[i][0][e] = gm[i][1][e] = 0.f;
-    const uint32_t ca = s_u32(Cs + (tile * 16 + a_row) * ldn + a_col), ba = s_u32(Bs + (s * 16 + b_row) * ldn + b_col);
-#pragma unroll 2
+  for (int blk = warp; blk < 36; blk += OW) {
+    int r = 0;
+    while ((r + 1) * (r + 2) / 2 <= blk) ++r;
+    const int s = blk - r * (r + 1) / 2;
+    float g0[4] = {0.f, 0.f, 0.f, 0.f}, g1[4] = {0.f, 0.f, 0.f, 0.f};
+    const uint32_t ca = s_u32(Cs + (r * 16 + a_row) * ldn + a_col), ba = s_u32(Ss + (s * 16 + b_row) * ldn + b_col);
+#pragma unroll 4
     for (int k0 = 0; k0 < NP; k0 += 16) {
       uint32_t cf[4], b[4];
       ldsm4(ca + k0 * 2, cf);
       ldsm4(ba + k0 * 2, b);
-      mma(gm[i][0], cf, b[0], b[1]);
-      mma(gm[i][1], cf, b[2], b[3]);
+      mma(g0, cf, b[0], b[1]);
+      mma(g1, cf, b[2], b[3]);
     }
+    float4* dst = reinterpret_cast<float4*>(Gs + blk * 256) + lane;  // two planes of 16 bytes per lane
+    dst[0] = make_float4(g0[0], g0[1], g0[2], g0[3]);
+    dst[32] = make_float4(g1[0], g1[1], g1[2], g1[3]);
   }
-  const int pc0 = half * PH * 16;  // first column of this warp
-  for (int hi = 0; hi < nh; ++hi) {
-    const int h = h0 + hi;
-    __syncthreads();  // B, or the previous head's tiles, have been read
-    load_tile(rows + h * P, ch, n, P, Q, PP, xs, ldx, vec);
+  __syncthreads();
+  auto fetch = [&](int hi) {
+    const int h = h0 + hi, buf = NBUF == 2 ? hi & 1 : 0;
+    load_tile<OW * 32>(rows + h * P, ch, n, P, Q, PP, xs + buf * Q * ldx, ldx, vec);
     if (carried) {
       const bf16* src = before + (static_cast<long long>(blockIdx.x) * a.heads + h) * 2 * P * N;
-      load_tile(src, N, P, N, PP, NP, Ss, ldn, vec);
-      load_tile(src + static_cast<long long>(P) * N, N, P, N, PP, NP, Ss + PP * ldn, ldn, vec);
+      bf16* dst = Ss + buf * 2 * PP * ldn;
+      load_tile<OW * 32>(src, N, P, N, PP, NP, dst, ldn, vec);
+      load_tile<OW * 32>(src + static_cast<long long>(P) * N, N, P, N, PP, NP, dst + PP * ldn, ldn, vec);
     }
-    cp_wait_all();
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  fetch(0);
+  const int pc0 = pg * PH * 16;  // first column of this warp
+  for (int hi = 0; hi < nh; ++hi) {
+    const int h = h0 + hi, buf = NBUF == 2 ? hi & 1 : 0;
+    if (NBUF == 2 && hi + 1 < nh) {
+      fetch(hi + 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
     __syncthreads();
-    const float* ac = acum + hi * Q;
-    const float* dt = dts + hi * Q;
-    const float D = to_f(static_cast<const bf16*>(a.D)[h]);
-    float o[2 * PH][4];
-#pragma unroll
-    for (int i = 0; i < 9; ++i) {
-      const int tile = i <= ta ? ta : tb, s0 = (i <= ta ? i : i - ta - 1) * 16;
-      const int r0 = tile * 16 + (lane >> 2);
-      const float ac0 = ac[r0], ac1 = ac[r0 + 8];
-      if (i == 0 || i == ta + 1) {  // a row tile begins: what the carried state gives
+    if (pc0 < P) {
+      const bf16* xb = xs + buf * Q * ldx;
+      const bf16* sb = Ss + buf * 2 * PP * ldn;
+      const float* ac = acum + hi * Q;
+      const float* from = srcs + hi * Q;
+      const float D = to_f(static_cast<const bf16*>(a.D)[h]);
+#pragma unroll 1
+      for (int half = 0; half < 2; ++half) {
+        const int tile = half == 0 ? ta : tb;
+        if (tile * 16 >= n) continue;
+        const int r0 = tile * 16 + (lane >> 2);
+        const float ac0 = ac[r0], ac1 = ac[r0 + 8];
+        float o[2 * PH][4];
 #pragma unroll
         for (int j = 0; j < 2 * PH; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-        if (carried) {
-          const uint32_t ca = s_u32(Cs + (tile * 16 + a_row) * ldn + a_col), sa = s_u32(Ss + (pc0 + b_row) * ldn + b_col);
-#pragma unroll 1
+        if (carried) {  // what the carried state gives; the two parts of the split in accumulators of their own
+          float q[2 * PH][4];
+#pragma unroll
+          for (int j = 0; j < 2 * PH; ++j) q[j][0] = q[j][1] = q[j][2] = q[j][3] = 0.f;
+          const uint32_t ca = s_u32(Cs + (tile * 16 + a_row) * ldn + a_col), sa = s_u32(sb + (pc0 + b_row) * ldn + b_col);
+#pragma unroll 4
           for (int k0 = 0; k0 < NP; k0 += 16) {
             uint32_t cf[4];
             ldsm4(ca + k0 * 2, cf);
 #pragma unroll
             for (int jp = 0; jp < PH; ++jp) {
-              uint32_t b[4];
+              uint32_t b[4], c[4];
               ldsm4(sa + (jp * 16 * ldn + k0) * 2, b);
+              ldsm4(sa + ((PP + jp * 16) * ldn + k0) * 2, c);
               mma(o[2 * jp], cf, b[0], b[1]);
               mma(o[2 * jp + 1], cf, b[2], b[3]);
-              ldsm4(sa + ((PP + jp * 16) * ldn + k0) * 2, b);
-              mma(o[2 * jp], cf, b[0], b[1]);
-              mma(o[2 * jp + 1], cf, b[2], b[3]);
+              mma(q[2 * jp], cf, c[0], c[1]);
+              mma(q[2 * jp + 1], cf, c[2], c[3]);
             }
           }
           const float e0 = ex2(ac0), e1 = ex2(ac1);
 #pragma unroll
           for (int j = 0; j < 2 * PH; ++j) {
-            o[j][0] *= e0; o[j][1] *= e0;
-            o[j][2] *= e1; o[j][3] *= e1;
+            o[j][0] = (o[j][0] + q[j][0]) * e0; o[j][1] = (o[j][1] + q[j][1]) * e0;
+            o[j][2] = (o[j][2] + q[j][2]) * e1; o[j][3] = (o[j][3] + q[j][3]) * e1;
           }
         }
-      }
-      // scores -> decay-weighted coefficients, split in two bf16 terms; accumulator layout = A-operand layout
-      uint32_t wh[4], wl[4];
+        const float4* gp = reinterpret_cast<const float4*>(Gs + tile * (tile + 1) / 2 * 256) + lane;
+        auto block = [&](int st, bool diag) {
+          const int s0 = st * 16;
+          // scores -> decay-weighted coefficients, split in two bf16 terms; accumulator layout = A-operand layout
+          uint32_t wh[4], wl[4];
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt) {
-        const int s = s0 + nt * 8 + (lane & 3) * 2;
-        const float2 as = *reinterpret_cast<const float2*>(ac + s), ds = *reinterpret_cast<const float2*>(dt + s);
-        float w[4];
-        w[0] = s <= r0 ? gm[i][nt][0] * ex2(ac0 - as.x) * ds.x : 0.f;
-        w[1] = s + 1 <= r0 ? gm[i][nt][1] * ex2(ac0 - as.y) * ds.y : 0.f;
-        w[2] = s <= r0 + 8 ? gm[i][nt][2] * ex2(ac1 - as.x) * ds.x : 0.f;
-        w[3] = s + 1 <= r0 + 8 ? gm[i][nt][3] * ex2(ac1 - as.y) * ds.y : 0.f;
-        split2(w[0], w[1], wh[nt * 2], wl[nt * 2]);
-        split2(w[2], w[3], wh[nt * 2 + 1], wl[nt * 2 + 1]);
-      }
-      const uint32_t xa = s_u32(xs + (s0 + v_row) * ldx + pc0 + v_col);
+          for (int nt = 0; nt < 2; ++nt) {
+            const int s = s0 + nt * 8 + (lane & 3) * 2;
+            const float4 gv = gp[st * 64 + nt * 32];
+            const float2 as = *reinterpret_cast<const float2*>(from + s);
+            float w0 = gv.x * ex2(ac0 - as.x), w1 = gv.y * ex2(ac0 - as.y), w2 = gv.z * ex2(ac1 - as.x), w3 = gv.w * ex2(ac1 - as.y);
+            if (diag) {  // only tokens up to t
+              w0 = s <= r0 ? w0 : 0.f;
+              w1 = s + 1 <= r0 ? w1 : 0.f;
+              w2 = s <= r0 + 8 ? w2 : 0.f;
+              w3 = s + 1 <= r0 + 8 ? w3 : 0.f;
+            }
+            split2(w0, w1, wh[nt * 2], wl[nt * 2]);
+            split2(w2, w3, wh[nt * 2 + 1], wl[nt * 2 + 1]);
+          }
+          const uint32_t xa = s_u32(xb + (s0 + v_row) * ldx + pc0 + v_col);
 #pragma unroll
-      for (int jp = 0; jp < PH; ++jp) {
-        uint32_t b[4];
-        ldsm4t(xa + jp * 32, b);
-        mma(o[2 * jp], wh, b[0], b[1]);
-        mma(o[2 * jp], wl, b[0], b[1]);
-        mma(o[2 * jp + 1], wh, b[2], b[3]);
-        mma(o[2 * jp + 1], wl, b[2], b[3]);
-      }
-      if (i == ta || i == 8) {  // the row tile is complete
+          for (int jp = 0; jp < PH; ++jp) {
+            uint32_t b[4];
+            ldsm4t(xa + jp * 32, b);
+            mma(o[2 * jp], wh, b[0], b[1]);
+            mma(o[2 * jp + 1], wh, b[2], b[3]);
+            mma(o[2 * jp], wl, b[0], b[1]);
+            mma(o[2 * jp + 1], wl, b[2], b[3]);
+          }
+        };
+#pragma unroll 2
+        for (int st = 0; st < tile; ++st) block(st, false);
+        block(tile, true);
 #pragma unroll
         for (int j = 0; j < 2 * PH; ++j) {
           const int p = pc0 + j * 8 + (lane & 3) * 2;
@@ -671,7 +728,8 @@ chunk_out_kernel(const HyMamba a, const bf16* __restrict__ xbc, const int4* __re
             const int t = r0 + e * 8;
             if (t >= n) continue;
             bf16* dst = y + static_cast<long long>(row0 + t) * inner + h * P + p;
-            const float u = o[j][2 * e] + D * to_f(xs[t * ldx + p]), v = o[j][2 * e + 1] + D * to_f(xs[t * ldx + p + 1]);
+            const float2 xv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(xb + t * ldx + p));
+            const float u = o[j][2 * e] + D * xv.x, v = o[j][2 * e + 1] + D * xv.y;
             if ((P & 1) == 0) {
               if (p < P) *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(u, v);
             } else {
@@ -682,6 +740,8 @@ chunk_out_kernel(const HyMamba a, const bf16* __restrict__ xbc, const int4* __re
         }
       }
     }
+    __syncthreads();  // this head's tiles have been read
+    if (NBUF == 1 && hi + 1 < nh) fetch(hi + 1);
   }
 }
 
@@ -740,10 +800,10 @@ size_t state_smem(int PT, int N) {
   const int NP = (N + 63) / 64 * 64;
   return static_cast<size_t>(2) * (2 * Q * (PT * 16 + LDX_PAD) + Q * (NP + LDX_PAD)) + 2 * MAX_HB * Q * sizeof(float);
 }
-size_t out_smem(int PH, int N) {
-  const int NP = (N + 15) / 16 * 16, PP = PH * 32;
-  return static_cast<size_t>(2) * (Q * (NP + LDX_PAD) + Q * (PP + LDX_PAD) + (Q > 2 * PP ? Q : 2 * PP) * (NP + LDX_PAD)) +
-         2 * MAX_HB * Q * sizeof(float);
+size_t out_smem(int PH, int N, int nbuf) {
+  const int NP = (N + 15) / 16 * 16, PP = PH * 64;
+  return sizeof(float) * (36 * 256 + 2 * MAX_HB * Q) +
+         static_cast<size_t>(2) * (Q * (NP + LDX_PAD) + nbuf * (Q * (PP + LDX_PAD) + 2 * PP * (NP + LDX_PAD)));
 }
 int half_tiles(int P) { return (P + 31) / 32; }
 
@@ -766,14 +826,14 @@ int launch_state(const HyMamba& a, const bf16* xbc, const int4* ck, int n_chunks
   return static_cast<int>(cudaGetLastError());
 }
 
-template <int PH>
+template <int PH, int NBUF>
 int launch_out(const HyMamba& a, const bf16* xbc, const int4* ck, int n_chunks, int hb, const bf16* before, bf16* y, bool vec, cudaStream_t s) {
-  const size_t smem = out_smem(PH, a.N);
-  auto kern = chunk_out_kernel<PH>;
+  const size_t smem = out_smem(PH, a.N, NBUF);
+  auto kern = chunk_out_kernel<PH, NBUF>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   const int hpg = a.heads / a.groups;
-  kern<<<dim3(n_chunks, a.groups * ((hpg + hb - 1) / hb)), CW * 32, smem, s>>>(a, xbc, ck, hb, before, y, vec);
+  kern<<<dim3(n_chunks, a.groups * ((hpg + hb - 1) / hb)), OW * 32, smem, s>>>(a, xbc, ck, hb, before, y, vec);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -792,7 +852,7 @@ int hy_mamba_step(bool f32, const HyMamba& a, const int* positions, int B, void*
 bool hy_chunk_scan_supported(int P, int N, int, int) {
   if (P < 1 || P > 128 || N < 1 || N > 256) return false;
   const int ph = half_tiles(P);
-  return state_smem(2 * ph, N) <= 227 * 1024 && out_smem(ph, N) <= 227 * 1024;
+  return state_smem(2 * ph, N) <= 227 * 1024 && out_smem(P <= 64 ? 1 : 2, N, 1) <= 227 * 1024;
 }
 
 int hy_chunk_scan(const HyMamba& a, const void* xbc_, const int* chunks, int n_chunks, const int* first_chunk, float* work,
@@ -818,12 +878,10 @@ int hy_chunk_scan(const HyMamba& a, const void* xbc_, const int* chunks, int n_c
     chunk_pass_kernel<1><<<dim3(static_cast<unsigned>((size + 255) / 256), a.heads, a.nseq), 256, 0, s>>>(a, first_chunk, decay, work, before);
   const cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return static_cast<int>(e);
-  switch (ph) {
-    case 1: return launch_out<1>(a, xbc, ck, n_chunks, hb, before, y, vec, s);
-    case 2: return launch_out<2>(a, xbc, ck, n_chunks, hb, before, y, vec, s);
-    case 3: return launch_out<3>(a, xbc, ck, n_chunks, hb, before, y, vec, s);
-    default: return launch_out<4>(a, xbc, ck, n_chunks, hb, before, y, vec, s);
-  }
+  const bool two = out_smem(a.P <= 64 ? 1 : 2, a.N, 2) <= 227 * 1024;
+  if (a.P <= 64)
+    return two ? launch_out<1, 2>(a, xbc, ck, n_chunks, hb, before, y, vec, s) : launch_out<1, 1>(a, xbc, ck, n_chunks, hb, before, y, vec, s);
+  return two ? launch_out<2, 2>(a, xbc, ck, n_chunks, hb, before, y, vec, s) : launch_out<2, 1>(a, xbc, ck, n_chunks, hb, before, y, vec, s);
 }
 
 }  // namespace mb

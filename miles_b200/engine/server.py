@@ -182,9 +182,8 @@ def serve(engine: Engine, host: str = "127.0.0.1", port: int = 30000, tokenizer=
     uvicorn.run(build_app(engine, tokenizer, model_path), host=host, port=port, log_level="warning")
 
 
-def main(argv=None) -> None:
-    """``python -m miles_b200.engine.server --model-preset qwen3-4B --port 30000``: one engine process on this GPU
-    (or on the CPU with the PyTorch model), ready to be driven over HTTP and to join a trainer's weight-update group."""
+def build_from_args(argv=None):
+    """Parse the server's command line and build the engine it describes: (engine, tokenizer, arguments)."""
     import argparse
 
     import torch
@@ -202,12 +201,19 @@ def main(argv=None) -> None:
     ap.add_argument("--context-length", type=int, default=9224)
     ap.add_argument("--mem-fraction-static", type=float, default=0.85)
     ap.add_argument("--quantization", default="none", choices=["none", "mxfp8", "nvfp4"])
+    ap.add_argument("--dtype", default="auto", choices=["auto", "bfloat16", "float32"],
+                    help="auto: bfloat16 on a GPU, float32 on the CPU; float32 on a GPU is built for models with a layer plan")
+    ap.add_argument("--max-prefill-tokens", type=int, default=16384, help="tokens of one prefill pass; planned-layer models compute longer prompts in portions")
     ap.add_argument("--seed", type=int, default=1234)
     ap.add_argument("--disable-radix-cache", action="store_true", help="turn the prefix (radix) cache off")
     ns = ap.parse_args(argv)
     cfg = get_config(ns.model_preset or ns.hf_checkpoint)
     on_gpu = ns.device.startswith("cuda")
-    dtype = torch.bfloat16 if on_gpu else torch.float32
+    dtype = (torch.bfloat16 if on_gpu else torch.float32) if ns.dtype == "auto" else getattr(torch, ns.dtype)
+    if on_gpu and dtype == torch.float32 and cfg.plan is None:
+        ap.error(f"{cfg.name} runs in bfloat16 on a GPU")
+    if ns.quantization != "none" and cfg.plan is not None:
+        ap.error("block-scaled weights are not built for models with a layer plan")
     store = ParamStore(cfg, ns.device, dtype, seed=ns.seed)
     tokenizer = None
     if ns.hf_checkpoint:
@@ -215,7 +221,11 @@ def main(argv=None) -> None:
         from ..utils.processing_utils import load_tokenizer
 
         load_hf(cfg, store, ns.hf_checkpoint)
-        tokenizer = load_tokenizer(ns.hf_checkpoint)
+        import os
+
+        # a design without a tokenizer of its own is served token-in / token-out
+        if cfg.plan is None or any(f.startswith("tokenizer") for f in os.listdir(ns.hf_checkpoint)):
+            tokenizer = load_tokenizer(ns.hf_checkpoint)
     model = build_model(cfg, store, "auto" if cfg.plan is not None else "b200" if (on_gpu and cfg.head_dim == 128) else "torch")
     if ns.quantization != "none" and hasattr(model, "enable_block_scaled"):
         model.enable_block_scaled(ns.quantization)
@@ -224,9 +234,16 @@ def main(argv=None) -> None:
         free, total = torch.cuda.mem_get_info()
         kv_bytes = max(int(free - (1.0 - ns.mem_fraction_static) * total), 1 << 28)
     engine = Engine(model, max_running=ns.max_running_requests, page_size=ns.page_size, max_seq_len=ns.context_length,
-                    kv_mem_bytes=kv_bytes, use_cuda_graph=on_gpu, eos_token_id=getattr(tokenizer, "eos_token_id", None),
+                    max_prefill_tokens=ns.max_prefill_tokens, kv_mem_bytes=kv_bytes, use_cuda_graph=on_gpu, eos_token_id=getattr(tokenizer, "eos_token_id", None),
                     prefix_cache=not ns.disable_radix_cache, memory_saver=on_gpu)
     engine.seed_salt = ns.seed * 1000003 + ns.port  # engines of one fleet share --seed and differ by port
+    return engine, tokenizer, ns
+
+
+def main(argv=None) -> None:
+    """``python -m miles_b200.engine.server --model-preset qwen3-4B --port 30000``: one engine process on this GPU
+    (or on the CPU with the PyTorch model), ready to be driven over HTTP and to join a trainer's weight-update group."""
+    engine, tokenizer, ns = build_from_args(argv)
     serve(engine, ns.host, ns.port, tokenizer, ns.hf_checkpoint or ns.model_preset or "")
 
 

@@ -30,7 +30,7 @@ from .torch_impl import InferMeta
 
 CONV_TILE = 32
 SMALL_T = 32       # rows up to which products stream the weights instead of filling tcgen05 tiles
-FUSED_SIDE_T = 256  # rows up to which the per-layer token input is one kernel
+FUSED_SIDE_T = 16  # rows up to which the per-layer token input is one kernel
 
 
 class B200Hybrid(TorchHybrid):
@@ -193,14 +193,14 @@ class B200Hybrid(TorchHybrid):
             self.launches += 1
         nn = self._next_norm(i)
         gate, sproj = P[p + "side.gate.weight"], P[p + "side.proj.weight"]
-        side = (x, delta, tokens, gate, sproj, P[p + "side.norm.weight"], P["side.embed.weight"], i, P[nn + ".weight"], P[nn + ".bias"],
+        side = (x, None, tokens, gate, sproj, P[p + "side.norm.weight"], P["side.embed.weight"], i, P[nn + ".weight"], P[nn + ".bias"],
                 P[nn + ".alpha"], h, self.plan.eps, self.status)
-        if T <= FUSED_SIDE_T or self.f32 or delta is not None or sproj.shape[1] % 8 or x.shape[1] % 8 or self.plain:
-            C.side_fused(*side)
+        if T <= FUSED_SIDE_T or self.f32 or sproj.shape[1] % 8 or x.shape[1] % 8 or self.plain:
+            C.side_fused(x, delta, *side[2:])
             self.launches += 1
             return
         xb = torch.empty_like(h)
-        C.cast_rows(x, xb)
+        C.cast_rows(x, delta, xb)
         g = torch.empty(T, gate.shape[0], dtype=h.dtype, device=self.dev)
         C.side_gate(*side, self.linear(xb, gate, torch.float32), g)
         C.side_finish(*side, self.linear(g, sproj, torch.float32))

@@ -12,7 +12,7 @@ from dataclasses import asdict, dataclass, field
 from pathlib import Path
 from typing import Any, Optional
 
-from .layer_plan import DESIGNS, LayerPlan, plan_specs, read_plan, write_plan
+from .layer_plan import DESIGNS, DenseFF, LatentAttention, Layer, LayerPlan, Mamba2, Rotary, plan_specs, read_plan, write_plan
 
 
 @dataclass
@@ -421,6 +421,22 @@ PRESETS: dict[str, ModelConfig] = {
     "mimo-7B-rl": _dense("mimo-7B-rl", 36, 4096, 32, 8, 11008, False, vocab=151680, qk_norm=False, qkv_bias=True,
                          rope_theta=640000.0, rms_eps=1e-5, hf_architecture="Qwen2ForCausalLM"),
 }
+
+
+def _rokivik_smoke() -> ModelConfig:
+    """A small Rokivik: recurrent, attention and latent-sharing layers, one of them without a feed-forward."""
+    rot = Rotary(base=1e4, dims=32)
+    attn = dict(heads=6, dim=32, rot_dim=32, vdim=48, kv_rank=96, q_rank=160, scale=0.125, rotary=rot)
+    layers = [Layer(Mamba2(heads=12, vdim=32, state=64, groups=3, conv=4, norm_groups=6), DenseFF(768)),
+              Layer(LatentAttention(window=192, **attn), DenseFF(768)),
+              Layer(LatentAttention(window=1024, kv_from=1, **attn)),
+              Layer(Mamba2(heads=8, vdim=64, state=32, groups=1, conv=4, norm_groups=1), DenseFF(768))]
+    plan = LayerPlan("Rokivik", layers, eps=1e-5, token_side=24)
+    plan.validate()
+    return ModelConfig.from_plan(plan, 4096, 384, name="rokivik-smoke")
+
+
+PRESETS["rokivik-smoke"] = _rokivik_smoke()
 
 
 def get_config(name: str) -> ModelConfig:

@@ -498,6 +498,9 @@ def _first_dense_layers(freq, num_layers: int) -> int:
 def _check_architecture_flags(args, cfg):
     """The model comes from a preset or a checkpoint: architecture flags that were given and say something else would
     otherwise be dropped without a word (and the job would train another model than the command line describes)."""
+    if cfg.plan is not None:
+        raise NotImplementedError(f"model {cfg.name!r} is served (engine, python -m miles_b200.engine.server, bin/trace_run), not trained: "
+                                  "its mixers have no backward pass here")
     moe = cfg.is_moe
     given = [("moe_router_score_function", cfg.router_score if moe else "softmax", "softmax"),
              ("moe_router_enable_expert_bias", bool(cfg.router_bias), False),

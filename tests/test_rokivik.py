@@ -241,3 +241,28 @@ def test_trace_run_command(tmp_path):
     want = O.model(cfg, W, toks)
     got = torch.frombuffer(bytearray((out / "0.f32").read_bytes() + (out / "2.f32").read_bytes()), dtype=torch.float32).view(3, -1)
     assert rel(got, want[[2, 6, 11]]) < TOL and not (out / "1.f32").exists()
+
+
+def test_server_command_line_serves_the_design_and_training_refuses_it(tmp_path):
+    from fastapi.testclient import TestClient
+
+    from miles_b200.engine.server import build_app, build_from_args
+    from miles_b200.utils.arguments import parse_args
+
+    cfg = CASES["mixed"]
+    W = O.random_weights(cfg, seed=3, dtype=torch.float32)
+    d = O.write_checkpoint(tmp_path, cfg, W)
+    engine, tokenizer, _ = build_from_args(["--hf-checkpoint", str(d), "--device", "cpu", "--max-running-requests", "2", "--page-size", "8",
+                                            "--context-length", "64", "--max-prefill-tokens", "9"])
+    assert tokenizer is None and engine.max_prefill_tokens == 9
+    toks = tokens_of(21, cfg["vocab"], 1)
+    with TestClient(build_app(engine)) as client:
+        r = client.post("/generate", json={"input_ids": toks, "sampling_params": {"temperature": 0.0, "max_new_tokens": 5}}).json()
+    lg = O.model(cfg, W, toks + r["output_ids"][:-1])[-5:]
+    assert (lg.max(-1).values - lg.gather(1, torch.tensor(r["output_ids"])[:, None])[:, 0]).max() < 1e-3
+    with pytest.raises(SystemExit):
+        build_from_args(["--hf-checkpoint", str(d), "--device", "cpu", "--quantization", "mxfp8"])
+    from miles_b200.utils.arguments import model_config_from_args
+
+    with pytest.raises(NotImplementedError):
+        model_config_from_args(parse_args(["--model-preset", "rokivik-smoke", "--num-rollout", "1", "--rollout-batch-size", "1"]))

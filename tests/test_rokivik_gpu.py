@@ -89,11 +89,13 @@ def test_recurrence_in_portions_and_steps(dims, mode):
     assert int(status) == 0
 
 
-def test_recurrence_batch_of_unequal_sequences():
-    H, P, N, G, taps = 4, 64, 64, 2, 4
+@pytest.mark.parametrize("lens", [[1, 130, 7, 256, 300], [40] * 500 + [257]])
+@pytest.mark.parametrize("dims", [(4, 64, 64, 2, 4), (24, 32, 32, 3, 4)])
+def test_recurrence_batch_of_unequal_sequences(lens, dims):
+    """(the long batch also gives every block of the chunked form several heads of a group)"""
+    H, P, N, G, taps = dims
     C = ext()
-    lens = [1, 130, 7, 256, 300]
-    ds = [mamba_inputs(H, P, N, G, taps, n, 10 + n, torch.bfloat16) for n in lens]
+    ds = [mamba_inputs(H, P, N, G, taps, n, 10 + i, torch.bfloat16) for i, n in enumerate(lens)]
     proj = torch.cat([d["proj"] for d in ds])
     w = ds[0]["weights"]
     for d in ds:
@@ -105,13 +107,16 @@ def test_recurrence_batch_of_unequal_sequences():
         chunks += [(b, cu[-1] + r, min(C.CHUNK, n - r), r // C.CHUNK) for r in range(0, n, C.CHUNK)]
         first.append(len(chunks))
         cu.append(cu[-1] + n)
-    ring = torch.zeros(6, taps, H * P + 2 * G * N, dtype=torch.bfloat16, device="cuda")
-    state = torch.zeros(6, H, P, N, device="cuda")
+    B = len(lens)
+    ring = torch.zeros(B + 1, taps, H * P + 2 * G * N, dtype=torch.bfloat16, device="cuda")
+    state = torch.zeros(B + 1, H, P, N, device="cuda")
     status = torch.zeros(1, dtype=torch.int32, device="cuda")
     y = torch.empty(cu[-1], H * P, dtype=torch.bfloat16, device="cuda")
-    C.mamba_prefill(proj, H, P, N, G, *w, ring, state, i32([4, 2, 0, 1, 3]), status, i32(cu), i32([0] * 5), i32(conv), i32(chunks), i32(first), y)
+    C.mamba_prefill(proj, H, P, N, G, *w, ring, state, i32([(b * 7 + 3) % B for b in range(B)]), status, i32(cu), i32([0] * B), i32(conv), i32(chunks), i32(first), y)
     for b, d in enumerate(ds):
-        close(y[cu[b]:cu[b + 1]], mamba_want(d, H, P, N, G), 0.02, lens[b])
+        if b < 4 or b > B - 3:
+            close(y[cu[b]:cu[b + 1]], mamba_want(d, H, P, N, G), 0.02, lens[b])
+    assert int(status) == 0
 
 
 def test_state_row_outside_the_cache_is_reported_not_followed():
@@ -122,6 +127,11 @@ def test_state_row_outside_the_cache_is_reported_not_followed():
     state = torch.zeros(2, H, P, N, device="cuda")
     ext().mamba_step(d["proj"], H, P, N, G, *d["weights"], ring, state, i32([7]), status, i32([3]), torch.empty(1, H * P, dtype=torch.bfloat16, device="cuda"))
     assert int(status) == 11 and float(state.abs().sum()) == 0
+    d = mamba_inputs(H, P, N, G, 4, 40, 1, torch.bfloat16)
+    for chunked in (False, True):
+        status.zero_()
+        y = run_portions(d, H, P, N, G, 4, [40], torch.bfloat16, chunked, ring, state, 2, status)
+        assert int(status) == 11 and float(state.abs().sum()) == 0 and torch.isfinite(y.float()).all()
 
 
 @pytest.mark.parametrize("inner,groups", [(64, 1), (96, 3), (512, 8), (130, 13), (4096, 2), (21, 7)])
