@@ -157,6 +157,7 @@ def floors(cfg, kind: str, s: dict, T: int, ctx: int, prefill: bool) -> dict:
             f["latent_decode"] = (T * L * W * 2 + T * h * (W * 2 + R * 4), 2 * T * L * h * (W + R))
             f["absorb_q"] = (h * 128 * R * 2 + T * h * (192 + W) * 2, 2 * T * h * 128 * R)
             f["latent_up"] = (h * 128 * R * 2 + T * h * (R * 4 + 128 * 2), 2 * T * h * 128 * R)
+            f["absorb_mma"], f["up_mma"] = f["absorb_q"], f["latent_up"]
             f["side_fused"] = (2 * s["side"] * H * 2 + T * H * (4 + 4 + 4 + 2), 4 * T * s["side"] * H)
     else:
         hq, hk = cfg.num_q_heads, cfg.num_kv_heads

@@ -578,6 +578,145 @@ size_t decode_smem(int MT, int rank, int rot) {
   return sizeof(bf16) * (static_cast<size_t>(2) * TOK * ld + MT * 16 * ld + MT * 16 * PLD) + sizeof(float) * 2 * DW * MT * 16;
 }
 
+// ------------------------------------------------------------------------------------------------ projections of many rows
+// Tensor-core forms of the two per-head projections (bf16, more rows than the kernels above share a weight read among).
+constexpr int HM = 32;    // rows per CTA
+constexpr int AN = 128;   // latent columns per CTA (queries into latent space)
+constexpr int UN = 32;    // output values per CTA (latent outputs back)
+
+// ql[t, h, r] = sum_d q[t, h, d] W_uk[h * dim + d, r]; the block after the last column tile writes rotated part and padding.
+template <typename O>
+__global__ void __launch_bounds__(128) absorb_mma_kernel(const HyLatent a, const bf16* __restrict__ q, const int* __restrict__ positions,
+                                                         int n_rows, O* __restrict__ ql, int qld, int nr) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  const int h = blockIdx.y, t0 = blockIdx.z * HM, qd = a.dim + a.rot;
+  if (static_cast<int>(blockIdx.x) == nr) {
+    for (int t = t0; t < min(n_rows, t0 + HM); t += TT) absorb_rotated<bf16, O>(a, q, positions, min(n_rows, t0 + HM), ql, qld, h, t);
+    return;
+  }
+  const int DP = (a.dim + 15) / 16 * 16, lda = DP + 8, ldb = AN + 8, r0 = blockIdx.x * AN;
+  bf16* As = reinterpret_cast<bf16*>(raw);  // [HM][lda]
+  bf16* Bs = As + HM * lda;                 // [DP][ldb]
+  for (int i = threadIdx.x; i < HM * (DP / 8); i += 128) {
+    const int r = i / (DP / 8), c = (i - r * (DP / 8)) * 8;
+    const bool ok = t0 + r < n_rows && c < a.dim;
+    cp_async16(s_u32(As + r * lda + c), q + (ok ? (static_cast<long long>(t0 + r) * a.heads + h) * qd + c : 0), ok ? 16 : 0);
+  }
+  const bf16* w = static_cast<const bf16*>(a.ukv) + static_cast<long long>(h) * a.dim * a.rank;
+  for (int i = threadIdx.x; i < DP * (AN / 8); i += 128) {
+    const int d = i / (AN / 8), c = (i & (AN / 8 - 1)) * 8;
+    const bool ok = d < a.dim && r0 + c < a.rank;
+    cp_async16(s_u32(Bs + d * ldb + c), w + (ok ? static_cast<long long>(d) * a.rank + r0 + c : 0), ok ? 16 : 0);
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wm = warp & 1, wn = warp >> 1;
+  float acc[8][4];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+#pragma unroll 2
+  for (int k0 = 0; k0 < DP; k0 += 16) {
+    uint32_t af[4];
+    ldsm4(s_u32(As + (wm * 16 + (lane & 15)) * lda + k0 + ((lane >> 4) << 3)), af);
+#pragma unroll
+    for (int jp = 0; jp < 4; ++jp) {
+      uint32_t b[4];
+      ldsm4t(s_u32(Bs + (k0 + (lane & 7) + (((lane >> 3) & 1) << 3)) * ldb + wn * 64 + jp * 16 + ((lane >> 4) << 3)), b);
+      mma(acc[2 * jp], af, b[0], b[1]);
+      mma(acc[2 * jp + 1], af, b[2], b[3]);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int r = r0 + wn * 64 + j * 8 + (lane & 3) * 2;
+    if (r >= a.rank) continue;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = t0 + wm * 16 + (lane >> 2) + e * 8;
+      if (t >= n_rows) continue;
+      O* dst = ql + (static_cast<long long>(t) * a.heads + h) * qld + r;
+      dst[0] = from_f<O>(acc[j][2 * e]);
+      dst[1] = from_f<O>(acc[j][2 * e + 1]);
+    }
+  }
+}
+
+// cat[t, h * vdim + v] = sum_r o[t, h, r] W_uv[h * vdim + v, r] over the merged split outputs (ml) or normalised ones.
+__global__ void __launch_bounds__(128) up_mma_kernel(const HyLatent a, const float* __restrict__ o, const float* __restrict__ ml,
+                                                     int splits, int n_rows, bf16* __restrict__ cat, int ldc) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  __shared__ float coef[HM][64];
+  const int h = blockIdx.y, t0 = blockIdx.z * HM, v0 = blockIdx.x * UN, rows = min(HM, n_rows - t0);
+  const int KP = (a.rank + 15) / 16 * 16, ld = KP + 8;
+  bf16* As = reinterpret_cast<bf16*>(raw);  // [HM][ld]
+  bf16* Bs = As + HM * ld;                  // [UN][ld]
+  const bf16* w = static_cast<const bf16*>(a.ukv) + (static_cast<long long>(a.heads) * a.dim + h * a.vdim) * a.rank;
+  for (int i = threadIdx.x; i < UN * (KP / 8); i += 128) {
+    const int v = i / (KP / 8), c = (i - v * (KP / 8)) * 8;
+    const bool ok = v0 + v < a.vdim && c < a.rank;
+    cp_async16(s_u32(Bs + v * ld + c), w + (ok ? static_cast<long long>(v0 + v) * a.rank + c : 0), ok ? 16 : 0);
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (static_cast<int>(threadIdx.x) < HM) {
+    const int b = threadIdx.x;
+    if (b < rows) {
+      float l = 0.f, m = -FLT_MAX;
+      if (ml) {
+        const float* p = ml + (static_cast<long long>(t0 + b) * a.heads + h) * splits * 2;
+        for (int s = 0; s < splits; ++s) m = fmaxf(m, p[2 * s]);
+        for (int s = 0; s < splits; ++s) {
+          const float c = p[2 * s] == -FLT_MAX ? 0.f : exp2f(p[2 * s] - m);
+          coef[b][s] = c;
+          l += c * p[2 * s + 1];
+        }
+        l = l > 0.f ? 1.f / l : 0.f;
+        for (int s = 0; s < splits; ++s) coef[b][s] *= l;
+      } else {
+        coef[b][0] = 1.f;
+      }
+    }
+  }
+  __syncthreads();
+  for (int i = threadIdx.x * 4; i < HM * KP; i += 128 * 4) {
+    const int b = i / KP, r = i - b * KP;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (b < rows && r < a.rank) {
+      const float* p = o + (static_cast<long long>(t0 + b) * a.heads + h) * splits * a.rank + r;
+#pragma unroll 2
+      for (int s = 0; s < splits; ++s) {
+        const float c = coef[b][s];
+        const float4 u = *reinterpret_cast<const float4*>(p + static_cast<long long>(s) * a.rank);
+        v.x += c * u.x; v.y += c * u.y; v.z += c * u.z; v.w += c * u.w;
+      }
+    }
+    const __nv_bfloat162 x = __floats2bfloat162_rn(v.x, v.y), y = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(As + b * ld + r) = make_uint2(*reinterpret_cast<const uint32_t*>(&x), *reinterpret_cast<const uint32_t*>(&y));
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  const int wm = warp & 1, wn = warp >> 1;
+  float acc[2][4];
+#pragma unroll
+  for (int j = 0; j < 2; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+#pragma unroll 4
+  for (int k0 = 0; k0 < KP; k0 += 16) {
+    uint32_t af[4], b[4];
+    ldsm4(s_u32(As + (wm * 16 + (lane & 15)) * ld + k0 + ((lane >> 4) << 3)), af);
+    ldsm4(s_u32(Bs + (wn * 16 + (lane & 7) + ((lane >> 4) << 3)) * ld + k0 + (((lane >> 3) & 1) << 3)), b);
+    mma(acc[0], af, b[0], b[1]);
+    mma(acc[1], af, b[2], b[3]);
+  }
+#pragma unroll
+  for (int j = 0; j < 2; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int v = v0 + wn * 16 + j * 8 + (lane & 3) * 2 + (e & 1), t = wm * 16 + (lane >> 2) + (e >> 1) * 8;
+      if (v < a.vdim && t < rows) cat[static_cast<long long>(t0 + t) * ldc + h * a.vdim + v] = __float2bfloat16(acc[j][e]);
+    }
+}
+
 // ------------------------------------------------------------------------------------------------ materialised form: inputs
 template <typename T>
 __global__ void __launch_bounds__(256) gather_rows_kernel(const HyLatent a, const int4* __restrict__ ranges, T* __restrict__ out) {
@@ -634,8 +773,18 @@ int absorb_t(const HyLatent& a, const void* q, const int* positions, int n, void
     kern<<<dim3(nr + 1, a.heads, (n + TT - 1) / TT), 256, smem, s>>>(a, static_cast<const T*>(q), positions, n, static_cast<O*>(ql), qld, nr);
     return static_cast<int>(cudaGetLastError());
   };
-  if constexpr (sizeof(T) == 2)
+  if constexpr (sizeof(T) == 2) {
+    const int DP = (a.dim + 15) / 16 * 16;
+    const size_t sm = sizeof(bf16) * (HM * (DP + 8) + DP * (AN + 8));
+    if (n > TT && a.rank % 8 == 0 && a.dim % 8 == 0 && a.rot % 8 == 0 && sm <= 200 * 1024 && aligned16<T>(a.ukv, a.rank) && aligned16<T>(q, 8)) {
+      auto kern = absorb_mma_kernel<O>;
+      cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(sm));
+      if (e != cudaSuccess) return static_cast<int>(e);
+      kern<<<dim3(nr + 1, a.heads, (n + HM - 1) / HM), 128, sm, s>>>(a, static_cast<const T*>(q), positions, n, static_cast<O*>(ql), qld, nr);
+      return static_cast<int>(cudaGetLastError());
+    }
     if (a.rank % 8 == 0 && aligned16<T>(a.ukv, a.rank)) return go(absorb_q_kernel<T, O, true>, sizeof(float) * (TT * a.dim + 8 * TT * 128));
+  }
   return go(absorb_q_kernel<T, O, false>, sizeof(float) * TT * a.dim);
 }
 
@@ -652,6 +801,15 @@ int up_rt(const HyLatent& a, const float* o, const float* ml, int splits, int n,
 
 template <typename T>
 int up_t(const HyLatent& a, const float* o, const float* ml, int splits, int n, void* cat, int ldc, cudaStream_t s) {
+  if constexpr (sizeof(T) == 2) {
+    const size_t sm = sizeof(bf16) * (HM + UN) * static_cast<size_t>((a.rank + 15) / 16 * 16 + 8);
+    if (n > TT && a.rank % 8 == 0 && sm <= 200 * 1024 && aligned16<T>(a.ukv, a.rank)) {
+      cudaError_t e = cudaFuncSetAttribute(up_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(sm));
+      if (e != cudaSuccess) return static_cast<int>(e);
+      up_mma_kernel<<<dim3((a.vdim + UN - 1) / UN, a.heads, (n + HM - 1) / HM), 128, sm, s>>>(a, o, ml, splits, n, static_cast<T*>(cat), ldc);
+      return static_cast<int>(cudaGetLastError());
+    }
+  }
   return n <= 2 ? up_rt<T, 1>(a, o, ml, splits, n, cat, ldc, s) : up_rt<T, 4>(a, o, ml, splits, n, cat, ldc, s);
 }
 

@@ -57,7 +57,7 @@ class B200Hybrid(TorchHybrid):
             return F.linear(x, w)
         T, (N, K) = x.shape[0], w.shape
         if K % 8:  # rows the tensor maps cannot describe: the vendor product
-            return F.linear(x, w).to(out_dtype)
+            return torch.mm(x, w.t(), out_dtype=out_dtype) if out_dtype != x.dtype else F.linear(x, w)
         out = torch.empty(T, N, dtype=out_dtype, device=x.device)
         self.launches += 1
         if T <= SMALL_T and N % 16 == 0 and K % 32 == 0 and (T <= 8 or N * K * 2 < (48 << 20)) and x.is_contiguous():

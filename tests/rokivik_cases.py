@@ -30,6 +30,9 @@ CASES = {
     "odd": config([latent(heads=1, dim=10, rot=6, vdim=7, kv_rank=19, q_rank=13, window=1, ff=31), mamba(heads=3, vdim=5, state=7, groups=1, conv=3, norm_groups=3, ff=29),
                    latent(heads=2, dim=9, rot=4, vdim=11, kv_rank=21, q_rank=17, window=13, ff=0), mamba(heads=6, vdim=9, state=33, groups=3, conv=6, norm_groups=1, ff=17)],
                   width=50, vocab=61, side=5, eps=1e-3),
+    # widths the tensor maps take but no vector store does (odd row counts of weights, an odd vocabulary)
+    "ragged": config([latent(heads=3, dim=24, rot=8, vdim=8, kv_rank=40, q_rank=24, window=21, ff=37), mamba(heads=5, vdim=8, state=8, groups=5, norm_groups=5, ff=23),
+                      latent(heads=1, dim=40, rot=16, vdim=72, kv_rank=136, q_rank=8, window=300, ff=0)], width=72, vocab=101, side=16),
     # recurrence only / attention only
     "recurrent": config([mamba(heads=2, vdim=32, state=64, groups=1, norm_groups=1), mamba(conv=2)]),
     "attention": config([latent(window=17), latent(window=40, kv_from=0, scale=0.9)]),
