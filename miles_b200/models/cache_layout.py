@@ -11,7 +11,7 @@ from typing import Optional
 
 import torch
 
-from .layer_plan import Mamba2
+from .layer_plan import Attention, LinearAttention, Mamba2, Parallel
 
 
 @dataclass
@@ -67,21 +67,32 @@ class CacheLayout:
         return out
 
 
+def _mixer_cache(m, dtype: torch.dtype) -> LayerCache:
+    """What one mixer keeps: latent attention one row (latent | rotated key part) per token; softmax attention one row (keys |
+    values) per token; Mamba-2 the last ``conv`` inputs of its convolution as a ring indexed by position (one more than it reads
+    back, so that writing a token's input never touches what is read for it) and the fp32 state ``[heads, vdim, state]``; linear
+    attention the fp32 state ``[heads, vdim, dim]``; two mixers side by side what each of them does."""
+    if isinstance(m, Mamba2):
+        return LayerCache(state=[((m.conv, m.channels), dtype), ((m.heads, m.vdim, m.state), torch.float32)])
+    if isinstance(m, LinearAttention):
+        return LayerCache(state=[((m.heads, m.vdim, m.dim), torch.float32)])
+    if isinstance(m, Attention):
+        return LayerCache(paged=[((m.row_width,), dtype)])
+    if isinstance(m, Parallel):
+        a, b = _mixer_cache(m.left, dtype), _mixer_cache(m.right, dtype)
+        return LayerCache(paged=a.paged + b.paged, state=a.state + b.state)
+    return LayerCache(paged=[((m.latent_width,), dtype)])
+
+
 def cache_layout(cfg, dtype: torch.dtype) -> CacheLayout:
-    """The cache of a model: keys and values per layer, or whatever the mixers of its layer plan keep. Latent attention
-    caches one row (latent | rotated key part) per token; Mamba-2 the last ``conv`` inputs of its convolution as a ring
-    indexed by position (one more than it reads back, so that writing a token's input never touches what is read for it)
-    and the fp32 state ``[heads, vdim, state]``."""
+    """The cache of a model: keys and values per layer, or whatever the mixers of its layer plan keep, one entry per run of a
+    layer (layers that run several times keep something for each pass)."""
     if cfg.plan is None:
         kv = [((cfg.num_kv_heads, cfg.head_dim), dtype)] * 2
         return CacheLayout([LayerCache(paged=kv) for _ in range(cfg.num_layers)])
     layers = []
-    for i, l in enumerate(cfg.plan.layers):
-        m = l.mixer
-        if isinstance(m, Mamba2):
-            layers.append(LayerCache(state=[((m.conv, m.channels), dtype), ((m.heads, m.vdim, m.state), torch.float32)]))
-        elif m.kv_from is not None:
-            layers.append(LayerCache(shares=m.kv_from))
-        else:
-            layers.append(LayerCache(paged=[((m.latent_width,), dtype)]))
+    for i in cfg.plan.runs():
+        m = cfg.plan.layers[i].mixer
+        src = getattr(m, "kv_from", None)
+        layers.append(LayerCache(shares=src) if src is not None else _mixer_cache(m, dtype))
     return CacheLayout(layers)

@@ -12,7 +12,8 @@ from dataclasses import asdict, dataclass, field
 from pathlib import Path
 from typing import Any, Optional
 
-from .layer_plan import DESIGNS, DenseFF, LatentAttention, Layer, LayerPlan, Mamba2, Rotary, plan_specs, read_plan, write_plan
+from .layer_plan import (DESIGNS, Attention, DenseFF, LatentAttention, Layer, LayerPlan, LinearAttention, Mamba2, Parallel, Rotary, checkpoint_shapes,
+                         plan_specs, read_plan, write_plan)
 
 
 @dataclass
@@ -192,13 +193,16 @@ class ModelConfig:
 
     @classmethod
     def from_hf_config(cls, cfg: dict | str | Path, name: str | None = None) -> "ModelConfig":
+        shapes = None
         if not isinstance(cfg, dict):
             p = Path(cfg)
             if p.is_dir():
                 p = p / "config.json"
             cfg = json.loads(p.read_text())
+            if cfg.get("architecture") in DESIGNS:
+                shapes = checkpoint_shapes(p.parent)
         if cfg.get("architecture") in DESIGNS:
-            return cls.from_plan(*read_plan(cfg), name=name)
+            return cls.from_plan(*read_plan(cfg, shapes), name=name)
         arch = (cfg.get("architectures") or ["Qwen3ForCausalLM"])[0]
         heads = cfg["num_attention_heads"]
         head_dim = cfg.get("head_dim") or cfg["hidden_size"] // heads
@@ -436,7 +440,21 @@ def _rokivik_smoke() -> ModelConfig:
     return ModelConfig.from_plan(plan, 4096, 384, name="rokivik-smoke")
 
 
+def _pesanex_smoke() -> ModelConfig:
+    """A small Pesanex: every mixer, layers with and without a feed-forward, the middle two run three times."""
+    rot = Rotary(base=1e5, dims=24, interleaved=False)
+    gla = dict(tau=8.0, norm_weight=True)
+    layers = [Layer(LinearAttention(heads=4, dim=40, vdim=64, rank=16, **gla)),
+              Layer(LinearAttention(heads=3, dim=64, vdim=96, decay=[0.9, 0.98, 0.998], rotary=rot, scale_keys=True, kind="retention"), DenseFF(640, act="relu")),
+              Layer(Parallel(Attention(heads=8, kv_heads=2, dim=48, vdim=32, scale=0.2, rotary=rot, unit_qk=True, sink=True),
+                             LinearAttention(heads=4, dim=32, vdim=64, rank=16, **gla)), DenseFF(896, act="relu"))]
+    plan = LayerPlan("Pesanex", layers, norm="layer_norm", eps=1e-5, parallel=False, loop=(1, 3, 3))
+    plan.validate()
+    return ModelConfig.from_plan(plan, 4096, 320, name="pesanex-smoke")
+
+
 PRESETS["rokivik-smoke"] = _rokivik_smoke()
+PRESETS["pesanex-smoke"] = _pesanex_smoke()
 
 
 def get_config(name: str) -> ModelConfig:

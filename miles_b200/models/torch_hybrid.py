@@ -16,7 +16,7 @@ import torch.nn.functional as F
 from ..ops import reference as R
 from .cache_layout import cache_layout
 from .config import ModelConfig
-from .layer_plan import Mamba2
+from .layer_plan import Mamba2, Parallel
 from .params import ParamStore
 from .torch_impl import InferMeta
 
@@ -27,8 +27,9 @@ class TorchHybrid:
         self.cfg, self.plan, self.store = cfg, cfg.plan, store
         self.dev = store.device
         self.in_segs = [{s.name: s for s in l.in_segments()} for l in cfg.plan.layers]
-        self.out_segs = [{s.name: s for s in l.out_segments()} for l in cfg.plan.layers]
-        self.capture: Optional[list] = None   # a list: receives the residual stream after every layer
+        self.out_segs = [{s.name: s for s in l.out_segments()} if l.parallel else {} for l in cfg.plan.layers]
+        self.runs = cfg.plan.runs()
+        self.capture: Optional[list] = None   # a list: receives the residual stream after every layer run
 
     # ------------------------------------------------------------------ pieces
     def linear(self, x, w):
@@ -36,7 +37,13 @@ class TorchHybrid:
 
     def _norm(self, x, name):
         P = self.store.params
+        if self.plan.norm == "layer_norm":
+            return R.layer_norm(x, P[name + ".weight"], self.plan.eps).to(self.store.dtype)
         return R.dynamic_tanh(x, P[name + ".weight"], P[name + ".bias"], P[name + ".alpha"]).to(self.store.dtype)
+
+    def _part(self, i, proj, name):
+        s = self.in_segs[i]["mix." + name]
+        return proj[:, s.start:s.start + s.size]
 
     def _sequences(self, meta: InferMeta, n_rows: int):
         """(first row, rows, cached tokens, pages, state slot) of every sequence of the pass."""
@@ -72,12 +79,8 @@ class TorchHybrid:
 
     def _latent_attention(self, i, proj, positions, meta, cache):
         m, P, p = self.plan.layers[i].mixer, self.store.params, f"layers.{i}.mix."
-        segs, eps, rows = self.in_segs[i], self.plan.eps, cache[0]
-
-        def part(name):
-            s = segs["mix." + name]
-            return proj[:, s.start:s.start + s.size]
-
+        eps, rows = self.plan.eps, cache[0]
+        part = lambda name: self._part(i, proj, name)
         cq = (R.unit_rms(part("dq").float(), eps) * P[p + "q_norm.weight"].float()).to(proj.dtype)
         q = self.linear(cq, P[p + "uq.weight"]).view(-1, m.heads, m.dim + m.rot_dim)
         qn, qr = q[..., :m.dim], R.rotate_pairs(q[..., m.dim:], positions, m.rotary.base)
@@ -102,6 +105,81 @@ class TorchHybrid:
             a = torch.softmax(s.masked_fill(~seen, float("-inf")), -1)
             outs.append(torch.einsum("hij,jhd->ihd", a, v.float()).reshape(n, -1).to(proj.dtype))
         return torch.cat(outs)
+
+    def _attention(self, i, m, pre, proj, positions, meta, rows):
+        """Softmax attention over cached key / value heads; ``pre``: name of the side the mixer is on."""
+        T, dt = proj.shape[0], proj.dtype
+        sink = self.store.params[f"layers.{i}.mix.{pre}sink"].float() if m.sink else None
+
+        def turned(x):
+            x = R.rotate_halves(x, positions, m.rotary.base, m.rotary.dims) if m.rotary is not None else x.float()
+            return (R.unit_rms(x, self.plan.eps) if m.unit_qk else x).to(dt)
+
+        q = turned(self._part(i, proj, pre + "q").reshape(T, m.heads, m.dim))
+        k = turned(self._part(i, proj, pre + "k").reshape(T, m.kv_heads, m.dim))
+        new = torch.cat([k.reshape(T, -1), self._part(i, proj, pre + "v")], 1)
+        rows[meta.slot_mapping.long(), :new.shape[1]] = new.to(rows.dtype)
+        ps, outs, rep, nk = meta.page_size, [], m.heads // m.kv_heads, m.kv_heads * m.dim
+        for r0, n, ctx, pages, _ in self._sequences(meta, T):
+            at = torch.arange(ctx + n, device=proj.device)
+            kv = rows[pages[at // ps] * ps + at % ps].float()
+            kk = kv[:, :nk].view(-1, m.kv_heads, m.dim).repeat_interleave(rep, 1)
+            vv = kv[:, nk:nk + m.kv_heads * m.vdim].view(-1, m.kv_heads, m.vdim).repeat_interleave(rep, 1)
+            s = torch.einsum("ihd,jhd->hij", q[r0:r0 + n].float(), kk) * m.scale
+            s = s.masked_fill(at[None, :] > torch.arange(ctx, ctx + n, device=proj.device)[:, None], float("-inf"))
+            outs.append(torch.einsum("hij,jhd->ihd", R.sink_softmax(s, sink), vv).reshape(n, -1).to(dt))
+        return torch.cat(outs)
+
+    def _linear_attention(self, i, m, pre, proj, positions, meta, states):
+        P, p, T = self.store.params, f"layers.{i}.mix.{pre}", proj.shape[0]
+        q, k, v, g = (self._part(i, proj, pre + n) for n in ("q", "k", "v", "g"))
+        q, k, v = q.reshape(T, m.heads, m.dim).float(), k.reshape(T, m.heads, m.dim).float(), v.reshape(T, m.heads, m.vdim).float()
+        if m.rotary is not None:
+            q, k = (R.rotate_halves(x, positions, m.rotary.base, m.rotary.dims) for x in (q, k))
+        if m.scale_keys:
+            k = k * m.dim ** -0.5
+        else:
+            q = q * m.dim ** -0.5
+        if m.rank:
+            z = F.linear(self._part(i, proj, pre + "a1").float(), P[p + "a2.weight"].float()) + P[p + "a2.bias"].float()
+            decay = (F.logsigmoid(z) / m.tau).view(T, m.heads, m.dim)
+        else:
+            decay = torch.tensor(m.decay, dtype=torch.float64, device=proj.device).log().float().view(1, -1, 1)
+        outs = []
+        for r0, n, ctx, _, slot in self._sequences(meta, T):
+            S = states[slot].clone() if ctx > 0 else torch.zeros_like(states[slot])
+            at = slice(r0, r0 + n)
+            o, states[slot] = R.linear_attention_scan(q[at], k[at], v[at], decay[at] if m.rank else decay, S)
+            outs.append(o)
+        o = R.unit_rms(torch.cat(outs), self.plan.eps)
+        if m.norm_weight:
+            o = o * P[p + "norm.weight"].float()
+        return (o.reshape(T, -1) * F.silu(g.float())).to(proj.dtype)
+
+    def _project_out(self, w, y):
+        """A product whose matrix has padding columns."""
+        return self.linear(F.pad(y, (0, w.shape[1] - y.shape[1])), w).float()
+
+    def _sequential_layer(self, i, x, positions, meta, cache):
+        """``x + norm(mixer(norm(x)))``, then the same around the feed-forward."""
+        l, P, p = self.plan.layers[i], self.store.params, f"layers.{i}."
+        m, eps = l.mixer, self.plan.eps
+        proj = self.linear(self._norm(x, p + "norm1"), P[p + "in.weight"])
+        if isinstance(m, Parallel):
+            a = self._attention(i, m.left, "left.", proj, positions, meta, cache[0])
+            b = self._linear_attention(i, m.right, "right.", proj, positions, meta, cache[1])
+            y = sum(R.unit_rms(self._project_out(P[p + f"{s}.o.weight"], o), eps) * P[p + f"mix.{s}.out_norm.weight"].float()
+                    for s, o in (("left", a), ("right", b))) / 2
+        else:
+            y = self._project_out(P[p + "o.weight"], self._linear_attention(i, m, "", proj, positions, meta, cache[0]))
+        x = x + R.layer_norm(y, P[p + "norm1b.weight"], eps)
+        if l.ff is not None:
+            s = {s.name: s for s in l.ff_segments()}
+            z = self.linear(self._norm(x, p + "norm2"), P[p + "ff_in.weight"])
+            g, u = (z[:, s[n].start:s[n].start + l.ff.ff] for n in ("mlp.gate", "mlp.up"))
+            y = self._project_out(P[p + "ff_out.weight"], (F.relu(g) if l.ff.act == "relu" else F.silu(g)) * u)
+            x = x + R.layer_norm(y, P[p + "norm2b.weight"], eps)
+        return x
 
     def _layer(self, i, x, h, tokens, positions, meta, cache):
         l, P, p = self.plan.layers[i], self.store.params, f"layers.{i}."
@@ -145,8 +223,11 @@ class TorchHybrid:
             meta, kv_cache = self.scratch_cache(cu_seqlens)
         P = self.store.params
         x = P["embed.weight"][tokens.long()].float()
-        for i in range(self.cfg.num_layers):
-            x = self._layer(i, x, self._norm(x, f"layers.{i}.norm1"), tokens, positions, meta, kv_cache[i])
+        for i, cache in zip(self.runs, kv_cache):
+            if self.plan.parallel:
+                x = self._layer(i, x, self._norm(x, f"layers.{i}.norm1"), tokens, positions, meta, cache)
+            else:
+                x = self._sequential_layer(i, x, positions, meta, cache)
             if self.capture is not None:
                 self.capture.append(x.clone())
         return self._norm(x, "final_norm")

@@ -299,6 +299,11 @@ def dynamic_tanh(x, weight, bias, alpha):
     return torch.tanh(alpha.float() * x.float()) * weight.float() + bias.float()
 
 
+def layer_norm(x, weight, eps: float):
+    """Layer norm with a weight and no bias, in fp32."""
+    return F.layer_norm(x.float(), x.shape[-1:], weight.float(), None, eps)
+
+
 def unit_rms(x, eps: float):
     return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
 
@@ -315,6 +320,34 @@ def rotate_pairs(x, positions, base: float):
     u, v = x[..., 0::2].float(), x[..., 1::2].float()
     c, s = torch.cos(a), torch.sin(a)
     return torch.stack((u * c - v * s, v * c + u * s), -1).flatten(-2).to(x.dtype)
+
+
+def rotate_halves(x, positions, base: float, dims: int):
+    """Rotary embedding of the first ``dims`` dimensions of ``x`` [T, heads, dim], dimension k paired with k + dims / 2; angles and
+    result in fp32."""
+    a = positions.float()[:, None, None] * pair_frequencies(dims, base, x.device)
+    u, v, rest = x.float().split([dims // 2, dims // 2, x.shape[-1] - dims], -1)
+    c, s = torch.cos(a), torch.sin(a)
+    return torch.cat((u * c - v * s, v * c + u * s, rest), -1)
+
+
+def linear_attention_scan(q, k, v, log_decay, state):
+    """``S <- S exp(log_decay) + v k^T`` and ``o = S q`` over one sequence: ``q`` / ``k`` [T, H, N], ``v`` [T, H, P], ``log_decay``
+    [T or 1, H, N or 1] natural, ``state`` [H, P, N]; fp32. Returns (o [T, H, P], state after the last token)."""
+    keep = torch.exp(log_decay)
+    os = []
+    for t in range(q.shape[0]):
+        state = state * keep[min(t, keep.shape[0] - 1)][:, None, :] + v[t][:, :, None] * k[t][:, None, :]
+        os.append((state * q[t][:, None, :]).sum(-1))
+    return torch.stack(os), state
+
+
+def sink_softmax(s, sink=None):
+    """Softmax over the last dimension of ``s`` [H, T, J] whose denominator also contains ``exp(sink_h)``."""
+    if sink is None:
+        return torch.softmax(s, -1)
+    full = torch.cat((s, sink.to(s.dtype).view(-1, 1, 1).expand(-1, s.shape[1], 1)), -1)
+    return torch.softmax(full, -1)[..., :-1]
 
 
 def causal_conv_silu(x, weight, bias):
