@@ -21,7 +21,8 @@ OBJ = CSRC / "build"
 TARGET = PKG / "_C.so"
 # planned-layer models load only this library, so serving one compiles a handful of files
 HYBRID_TARGET = PKG / "_hybrid.so"
-HYBRID_ONLY = {"hybrid_ops.cu", "mamba2.cu", "latent_attention.cu", "latent_prefill.cu", "hybrid_bindings.cpp"}
+HYBRID_ONLY = {"hybrid_ops.cu", "mamba2.cu", "latent_attention.cu", "cached_attention.cu", "cached_prefill.cu", "linear_attention.cu",
+               "sequential_ops.cu", "hybrid_bindings.cpp"}
 HYBRID_SHARED = {"gemm.cu", "decode_small.cu", "decode_stream.cu", "sampling.cu", "serve_bindings.cpp"}
 TARGETS = {"_C": TARGET, "_hybrid": HYBRID_TARGET}
 

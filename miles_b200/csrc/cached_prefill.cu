@@ -1,13 +1,13 @@
-// Prompt attention of latent-attention layers on tcgen05: causal with an optional sliding window, over keys and values that
-// were projected from the cached latents of the visible range.
+// Prompt attention over gathered cache rows on tcgen05: causal, with an optional sliding window and an optional sink per head.
 //
 // Same pipeline as attention_fwd.cu (TMA producer warp, MMA issuer warp, two softmax threads per query row, scores double
 // buffered and the output accumulated in TMEM); what differs:
-//   * a key is two parts: dim values of the head's own (64-column boxes of the key / value product) and rot values shared by
-//     all heads (a box of the latent rows). The score product runs over both, queries carry zeros where a box reaches past
-//     its part, so neither part is copied next to the other;
+//   * keys and values are column ranges of the rows they come from, wherever these are: a key head's own 64-column boxes, and
+//     (SHARED, latent attention) one more box of other rows that all heads have in common. The score product runs over both,
+//     queries carry zeros where a box reaches past its part, so that nothing is copied next to anything;
 //   * queries see keys in (position - window, position]: a tile starts at the first block its first query sees;
-//   * value width and key width differ, and the output goes straight into the layer's fused output row.
+//   * value width and key width differ, and the output goes straight into the rows of the product that follows;
+//   * a sink is one more term of the denominator: it enters once, at the end.
 #include <cuda.h>
 #include <float.h>
 #include <stdio.h>
@@ -28,7 +28,10 @@ constexpr int LP_THREADS = 320;
 
 struct LpArgs {
   const int4* tiles;
-  int heads, dim, vdim, rank, window;
+  int heads, group, vdim, window;
+  int k_col, k_step, v_col, v_step;  // columns of key head g: k_col + g * k_step ..
+  int shared_col;                    // of the part all heads share, in its own rows
+  const __nv_bfloat16* sink;
   __nv_bfloat16* out;
   int ldc;
   float scale_log2;
@@ -42,19 +45,19 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
-template <int NN, int NV>
+template <int NN, int NV, bool SHARED>
 struct Lp {
-  static constexpr int KA = NN + 1;               // 64-column atoms of a key: NN own, one shared
-  static constexpr int VST = NN == 1 ? 2 : 1;     // value stages (one where keys take the room; its load hides behind the softmax)
+  static constexpr int KA = NN + (SHARED ? 1 : 0);  // 64-column atoms of a key: NN own, one shared
+  static constexpr int VST = KA <= 2 ? 2 : 1;       // value stages (one where keys take the room; its load hides behind the softmax)
   static constexpr int Q_BYTES = KA * ATOM, P_BYTES = 2 * ATOM, K_BYTES = KA * ATOM, V_BYTES = NV * ATOM;
   static constexpr int SMEM = Q_BYTES + P_BYTES + 2 * K_BYTES + VST * V_BYTES + 256 + 1024;
 };
 
-template <int NN, int NV>
+template <int NN, int NV, bool SHARED>
 __global__ void __launch_bounds__(LP_THREADS, 1)
-latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
+cached_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                       const __grid_constant__ CUtensorMap map_c, const LpArgs p) {
-  using L = Lp<NN, NV>;
+  using L = Lp<NN, NV, SHARED>;
   constexpr int VST = L::VST;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -94,7 +97,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     fence_barrier_init();
     prefetch_tensormap(&map_q);
     prefetch_tensormap(&map_kv);
-    prefetch_tensormap(&map_c);
+    if (SHARED) prefetch_tensormap(&map_c);
   }
   if (warp == 1) {
     tmem_alloc(tmem_slot, 512);
@@ -116,6 +119,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
       bool ok = true;
+      const int g = head / p.group, k_col = p.k_col + g * p.k_step, v_col = p.v_col + g * p.v_step;
       mbar_expect_tx(BAR(B_QF), L::Q_BYTES);
 #pragma unroll
       for (int i = 0; i < L::KA; ++i) tma_load_2d(q_s + i * ATOM, &map_q, BAR(B_QF), (head * L::KA + i) * 64, q_row0);
@@ -125,8 +129,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         mbar_expect_tx(BAR(B_KF + st), L::K_BYTES);
         const uint32_t dst = k_s + st * L::K_BYTES;
 #pragma unroll
-        for (int i = 0; i < NN; ++i) tma_load_2d(dst + i * ATOM, &map_kv, BAR(B_KF + st), head * p.dim + i * 64, row);
-        tma_load_2d(dst + NN * ATOM, &map_c, BAR(B_KF + st), p.rank, row);
+        for (int i = 0; i < NN; ++i) tma_load_2d(dst + i * ATOM, &map_kv, BAR(B_KF + st), k_col + i * 64, row);
+        if (SHARED) tma_load_2d(dst + NN * ATOM, &map_c, BAR(B_KF + st), p.shared_col, row);
         return true;
       };
       auto load_v = [&](int j) -> bool {
@@ -136,7 +140,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         const uint32_t dst = v_s + st * L::V_BYTES;
 #pragma unroll
         for (int i = 0; i < NV; ++i)
-          tma_load_2d(dst + i * ATOM, &map_kv, BAR(B_VF + st), p.heads * p.dim + head * p.vdim + i * 64, row);
+          tma_load_2d(dst + i * ATOM, &map_kv, BAR(B_VF + st), v_col + i * 64, row);
         return true;
       };
       ok = load_k(0);
@@ -309,7 +313,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       if (lane == 0) mbar_arrive(pair_bar);
       ok = mbar_wait(pair_bar, n_blocks & 1, abort_flag, p.status, ERR_WAIT_PEER);
       if (ok) {
-        const float l_tot = l + xch[b][half ^ 1][row];
+        float l_tot = l + xch[b][half ^ 1][row];
+        if (p.sink) l_tot += ex2(__bfloat162float(p.sink[head]) * 1.4426950408889634f - m_used);
         const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
         const bool live = row < q_rows;
         __nv_bfloat16* dst = p.out + static_cast<long long>(q_row0 + row) * p.ldc + head * p.vdim + half * OC;
@@ -377,10 +382,10 @@ int lp_map(CUtensorMap* map, const void* ptr, long long rows, long long cols, lo
   return 0;
 }
 
-template <int NN, int NV>
+template <int NN, int NV, bool SHARED>
 int lp_launch(const CUtensorMap& mq, const CUtensorMap& mkv, const CUtensorMap& mc, const LpArgs& a, int n_tiles, cudaStream_t s) {
-  auto kern = latent_prefill_kernel<NN, NV>;
-  constexpr int smem = Lp<NN, NV>::SMEM;
+  auto kern = cached_prefill_kernel<NN, NV, SHARED>;
+  constexpr int smem = Lp<NN, NV, SHARED>::SMEM;
   static_assert(smem <= 227 * 1024, "shared memory of the prompt attention kernel");
   if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
     return lp_fail("cudaFuncSetAttribute(MaxDynamicSharedMemorySize) failed for prompt attention");
@@ -389,40 +394,50 @@ int lp_launch(const CUtensorMap& mq, const CUtensorMap& mkv, const CUtensorMap& 
   return 0;
 }
 
+template <bool SHARED>
+int lp_pick(int q_pad, const CUtensorMap& mq, const CUtensorMap& mkv, const CUtensorMap& mc, const LpArgs& p, int n_tiles, cudaStream_t s) {
+  if (q_pad == 64) return p.vdim <= 64 ? lp_launch<1, 1, SHARED>(mq, mkv, mc, p, n_tiles, s) : lp_launch<1, 2, SHARED>(mq, mkv, mc, p, n_tiles, s);
+  return p.vdim <= 64 ? lp_launch<2, 1, SHARED>(mq, mkv, mc, p, n_tiles, s) : lp_launch<2, 2, SHARED>(mq, mkv, mc, p, n_tiles, s);
+}
+
 }  // namespace
 
 const char* hy_prefill_last_error() { return g_lp_err.c_str(); }
 
 bool hy_prefill_supported(int dim, int rot, int vdim, int rank, int width) {
   // every box starts at a column that is a multiple of 8 (16 bytes)
-  return dim % 8 == 0 && vdim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && width % 8 == 0 && dim >= 8 && dim <= 128 && rot >= 8 &&
+  return dim % 8 == 0 && vdim % 8 == 0 && rot % 8 == 0 && rank % 8 == 0 && width % 8 == 0 && dim >= 8 && dim <= 128 && rot >= 0 &&
          rot <= 64 && vdim >= 8 && vdim <= 128;
 }
 
-int hy_latent_prefill(const HyLatent& a, const void* q, int nope_pad, const void* kv, long long kv_ld, const void* latent,
-                      long long ctx_rows, const int* tiles, int n_tiles, int T, void* out, int ldc, cudaStream_t s) {
-  if (!hy_prefill_supported(a.dim, a.rot, a.vdim, a.rank, a.width)) return lp_fail("head sizes are not supported by the tensor-core prompt attention");
-  if ((nope_pad != 64 && nope_pad != 128) || nope_pad < a.dim) return lp_fail("queries must be padded to 64 or 128 columns");
+int hy_prefill(const HyPrefill& a, const int* tiles, int n_tiles, int T, void* out, int ldc, cudaStream_t s) {
+  const bool shared = a.shared != nullptr;
+  if (!hy_prefill_supported(a.dim, shared ? a.rot : 0, a.vdim, a.shared_col, shared ? a.shared_width : 0) ||
+      (a.k_col | a.k_step | a.v_col | a.v_step) % 8 != 0 || (shared && a.rot < 8))
+    return lp_fail("head sizes are not supported by the tensor-core prompt attention");
+  if ((a.q_pad != 64 && a.q_pad != 128) || a.q_pad < a.dim) return lp_fail("queries must be padded to 64 or 128 columns");
   if (ldc % 8 != 0 || (reinterpret_cast<uintptr_t>(out) & 15) != 0) return lp_fail("the output rows must be 16-byte aligned");
   if (n_tiles == 0) return 0;
   CUtensorMap mq, mkv, mc;
-  const long long qw = static_cast<long long>(a.heads) * (nope_pad + 64);
-  if (lp_map(&mq, q, T, qw, qw)) return -1;
-  if (lp_map(&mkv, kv, ctx_rows, static_cast<long long>(a.heads) * (a.dim + a.vdim), kv_ld)) return -1;
-  if (lp_map(&mc, latent, ctx_rows, a.width, a.width)) return -1;
+  const long long qw = static_cast<long long>(a.heads) * (a.q_pad + (shared ? 64 : 0));
+  if (lp_map(&mq, a.q, T, qw, qw)) return -1;
+  if (lp_map(&mkv, a.kv, a.ctx_rows, a.kv_cols, a.kv_ld)) return -1;
+  mc = mkv;
+  if (shared && lp_map(&mc, a.shared, a.ctx_rows, a.shared_width, a.shared_width)) return -1;
   LpArgs p;
   p.tiles = reinterpret_cast<const int4*>(tiles);
   p.heads = a.heads;
-  p.dim = a.dim;
+  p.group = a.group;
   p.vdim = a.vdim;
-  p.rank = a.rank;
   p.window = a.window;
+  p.k_col = a.k_col; p.k_step = a.k_step; p.v_col = a.v_col; p.v_step = a.v_step;
+  p.shared_col = a.shared_col;
+  p.sink = static_cast<const __nv_bfloat16*>(a.sink);
   p.out = static_cast<__nv_bfloat16*>(out);
   p.ldc = ldc;
   p.scale_log2 = a.scale * 1.4426950408889634f;
   p.status = a.status;
-  if (nope_pad == 64) return a.vdim <= 64 ? lp_launch<1, 1>(mq, mkv, mc, p, n_tiles, s) : lp_launch<1, 2>(mq, mkv, mc, p, n_tiles, s);
-  return a.vdim <= 64 ? lp_launch<2, 1>(mq, mkv, mc, p, n_tiles, s) : lp_launch<2, 2>(mq, mkv, mc, p, n_tiles, s);
+  return shared ? lp_pick<true>(a.q_pad, mq, mkv, mc, p, n_tiles, s) : lp_pick<false>(a.q_pad, mq, mkv, mc, p, n_tiles, s);
 }
 
 }  // namespace mb

@@ -83,6 +83,15 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
+// State row of a sequence; one outside the cache is reported and not followed (-1: the sequence starts from nothing and its state
+// is not kept).
+__device__ __forceinline__ long long state_row(const int* slots, int sequences, int seq, int* status) {
+  const int slot = slots[seq];
+  if (slot >= 0 && slot < sequences) return slot;
+  if (status) atomicCAS(status, 0, 11);
+  return -1;
+}
+
 template <typename T>
 inline bool aligned16(const void* p, long long stride_elems) {
   return (reinterpret_cast<uintptr_t>(p) & 15) == 0 && (stride_elems * static_cast<long long>(sizeof(T))) % 16 == 0;

@@ -5,14 +5,14 @@
 //  * absorbed: queries are taken into latent space (W_uk^T q), scores and outputs are products with the cached rows
 //    themselves, all heads of a token reading the same bytes; W_uv brings the result back. Decoding uses it: the cache is
 //    the only thing that grows with the context, and it is read once for all heads.
-//  * materialised (latent_prefill.cu): keys and values of the visible range are projected once, which needs far fewer
+//  * materialised (cached_prefill.cu): keys and values of the visible range are projected once, which needs far fewer
 //    operations when many queries share them. Prompts use it.
-// This file has the absorbed form (tensor-core decode kernel, and a plain kernel for any sizes and for 32-bit), the query /
-// output projections around it, and the row gather and query layout the materialised form starts from.
+// This file has the query / output projections around the absorbed form (whose kernels are those of cached_attention.cu) and the
+// query layout of the materialised one.
 #include <float.h>
 
 #include "hybrid.h"
-#include "hybrid_common.cuh"
+#include "hybrid_mma.cuh"
 
 namespace mb {
 namespace {
@@ -20,14 +20,6 @@ namespace {
 using namespace hy;
 
 constexpr int TT = 8;  // rows that share the weight reads of a projection block
-
-__device__ __forceinline__ long long row_slot(const HyLatent& a, int seq, int pos) {
-  const int pg = pos / a.page_size;
-  if (pg >= a.max_pages) return -1;
-  const long long page = a.table[static_cast<long long>(seq) * a.max_pages + pg];
-  const long long slot = page * a.page_size + pos % a.page_size;
-  return (page < 0 || slot >= a.num_slots) ? -1 : slot;
-}
 
 // ------------------------------------------------------------------------------------------------ projections
 // Rotated part and padding of row t, head h (all threads of the block, rows t0 .. t0 + TT).
@@ -274,310 +266,6 @@ __global__ void __launch_bounds__(256) latent_up_kernel(const HyLatent a, const 
     }
 }
 
-// ------------------------------------------------------------------------------------------------ plain attention
-// CTA = (head, row); 4 warps stride over the visible keys, each with its own running softmax; NR * 32 >= rank.
-template <typename T, int NR>
-__global__ void __launch_bounds__(128) attend_kernel(const HyLatent a, const float* __restrict__ ql, int qld,
-                                                     const int* __restrict__ positions, const int* __restrict__ row_seq,
-                                                     float* __restrict__ out) {
-  extern __shared__ float sm[];  // query [rank + rot]; later the warps' outputs [4][rank]
-  __shared__ float wm[4], wl[4];
-  const int h = blockIdx.x, t = blockIdx.y, K = a.rank + a.rot;
-  const int seq = row_seq ? row_seq[t] : t, pos = positions[t];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const float* qr = ql + (static_cast<long long>(t) * a.heads + h) * qld;
-  for (int i = threadIdx.x; i < K; i += blockDim.x) sm[i] = qr[i];
-  __syncthreads();
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-  float m = -FLT_MAX, l = 0.f, o[NR];
-#pragma unroll
-  for (int i = 0; i < NR; ++i) o[i] = 0.f;
-  for (int j = lo + warp; j <= pos; j += 4) {
-    const long long slot = row_slot(a, seq, j);
-    if (slot < 0) {
-      if (lane == 0 && a.status) atomicCAS(a.status, 0, 9);
-      continue;
-    }
-    const T* row = static_cast<const T*>(a.rows) + slot * a.width;
-    float c[NR], s = 0.f;
-#pragma unroll
-    for (int i = 0; i < NR; ++i) {
-      const int k = lane + 32 * i;
-      c[i] = k < a.rank ? to_f(row[k]) : 0.f;
-      if (k < a.rank) s += c[i] * sm[k];
-    }
-    for (int k = a.rank + lane; k < K; k += 32) s += to_f(row[k]) * sm[k];
-    s = warp_sum(s) * a.scale;
-    const float mn = fmaxf(m, s);
-    const float corr = m == -FLT_MAX ? 0.f : expf(m - mn), p = expf(s - mn);
-    l = l * corr + p;
-    m = mn;
-#pragma unroll
-    for (int i = 0; i < NR; ++i) o[i] = o[i] * corr + p * c[i];
-  }
-  __syncthreads();
-#pragma unroll
-  for (int i = 0; i < NR; ++i)
-    if (lane + 32 * i < a.rank) sm[warp * a.rank + lane + 32 * i] = o[i];
-  if (lane == 0) {
-    wm[warp] = m;
-    wl[warp] = l;
-  }
-  __syncthreads();
-  float gm = -FLT_MAX, gl = 0.f, c[4];
-#pragma unroll
-  for (int w = 0; w < 4; ++w) gm = fmaxf(gm, wm[w]);
-#pragma unroll
-  for (int w = 0; w < 4; ++w) {
-    c[w] = wm[w] == -FLT_MAX ? 0.f : expf(wm[w] - gm);
-    gl += c[w] * wl[w];
-  }
-  const float inv = gl > 0.f ? 1.f / gl : 0.f;
-  for (int i = threadIdx.x; i < a.rank; i += blockDim.x) {
-    float v = 0.f;
-#pragma unroll
-    for (int w = 0; w < 4; ++w) v += c[w] * sm[w * a.rank + i];
-    out[(static_cast<long long>(t) * a.heads + h) * a.rank + i] = v * inv;
-  }
-}
-
-// ------------------------------------------------------------------------------------------------ tensor-core decode
-constexpr int DW = 8;     // warps
-constexpr int TOK = 64;   // tokens per stage
-constexpr int PLD = TOK + 8;
-
-__device__ __forceinline__ uint32_t s_u32(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, int bytes) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
-__host__ __device__ inline int decode_k(int rank, int rot) { return (rank + rot + 31) / 32 * 32; }
-
-// CTA = (sequence, group of MT * 16 heads, split). Warp (wm, wt): head tile wm; scores of the wt-th token group, outputs of the
-// wt-th group of latent columns. Rows of a stage are read from the cache once for all heads of the group; queries stay in
-// registers (as far as they fit: the first QI chunks of 32), so that shared memory carries little more than the rows.
-template <int MT>
-__global__ void __launch_bounds__(DW * 32) latent_decode_kernel(const HyLatent a, const bf16* __restrict__ ql, int qld,
-                                                                const int* __restrict__ seq_lens, int splits,
-                                                                float* __restrict__ po, float* __restrict__ pml) {
-  constexpr int NG = DW / MT;           // token groups, column groups
-  constexpr int KI = 18;                // 32-wide chunks of a query at most (576 values)
-  constexpr int QI = MT == 1 ? 18 : 10; // of which in registers
-  constexpr int NTM = 8 * MT;           // 8-wide output tiles per warp at most (512 columns over NG warps)
-  extern __shared__ __align__(16) unsigned char raw[];
-  __shared__ int slot_s[2][TOK];
-  const int KP = decode_k(a.rank, a.rot), ld = KP + 8;
-  bf16* Ks = reinterpret_cast<bf16*>(raw);             // [2][TOK][ld]
-  bf16* Qs = Ks + 2 * TOK * ld;                        // [MT * 16][ld]
-  bf16* Ps = Qs + MT * 16 * ld;                        // [MT * 16][PLD]
-  float* wmax = reinterpret_cast<float*>(Ps + MT * 16 * PLD);  // [NG][MT * 16]
-  float* wsum = wmax + DW * MT * 16;                   // [NG][MT * 16]
-  const int b = blockIdx.x, h0 = blockIdx.y * MT * 16, split = blockIdx.z;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int wm = warp % MT, wt = warp / MT;
-  int len = seq_lens[b];
-  const long long cap = static_cast<long long>(a.max_pages) * a.page_size;
-  if (len < 0 || len > cap) {
-    if (threadIdx.x == 0 && a.status) atomicCAS(a.status, 0, 8);
-    len = len < 0 ? 0 : static_cast<int>(cap);
-  }
-  const int lo = a.window > 0 ? max(0, len - a.window) : 0;
-  int per = (len - lo + splits - 1) / splits;
-  per = (per + TOK - 1) / TOK * TOK;
-  const int t_lo = min(len, lo + split * per), t_hi = min(len, t_lo + per);
-  const int n_ch = (t_hi - t_lo + TOK - 1) / TOK;
-  const int chunks = KP / 8, wchunks = a.width / 8;
-
-  auto find_slots = [&](int ch) {  // by the first TOK threads, a barrier before they are used
-    if (threadIdx.x >= TOK || ch >= n_ch) return;
-    const int t = t_lo + ch * TOK + static_cast<int>(threadIdx.x);
-    long long slot = -1;
-    if (t < t_hi) {
-      slot = row_slot(a, b, t);
-      if (slot < 0 && a.status) atomicCAS(a.status, 0, 9);
-    }
-    slot_s[ch & 1][threadIdx.x] = static_cast<int>(slot);
-  };
-  auto issue = [&](int ch, int stage) {
-#pragma unroll 2
-    for (int r = warp; r < TOK; r += DW) {
-      const int slot = slot_s[ch & 1][r];
-      const bf16* src = static_cast<const bf16*>(a.rows) + static_cast<long long>(slot < 0 ? 0 : slot) * a.width;
-      const uint32_t dst = s_u32(Ks + (stage * TOK + r) * ld);
-      for (int c = lane; c < chunks; c += 32) {
-        const bool ok = slot >= 0 && c < wchunks;
-        cp_async16(dst + c * 16, src + (ok ? c * 8 : 0), ok ? 16 : 0);
-      }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  find_slots(0);
-  for (int r = warp; r < MT * 16; r += DW)
-    for (int c = lane * 8; c < KP; c += 256) {
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (h0 + r < a.heads && c < qld) v = *reinterpret_cast<const uint4*>(ql + (static_cast<long long>(b) * a.heads + h0 + r) * qld + c);
-      *reinterpret_cast<uint4*>(Qs + r * ld + c) = v;
-    }
-  __syncthreads();
-  if (n_ch > 0) issue(0, 0);
-  find_slots(1);
-  const uint32_t qaddr = s_u32(Qs + (wm * 16 + (lane & 15)) * ld + ((lane >> 4) << 3));
-  uint32_t qa[QI][2][4];
-#pragma unroll
-  for (int i = 0; i < QI; ++i)
-    if (i * 32 < KP) {
-      ldsm4(qaddr + i * 64, qa[i][0]);
-      ldsm4(qaddr + i * 64 + 32, qa[i][1]);
-    }
-  const float sl2 = a.scale * 1.4426950408889634f;
-  float m_run[2] = {-FLT_MAX, -FLT_MAX}, l_run[2] = {0.f, 0.f}, o[NTM][4];
-#pragma unroll
-  for (int j = 0; j < NTM; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-  const int NT = (a.rank + 8 * NG - 1) / (8 * NG);  // 8-wide column tiles per warp
-  const int col0 = wt * NT * 8;
-  const int r0 = lane >> 2;
-  __syncthreads();  // slots of the second stage
-  for (int ch = 0; ch < n_ch; ++ch) {
-    const int stage = ch & 1;
-    if (ch + 1 < n_ch) {
-      issue(ch + 1, stage ^ 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
-    __syncthreads();
-    find_slots(ch + 2);  // (the ones of chunk ch have been used)
-    const bf16* Kst = Ks + stage * TOK * ld;
-    float sc[MT][4];
-#pragma unroll
-    for (int nt = 0; nt < MT; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
-    const uint32_t kaddr = s_u32(Kst + (wt * 8 * MT + (lane & 7)) * ld + (lane >> 3) * 8);
-#pragma unroll
-    for (int i = 0; i < KI; ++i) {
-      if (i * 32 >= KP) break;
-      uint32_t q0[4], q1[4];
-      if (i < QI) {
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          q0[k] = qa[i < QI ? i : 0][0][k];
-          q1[k] = qa[i < QI ? i : 0][1][k];
-        }
-      } else {
-        ldsm4(qaddr + i * 64, q0);
-        ldsm4(qaddr + i * 64 + 32, q1);
-      }
-#pragma unroll
-      for (int nt = 0; nt < MT; ++nt) {
-        uint32_t kb[4];
-        ldsm4(kaddr + (nt * 8 * ld + i * 32) * 2, kb);
-        mma(sc[nt], q0, kb[0], kb[1]);
-        mma(sc[nt], q1, kb[2], kb[3]);
-      }
-    }
-    const int tok = t_lo + ch * TOK + wt * 8 * MT + (lane & 3) * 2;
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      float mx = -FLT_MAX;
-#pragma unroll
-      for (int nt = 0; nt < MT; ++nt)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          float& v = sc[nt][2 * r + e];
-          v = tok + nt * 8 + e < t_hi ? v * sl2 : -FLT_MAX;
-          mx = fmaxf(mx, v);
-        }
-      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-      mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-      if ((lane & 3) == 0) wmax[wt * MT * 16 + wm * 16 + r0 + 8 * r] = mx;
-    }
-    __syncthreads();
-    float corr[2];
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int row = wm * 16 + r0 + 8 * r;
-      float mn = m_run[r];
-#pragma unroll
-      for (int w = 0; w < NG; ++w) mn = fmaxf(mn, wmax[w * MT * 16 + row]);
-      corr[r] = m_run[r] == -FLT_MAX ? 0.f : exp2f(m_run[r] - mn);
-      m_run[r] = mn;
-      l_run[r] *= corr[r];
-#pragma unroll
-      for (int nt = 0; nt < MT; ++nt) {
-        const float p0 = sc[nt][2 * r] == -FLT_MAX ? 0.f : exp2f(sc[nt][2 * r] - mn);
-        const float p1 = sc[nt][2 * r + 1] == -FLT_MAX ? 0.f : exp2f(sc[nt][2 * r + 1] - mn);
-        l_run[r] += p0 + p1;
-        *reinterpret_cast<__nv_bfloat162*>(Ps + row * PLD + (wt * MT + nt) * 8 + (lane & 3) * 2) = __floats2bfloat162_rn(p0, p1);
-      }
-    }
-    __syncthreads();
-    if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
-#pragma unroll
-      for (int j = 0; j < NTM; ++j) {
-        o[j][0] *= corr[0]; o[j][1] *= corr[0];
-        o[j][2] *= corr[1]; o[j][3] *= corr[1];
-      }
-    }
-#pragma unroll
-    for (int k0 = 0; k0 < TOK; k0 += 16) {
-      uint32_t pa[4];
-      ldsm4(s_u32(Ps + (wm * 16 + (lane & 15)) * PLD + k0 + ((lane >> 4) << 3)), pa);
-      const uint32_t vrow = s_u32(Kst + (k0 + (lane & 7) + (((lane >> 3) & 1) << 3)) * ld);
-#pragma unroll
-      for (int jp = 0; jp < NTM / 2; ++jp) {
-        if (2 * jp >= NT) break;
-        const int c = col0 + jp * 16 + ((lane >> 4) << 3);
-        uint32_t vb[4];
-        ldsm4t(vrow + min(c, KP - 8) * 2, vb);  // (columns past the row end belong to tiles that are not stored)
-        mma(o[2 * jp], pa, vb[0], vb[1]);
-        mma(o[2 * jp + 1], pa, vb[2], vb[3]);
-      }
-    }
-    __syncthreads();  // the stage is refilled next
-  }
-  // sums over the token groups
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    float l = l_run[r];
-    l += __shfl_xor_sync(0xffffffffu, l, 1);
-    l += __shfl_xor_sync(0xffffffffu, l, 2);
-    if ((lane & 3) == 0) wsum[wt * MT * 16 + wm * 16 + r0 + 8 * r] = l;
-  }
-  __syncthreads();
-#pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    const int row = wm * 16 + r0 + 8 * r, h = h0 + row;
-    if (h >= a.heads) continue;
-    const long long base = (static_cast<long long>(b) * a.heads + h) * splits + split;
-    if (wt == 0 && (lane & 3) == 0) {
-      float l = 0.f;
-      for (int w = 0; w < NG; ++w) l += wsum[w * MT * 16 + row];
-      pml[base * 2] = m_run[r];
-      pml[base * 2 + 1] = l;
-    }
-#pragma unroll
-    for (int j = 0; j < NTM; ++j) {
-      const int c = col0 + j * 8 + (lane & 3) * 2;
-      if (j < NT && c < a.rank) *reinterpret_cast<float2*>(po + base * a.rank + c) = make_float2(o[j][2 * r], o[j][2 * r + 1]);
-    }
-  }
-}
-
-size_t decode_smem(int MT, int rank, int rot) {
-  const int ld = decode_k(rank, rot) + 8;
-  return sizeof(bf16) * (static_cast<size_t>(2) * TOK * ld + MT * 16 * ld + MT * 16 * PLD) + sizeof(float) * 2 * DW * MT * 16;
-}
-
 // ------------------------------------------------------------------------------------------------ projections of many rows
 // Tensor-core forms of the two per-head projections (bf16, more rows than the kernels above share a weight read among).
 constexpr int HM = 32;    // rows per CTA
@@ -600,13 +288,13 @@ __global__ void __launch_bounds__(128) absorb_mma_kernel(const HyLatent a, const
   for (int i = threadIdx.x; i < HM * (DP / 8); i += 128) {
     const int r = i / (DP / 8), c = (i - r * (DP / 8)) * 8;
     const bool ok = t0 + r < n_rows && c < a.dim;
-    cp_async16(s_u32(As + r * lda + c), q + (ok ? (static_cast<long long>(t0 + r) * a.heads + h) * qd + c : 0), ok ? 16 : 0);
+    cp16(s_u32(As + r * lda + c), q + (ok ? (static_cast<long long>(t0 + r) * a.heads + h) * qd + c : 0), ok ? 16 : 0);
   }
   const bf16* w = static_cast<const bf16*>(a.ukv) + static_cast<long long>(h) * a.dim * a.rank;
   for (int i = threadIdx.x; i < DP * (AN / 8); i += 128) {
     const int d = i / (AN / 8), c = (i & (AN / 8 - 1)) * 8;
     const bool ok = d < a.dim && r0 + c < a.rank;
-    cp_async16(s_u32(Bs + d * ldb + c), w + (ok ? static_cast<long long>(d) * a.rank + r0 + c : 0), ok ? 16 : 0);
+    cp16(s_u32(Bs + d * ldb + c), w + (ok ? static_cast<long long>(d) * a.rank + r0 + c : 0), ok ? 16 : 0);
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
   asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -655,7 +343,7 @@ __global__ void __launch_bounds__(128) up_mma_kernel(const HyLatent a, const flo
   for (int i = threadIdx.x; i < UN * (KP / 8); i += 128) {
     const int v = i / (KP / 8), c = (i - v * (KP / 8)) * 8;
     const bool ok = v0 + v < a.vdim && c < a.rank;
-    cp_async16(s_u32(Bs + v * ld + c), w + (ok ? static_cast<long long>(v0 + v) * a.rank + c : 0), ok ? 16 : 0);
+    cp16(s_u32(Bs + v * ld + c), w + (ok ? static_cast<long long>(v0 + v) * a.rank + c : 0), ok ? 16 : 0);
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -718,23 +406,6 @@ __global__ void __launch_bounds__(128) up_mma_kernel(const HyLatent a, const flo
 }
 
 // ------------------------------------------------------------------------------------------------ materialised form: inputs
-template <typename T>
-__global__ void __launch_bounds__(256) gather_rows_kernel(const HyLatent a, const int4* __restrict__ ranges, T* __restrict__ out) {
-  const int4 rg = ranges[blockIdx.y];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int i = blockIdx.x * 8 + warp;
-  if (i >= rg.w) return;
-  const long long slot = row_slot(a, rg.x, rg.y + i);
-  T* dst = out + static_cast<long long>(rg.z + i) * a.width;
-  constexpr int N = 16 / sizeof(T);
-  for (int c = lane * N; c < a.width; c += 32 * N) {
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (slot >= 0) v = *reinterpret_cast<const uint4*>(static_cast<const T*>(a.rows) + slot * a.width + c);
-    *reinterpret_cast<uint4*>(dst + c) = v;
-  }
-  if (slot < 0 && lane == 0 && a.status) atomicCAS(a.status, 0, 9);
-}
-
 __global__ void __launch_bounds__(256) pad_q_kernel(const HyLatent a, const bf16* __restrict__ q, const int* __restrict__ positions,
                                                     bf16* __restrict__ out, int nope, int rot) {
   const long long t = blockIdx.x;
@@ -813,33 +484,6 @@ int up_t(const HyLatent& a, const float* o, const float* ml, int splits, int n, 
   return n <= 2 ? up_rt<T, 1>(a, o, ml, splits, n, cat, ldc, s) : up_rt<T, 4>(a, o, ml, splits, n, cat, ldc, s);
 }
 
-template <typename T>
-int attend_t(const HyLatent& a, const float* ql, int qld, const int* positions, const int* row_seq, int n, float* o, cudaStream_t s) {
-  const size_t smem = sizeof(float) * static_cast<size_t>(a.rank + a.rot > 4 * a.rank ? a.rank + a.rot : 4 * a.rank);
-  auto go = [&](auto kern) -> int {
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-    if (e != cudaSuccess) return static_cast<int>(e);
-    kern<<<dim3(a.heads, n), 128, smem, s>>>(a, ql, qld, positions, row_seq, o);
-    return static_cast<int>(cudaGetLastError());
-  };
-  if (a.rank <= 128) return go(attend_kernel<T, 4>);
-  if (a.rank <= 256) return go(attend_kernel<T, 8>);
-  if (a.rank <= 512) return go(attend_kernel<T, 16>);
-  if (a.rank <= 1024) return go(attend_kernel<T, 32>);
-  if (a.rank <= 2048) return go(attend_kernel<T, 64>);
-  return static_cast<int>(cudaErrorInvalidValue);
-}
-
-template <int MT>
-int decode_t(const HyLatent& a, const bf16* ql, int qld, const int* seq_lens, int B, int splits, float* o, float* ml, cudaStream_t s) {
-  const size_t smem = decode_smem(MT, a.rank, a.rot);
-  auto kern = latent_decode_kernel<MT>;
-  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-  if (e != cudaSuccess) return static_cast<int>(e);
-  kern<<<dim3(B, (a.heads + MT * 16 - 1) / (MT * 16), splits), DW * 32, smem, s>>>(a, ql, qld, seq_lens, splits, o, ml);
-  return static_cast<int>(cudaGetLastError());
-}
-
 }  // namespace
 
 int hy_absorb_q(bool f32, const HyLatent& a, const void* q, const int* positions, int T, void* ql, int qld, bool out_f32,
@@ -849,38 +493,20 @@ int hy_absorb_q(bool f32, const HyLatent& a, const void* q, const int* positions
   return absorb_t<bf16, bf16>(a, q, positions, T, ql, qld, s);
 }
 
-int hy_latent_attend(bool f32, const HyLatent& a, const void* ql, int qld, const int* positions, const int* row_seq, int T,
-                     float* o, cudaStream_t s) {
-  const float* q = static_cast<const float*>(ql);
-  return f32 ? attend_t<float>(a, q, qld, positions, row_seq, T, o, s) : attend_t<bf16>(a, q, qld, positions, row_seq, T, o, s);
+HyAttend hy_latent_view(const HyLatent& a) {
+  HyAttend v = {};
+  static_cast<HyCache&>(v) = a;
+  v.heads = v.group = a.heads;   // all heads read the same row: scores over all of it, outputs of its first `rank` columns
+  v.kd = a.rank + a.rot;
+  v.vd = a.rank;
+  v.window = a.window;
+  v.scale = a.scale;
+  return v;
 }
 
 int hy_latent_up(bool f32, const HyLatent& a, const float* o, const float* ml, int splits, int T, void* cat, int ldc, cudaStream_t s) {
   if (splits < 1 || splits > 64) return static_cast<int>(cudaErrorInvalidValue);
   return f32 ? up_t<float>(a, o, ml, splits, T, cat, ldc, s) : up_t<bf16>(a, o, ml, splits, T, cat, ldc, s);
-}
-
-bool hy_latent_decode_supported(int heads, int rank, int rot, int width) {
-  return heads >= 1 && rank % 8 == 0 && rank >= 8 && rank <= 512 && decode_k(rank, rot) <= 576 && width % 8 == 0 && decode_smem(heads > 16 ? 2 : 1, rank, rot) <= 227 * 1024;
-}
-
-int hy_latent_decode(const HyLatent& a, const void* ql, int qld, const int* seq_lens, int B, int splits, float* o, float* ml,
-                     cudaStream_t s) {
-  if (!hy_latent_decode_supported(a.heads, a.rank, a.rot, a.width) || qld % 8 != 0 || splits < 1 || splits > 64 || a.num_slots > 0x7fffffffll)
-    return static_cast<int>(cudaErrorInvalidValue);
-  const bf16* q = static_cast<const bf16*>(ql);
-  return a.heads > 16 ? decode_t<2>(a, q, qld, seq_lens, B, splits, o, ml, s) : decode_t<1>(a, q, qld, seq_lens, B, splits, o, ml, s);
-}
-
-int hy_gather_rows(bool f32, const HyLatent& a, const int* ranges, int n, int max_rows, void* out, cudaStream_t s) {
-  if (n <= 0 || max_rows <= 0) return 0;
-  const dim3 grid((max_rows + 7) / 8, n);
-  const int4* rg = reinterpret_cast<const int4*>(ranges);
-  if (f32)
-    gather_rows_kernel<float><<<grid, 256, 0, s>>>(a, rg, static_cast<float*>(out));
-  else
-    gather_rows_kernel<bf16><<<grid, 256, 0, s>>>(a, rg, static_cast<bf16*>(out));
-  return static_cast<int>(cudaGetLastError());
 }
 
 int hy_pad_q(const HyLatent& a, const void* q, const int* positions, int T, int nope_pad, int rot_pad, void* out, cudaStream_t s) {

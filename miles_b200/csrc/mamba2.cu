@@ -13,7 +13,7 @@
 // The convolution keeps its inputs in a ring of `taps` rows indexed by position: the row a token writes is never one that is
 // read for it, so all heads of a group can read the shared B / C channels while one of them stores.
 #include "hybrid.h"
-#include "hybrid_common.cuh"
+#include "hybrid_mma.cuh"
 
 namespace mb {
 namespace {
@@ -32,14 +32,7 @@ struct Decay {
   __device__ __forceinline__ float operator()(float s) const { return fmaf(c, s, k * s); }
 };
 
-// State row of a sequence; one outside the cache is reported and not followed (-1: the sequence starts from nothing and its state
-// is not kept).
-__device__ __forceinline__ long long state_row(const HyMamba& a, int seq) {
-  const int slot = a.slots[seq];
-  if (slot >= 0 && slot < a.sequences) return slot;
-  if (a.status) atomicCAS(a.status, 0, 11);
-  return -1;
-}
+__device__ __forceinline__ long long state_row(const HyMamba& a, int seq) { return hy::state_row(a.slots, a.sequences, seq, a.status); }
 
 // ------------------------------------------------------------------------------------------------ convolution (prefill)
 template <typename T, int TAPS>
@@ -293,58 +286,34 @@ constexpr int Q = HY_CHUNK;      // tokens per chunk
 constexpr int CW = 8;            // warps
 constexpr int LDX_PAD = 8;       // bf16 elements added to shared rows: conflict-free ldmatrix
 
-__device__ __forceinline__ uint32_t s_u32(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
-__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// fp32 pair -> two bf16 terms whose sum keeps 16 bits of mantissa
-__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  const float2 f = __bfloat1622float2(h);
-  const __nv_bfloat162 l = __floats2bfloat162_rn(x - f.x, y - f.y);
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = *reinterpret_cast<const uint32_t*>(&l);
-}
-
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src, int bytes) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void cp_wait_all() {
-  asm volatile("cp.async.commit_group;" ::: "memory");
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
-}
-
-constexpr float LOG2E = 1.4426950408889634f;
 constexpr int MAX_HB = 8;        // heads of one group a CTA works on (a warp computes the decays of each)
 
 // Warp w, head h0 + w, in units of log2: acum = running sum of -exp(A_log) dt over the chunk, src = acum - log2(dt), so that what
-// token s hands to token t is exp2(acum_t - src_s) = exp(..) dt_s. Tokens past n get dt = 0: the sum stays flat, src = +inf.
+// token s hands to token t is exp2(acum_t - src_s) = exp(..) dt_s. Tokens past n get dt = 0: the sum stays flat, src = +inf. With
+// log2_decay every token decays the state of head h by that much and dt = 1.
 __device__ __forceinline__ void chunk_decays(const HyMamba& a, int h0, int nh, int row0, int n, float* src, float* acum) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (warp >= nh) return;
   const int h = h0 + warp, inner = a.heads * a.P, ch = inner + 2 * a.groups * a.N;
-  const bf16* col = static_cast<const bf16*>(a.proj) + inner + ch + h;
-  const float bias = to_f(static_cast<const bf16*>(a.dt_bias)[h]), A = -expf(to_f(static_cast<const bf16*>(a.A_log)[h])) * LOG2E;
   float dt[Q / 32], v[Q / 32], run = 0.f;
+  if (a.log2_decay) {
+    const float A = a.log2_decay[h];
 #pragma unroll
-  for (int i = 0; i < Q / 32; ++i) {
-    const int t = lane * (Q / 32) + i;
-    dt[i] = t < n ? softplus_f(to_f(col[static_cast<long long>(row0 + t) * a.ld]) + bias) : 0.f;
-    run += A * dt[i];
-    v[i] = run;
+    for (int i = 0; i < Q / 32; ++i) {
+      dt[i] = lane * (Q / 32) + i < n ? 1.f : 0.f;
+      run += A * dt[i];
+      v[i] = run;
+    }
+  } else {
+    const bf16* col = static_cast<const bf16*>(a.proj) + inner + ch + h;
+    const float bias = to_f(static_cast<const bf16*>(a.dt_bias)[h]), A = -expf(to_f(static_cast<const bf16*>(a.A_log)[h])) * LOG2E;
+#pragma unroll
+    for (int i = 0; i < Q / 32; ++i) {
+      const int t = lane * (Q / 32) + i;
+      dt[i] = t < n ? softplus_f(to_f(col[static_cast<long long>(row0 + t) * a.ld]) + bias) : 0.f;
+      run += A * dt[i];
+      v[i] = run;
+    }
   }
   float base = run;
 #pragma unroll
@@ -360,38 +329,6 @@ __device__ __forceinline__ void chunk_decays(const HyMamba& a, int h0, int nh, i
   }
 }
 
-// rows [n, w] of a row-major bf16 matrix (pitch `pitch`) into smem [rows][ld], zero filled to wp columns; vec: by 16-byte
-// asynchronous copies the caller waits for
-template <int THREADS>
-__device__ __forceinline__ void load_tile(const bf16* __restrict__ src, long long pitch, int n, int w, int rows, int wp, bf16* dst,
-                                          int ld, bool vec) {
-  if (vec) {
-    const int per = wp / 8;
-    if ((THREADS) % per == 0) {  // every thread keeps its column
-      const int step = THREADS / per, r0 = threadIdx.x / per, c = (threadIdx.x - r0 * per) * 8;
-      const bool col = c < w;
-      const bf16* p = src + r0 * pitch + c;
-      uint32_t d = s_u32(dst + r0 * ld + c);
-#pragma unroll 4
-      for (int r = r0; r < rows; r += step, p += step * pitch, d += step * ld * 2) {
-        const bool ok = col && r < n;
-        cp16(d, ok ? p : src, ok ? 16 : 0);
-      }
-      return;
-    }
-    for (int i = threadIdx.x; i < rows * per; i += THREADS) {
-      const int r = i / per, c = (i - r * per) * 8;
-      const bool ok = r < n && c < w;
-      cp16(s_u32(dst + r * ld + c), src + (ok ? r * pitch + c : 0), ok ? 16 : 0);
-    }
-  } else {
-    for (int i = threadIdx.x; i < rows * wp; i += THREADS) {
-      const int r = i / wp, c = i - r * wp;
-      dst[r * ld + c] = (r < n && c < w) ? src[r * pitch + c] : __float2bfloat16(0.f);
-    }
-  }
-}
-
 // (1) work[chunk, h, p, n] = sum_t exp(acum_end - acum_t) dt_t x_t[p] B_t[n];  decay[chunk, h] = exp(acum_end). A CTA takes
 // several heads of a group: their B is the same tile.
 template <int PT>
@@ -403,7 +340,6 @@ __global__ void __launch_bounds__(CW * 32, 2) chunk_state_kernel(const HyMamba a
   const int row0 = ck.y, n = ck.z;
   const int P = a.P, N = a.N, NP = (N + 63) / 64 * 64, hpg = a.heads / a.groups;
   constexpr int PP = PT * 16, ldx = PP + LDX_PAD, XV = PP * Q / 8 / (CW * 32);
-  const int inner = a.heads * P, ch = inner + 2 * a.groups * N;
   const int per_group = (hpg + hb - 1) / hb, g = blockIdx.y / per_group;
   const int h0 = g * hpg + (blockIdx.y - g * per_group) * hb, nh = min(hb, (g + 1) * hpg - h0);
   const int ldb = NP + LDX_PAD;
@@ -412,7 +348,7 @@ __global__ void __launch_bounds__(CW * 32, 2) chunk_state_kernel(const HyMamba a
   bf16* Bs = xl + Q * ldx;                   // [Q][ldb]
   float* srcs = reinterpret_cast<float*>(Bs + Q * ldb);  // [MAX_HB][Q]
   float* acum = srcs + MAX_HB * Q;
-  load_tile<CW * 32>(xbc + static_cast<long long>(row0) * ch + inner + g * N, ch, n, N, Q, NP, Bs, ldb, vec);
+  load_tile<CW * 32>(xbc + row0 * a.xld + a.b_col + g * N, a.xld, n, N, Q, NP, Bs, ldb, vec);
   uint4 xr[XV];
   auto fetch = [&](int h) {
 #pragma unroll
@@ -420,7 +356,7 @@ __global__ void __launch_bounds__(CW * 32, 2) chunk_state_kernel(const HyMamba a
       const int k = threadIdx.x + i * CW * 32, r = k / (PP / 8), c = (k - r * (PP / 8)) * 8;
       xr[i] = make_uint4(0u, 0u, 0u, 0u);
       if (r >= n || c >= P) continue;
-      const bf16* src = xbc + static_cast<long long>(row0 + r) * ch + h * P + c;
+      const bf16* src = xbc + (row0 + r) * a.xld + a.x_col + h * P + c;
       if (vec) {
         xr[i] = *reinterpret_cast<const uint4*>(src);
       } else {
@@ -505,8 +441,9 @@ __global__ void __launch_bounds__(CW * 32, 2) chunk_state_kernel(const HyMamba a
 }
 
 // (2) the state before every chunk, as two bf16 planes (high part, low part) [chunk, h, 2, P, N]; the state after the last chunk
-// goes to the sequence's row
-template <int V>
+// goes to the sequence's row. Decays are one per head, or (COLS) [chunk, h, 2, N]: one per column n, and a factor the planes are
+// multiplied by
+template <int V, bool COLS>
 __global__ void __launch_bounds__(256) chunk_pass_kernel(const HyMamba a, const int* __restrict__ first_chunk,
                                                          const float* __restrict__ decay, const float* __restrict__ work,
                                                          bf16* __restrict__ before) {
@@ -518,7 +455,7 @@ __global__ void __launch_bounds__(256) chunk_pass_kernel(const HyMamba a, const 
   float* st = a.state + ((slot < 0 ? 0 : slot) * a.heads + h) * size + i;
   float s[V];
   const bool cont = slot >= 0 && a.ctx[seq] > 0;
-  auto load = [](const float* p, float (&v)[V]) {
+  auto load = [](const float* p, auto& v) {
     if constexpr (V == 4) {
       const float4 t = *reinterpret_cast<const float4*>(p);
       v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
@@ -530,31 +467,42 @@ __global__ void __launch_bounds__(256) chunk_pass_kernel(const HyMamba a, const 
   for (int k = 0; k < V; ++k) s[k] = 0.f;
   if (cont) load(st, s);
   const int c0 = first_chunk[seq], c1 = first_chunk[seq + 1];
-  constexpr int U = 8;  // loads of several chunks in flight
+  constexpr int U = COLS ? 4 : 8;  // loads of several chunks in flight
+  const int col = COLS ? static_cast<int>(i % a.N) : 0;
   for (int c = c0; c < c1; c += U) {
-    float v[U][V], d[U];
+    float v[U][V], d[U][COLS ? V : 1], f[U][COLS ? V : 1];
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       if (c + u >= c1) break;
-      load(work + (static_cast<long long>(c + u) * a.heads + h) * size + i, v[u]);
-      d[u] = decay[static_cast<long long>(c + u) * a.heads + h];
+      const long long at = static_cast<long long>(c + u) * a.heads + h;
+      load(work + at * size + i, v[u]);
+      if constexpr (COLS) {
+        load(decay + at * 2 * a.N + col, d[u]);
+        load(decay + (at * 2 + 1) * a.N + col, f[u]);
+      } else {
+        d[u][0] = decay[at];
+      }
     }
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       if (c + u >= c1) break;
       bf16* dst = before + (static_cast<long long>(c + u) * a.heads + h) * 2 * size + i;
+      float b[V];
+#pragma unroll
+      for (int k = 0; k < V; ++k) b[k] = COLS ? s[k] * f[u][COLS ? k : 0] : s[k];
       if constexpr (V == 4) {
         uint32_t hi[2], lo[2];
-        split2(s[0], s[1], hi[0], lo[0]);
-        split2(s[2], s[3], hi[1], lo[1]);
+        split2(b[0], b[1], hi[0], lo[0]);
+        split2(b[2], b[3], hi[1], lo[1]);
         *reinterpret_cast<uint2*>(dst) = make_uint2(hi[0], hi[1]);
         *reinterpret_cast<uint2*>(dst + size) = make_uint2(lo[0], lo[1]);
       } else {
-        dst[0] = __float2bfloat16(s[0]);
-        dst[size] = __float2bfloat16(s[0] - to_f(dst[0]));
+        const bf16 top = __float2bfloat16(b[0]);
+        dst[0] = top;
+        dst[size] = __float2bfloat16(b[0] - to_f(top));
       }
 #pragma unroll
-      for (int k = 0; k < V; ++k) s[k] = d[u] * s[k] + v[u][k];
+      for (int k = 0; k < V; ++k) s[k] = d[u][COLS ? k : 0] * s[k] + v[u][k];
     }
   }
   if (slot < 0) return;
@@ -579,7 +527,7 @@ chunk_out_kernel(const HyMamba a, const bf16* __restrict__ xbc, const int4* __re
   const int4 ck = chunks[blockIdx.x];
   const int seq = ck.x, row0 = ck.y, n = ck.z;
   const int P = a.P, N = a.N, NP = (N + 15) / 16 * 16, hpg = a.heads / a.groups;
-  const int inner = a.heads * P, ch = inner + 2 * a.groups * N;
+  const int inner = a.heads * P;
   const int per_group = (hpg + hb - 1) / hb, g = blockIdx.y / per_group;
   const int h0 = g * hpg + (blockIdx.y - g * per_group) * hb, nh = min(hb, (g + 1) * hpg - h0);
   constexpr int PP = PH * 64;
@@ -592,9 +540,9 @@ chunk_out_kernel(const HyMamba a, const bf16* __restrict__ xbc, const int4* __re
   bf16* xs = Cs + Q * ldn;                               // [NBUF][Q][ldx]
   bf16* Ss = xs + NBUF * Q * ldx;                        // [NBUF][2][PP][ldn]; the first one holds B before that
   const bool carried = ck.w > 0 || a.ctx[seq] > 0;
-  const bf16* rows = xbc + static_cast<long long>(row0) * ch;
-  load_tile<OW * 32>(rows + inner + a.groups * N + g * N, ch, n, N, Q, NP, Cs, ldn, vec);
-  load_tile<OW * 32>(rows + inner + g * N, ch, n, N, Q, NP, Ss, ldn, vec);
+  const bf16* rows = xbc + row0 * a.xld;
+  load_tile<OW * 32>(rows + a.c_col + g * N, a.xld, n, N, Q, NP, Cs, ldn, vec);
+  load_tile<OW * 32>(rows + a.b_col + g * N, a.xld, n, N, Q, NP, Ss, ldn, vec);
   chunk_decays(a, h0, nh, row0, n, srcs, acum);
   cp_wait_all();
   __syncthreads();
@@ -624,7 +572,7 @@ chunk_out_kernel(const HyMamba a, const bf16* __restrict__ xbc, const int4* __re
   __syncthreads();
   auto fetch = [&](int hi) {
     const int h = h0 + hi, buf = NBUF == 2 ? hi & 1 : 0;
-    load_tile<OW * 32>(rows + h * P, ch, n, P, Q, PP, xs + buf * Q * ldx, ldx, vec);
+    load_tile<OW * 32>(rows + a.x_col + h * P, a.xld, n, P, Q, PP, xs + buf * Q * ldx, ldx, vec);
     if (carried) {
       const bf16* src = before + (static_cast<long long>(blockIdx.x) * a.heads + h) * 2 * P * N;
       bf16* dst = Ss + buf * 2 * PP * ldn;
@@ -649,7 +597,7 @@ chunk_out_kernel(const HyMamba a, const bf16* __restrict__ xbc, const int4* __re
       const bf16* sb = Ss + buf * 2 * PP * ldn;
       const float* ac = acum + hi * Q;
       const float* from = srcs + hi * Q;
-      const float D = to_f(static_cast<const bf16*>(a.D)[h]);
+      const float D = a.D ? to_f(static_cast<const bf16*>(a.D)[h]) : 0.f;
 #pragma unroll 1
       for (int half = 0; half < 2; ++half) {
         const int tile = half == 0 ? ta : tb;
@@ -855,13 +803,25 @@ bool hy_chunk_scan_supported(int P, int N, int, int) {
   return state_smem(2 * ph, N) <= 227 * 1024 && out_smem(P <= 64 ? 1 : 2, N, 1) <= 227 * 1024;
 }
 
+int hy_chunk_pass(const HyMamba& a, const int* first_chunk, const float* decay, bool cols, const float* work, void* before_, cudaStream_t s) {
+  const long long size = static_cast<long long>(a.P) * a.N;
+  bf16* before = static_cast<bf16*>(before_);
+  const bool four = cols ? a.N % 4 == 0 : size % 4 == 0;
+  const dim3 grid(static_cast<unsigned>(((four ? size / 4 : size) + 255) / 256), a.heads, a.nseq);
+  if (four && cols) chunk_pass_kernel<4, true><<<grid, 256, 0, s>>>(a, first_chunk, decay, work, before);
+  else if (four) chunk_pass_kernel<4, false><<<grid, 256, 0, s>>>(a, first_chunk, decay, work, before);
+  else if (cols) chunk_pass_kernel<1, true><<<grid, 256, 0, s>>>(a, first_chunk, decay, work, before);
+  else chunk_pass_kernel<1, false><<<grid, 256, 0, s>>>(a, first_chunk, decay, work, before);
+  return static_cast<int>(cudaGetLastError());
+}
+
 int hy_chunk_scan(const HyMamba& a, const void* xbc_, const int* chunks, int n_chunks, const int* first_chunk, float* work,
                   float* decay, void* before_, void* y_, cudaStream_t s) {
   if (!hy_chunk_scan_supported(a.P, a.N, a.heads, a.groups)) return static_cast<int>(cudaErrorInvalidValue);
   const bf16* xbc = static_cast<const bf16*>(xbc_);
   bf16 *y = static_cast<bf16*>(y_), *before = static_cast<bf16*>(before_);
   const int4* ck = reinterpret_cast<const int4*>(chunks);
-  const bool vec = a.P % 8 == 0 && a.N % 8 == 0 && (reinterpret_cast<uintptr_t>(xbc) & 15) == 0;
+  const bool vec = a.P % 8 == 0 && a.N % 8 == 0 && (a.x_col | a.b_col | a.c_col) % 8 == 0 && aligned16<bf16>(xbc, a.xld);
   const int ph = half_tiles(a.P), hb = heads_per_cta(n_chunks, a.heads, a.groups);
   int rc = 0;
   switch (ph) {
@@ -871,13 +831,8 @@ int hy_chunk_scan(const HyMamba& a, const void* xbc_, const int* chunks, int n_c
     default: rc = launch_state<8>(a, xbc, ck, n_chunks, hb, work, decay, vec, s); break;
   }
   if (rc != 0) return rc;
-  const long long size = static_cast<long long>(a.P) * a.N;
-  if (size % 4 == 0)
-    chunk_pass_kernel<4><<<dim3(static_cast<unsigned>((size / 4 + 255) / 256), a.heads, a.nseq), 256, 0, s>>>(a, first_chunk, decay, work, before);
-  else
-    chunk_pass_kernel<1><<<dim3(static_cast<unsigned>((size + 255) / 256), a.heads, a.nseq), 256, 0, s>>>(a, first_chunk, decay, work, before);
-  const cudaError_t e = cudaGetLastError();
-  if (e != cudaSuccess) return static_cast<int>(e);
+  rc = hy_chunk_pass(a, first_chunk, decay, false, work, before, s);
+  if (rc != 0) return rc;
   const bool two = out_smem(a.P <= 64 ? 1 : 2, a.N, 2) <= 227 * 1024;
   if (a.P <= 64)
     return two ? launch_out<1, 2>(a, xbc, ck, n_chunks, hb, before, y, vec, s) : launch_out<1, 1>(a, xbc, ck, n_chunks, hb, before, y, vec, s);

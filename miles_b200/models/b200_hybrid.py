@@ -8,6 +8,14 @@ A parallel layer is two large products with fused kernels between them:
     x   += [o | down] cat                          one product over everything that writes the residual, fp32
     x   += rmsnorm(proj(gelu(gate x) * e)) * norm  per-layer token input, ending in the next layer's norm
 
+A sequential layer has one product in front of and one behind each mixer or feed-forward, and one kernel per sublayer that norms
+its output, adds it to the residual and norms that for whatever reads it next:
+
+    proj = [everything the mixer reads] h
+    out  = mixer kernels on proj                   (csrc/linear_attention.cu, cached_attention.cu, cached_prefill.cu)
+    y    = o out (fp32; two of them where two mixers run side by side)
+    x   += norm(y), h = norm(x)                    (csrc/sequential_ops.cu)
+
 bf16 stores run the products on the tcgen05 GEMM (few rows: the weight-streaming kernel), prompts through the chunked
 recurrence and the tcgen05 attention. fp32 stores run the same layer code with 32-bit products and the plain kernels of any
 size. Head sizes the tensor-core kernels do not take fall to those plain kernels too, in bf16.
@@ -23,7 +31,7 @@ from ..ops import _ext
 from ..ops.attention import TILE_Q
 from ..ops.reference import pair_frequencies
 from .config import ModelConfig
-from .layer_plan import Mamba2
+from .layer_plan import LinearAttention, Mamba2, Parallel
 from .params import ParamStore
 from .torch_hybrid import TorchHybrid
 from .torch_impl import InferMeta
@@ -42,10 +50,15 @@ class B200Hybrid(TorchHybrid):
         self.status = torch.zeros(1, dtype=torch.int32, device=self.dev)
         self.launches = 0
         self.freq = {}
-        for l in cfg.plan.layers:
-            if not isinstance(l.mixer, Mamba2):
-                r = l.mixer.rotary
-                self.freq[(r.base, r.dims)] = pair_frequencies(r.dims, r.base, self.dev)
+        self.fixed_decay = {}  # (layer, side) -> decays - 1 and their base-2 logarithms
+        for i, l in enumerate(cfg.plan.layers):
+            for side, m in l.mixer.sides() if isinstance(l.mixer, Parallel) else [("", l.mixer)]:
+                r = getattr(m, "rotary", None)
+                if r is not None:
+                    self.freq[(r.base, r.dims)] = pair_frequencies(r.dims, r.base, self.dev)
+                if isinstance(m, LinearAttention) and m.decay is not None:
+                    d = torch.tensor(m.decay, dtype=torch.float64)
+                    self.fixed_decay[(i, side)] = ((d - 1).float().to(self.dev), d.log2().clamp(min=-1e4).float().to(self.dev))
         self.sms = torch.cuda.get_device_properties(self.dev).multi_processor_count
         self.plain = False  # True: the kernels of any size everywhere (what the fast ones are checked against)
 
@@ -81,7 +94,7 @@ class B200Hybrid(TorchHybrid):
     def _tables(self, meta: InferMeta) -> dict:
         """Convolution tiles and chunks of a pass: {sequence, first row, rows, index in the sequence}."""
         t = meta.tables
-        if "conv" not in t:
+        if "chunks" not in t:
             cu, q = meta.cu_list, self.C.CHUNK
             conv, chunks, first = [], [], [0]
             for b in range(len(cu) - 1):
@@ -157,7 +170,7 @@ class B200Hybrid(TorchHybrid):
                 longest = meta.block_table.shape[1] * meta.page_size
                 if m.window:
                     longest = min(longest, m.window)
-                splits = max(1, min(self.sms // max(1, B * groups), (longest + 63) // 64, 32))
+                splits = self._decode_splits(B, groups, longest)
                 C.latent_decode(*args, q, positions, meta.seq_lens, splits, cat)
             else:
                 C.latent_attend(*args, q, positions, None, cat)
@@ -169,7 +182,94 @@ class B200Hybrid(TorchHybrid):
         else:
             C.latent_attend(*args, q, positions, self._row_seq(meta), cat)
 
+    def _rows_for(self, T: int, width: int, used: int):
+        """Input rows of a product with ``width`` columns, of which the mixer fills ``used``."""
+        return (torch.empty if used == width else torch.zeros)(T, width, dtype=self.store.dtype, device=self.dev)
+
+    def _decode_splits(self, B: int, groups: int, longest: int) -> int:
+        return max(1, min(self.sms // max(1, B * groups), (longest + 63) // 64, 32))
+
+    def _attention(self, i, m, side, proj, positions, meta, rows):
+        """Softmax attention over cached key / value heads; keys and values of ``proj`` go to their cache rows."""
+        P, C, T = self.store.params, self.C, proj.shape[0]
+        col = {n: self.in_segs[i][f"mix.{side}{n}"].start for n in ("q", "k", "v")}
+        r = m.rotary
+        rot, freq = (r.dims, self.freq[(r.base, r.dims)]) if r is not None else (0, None)
+        fast = not self.f32 and not self.plain
+        if meta.is_prefill:
+            fast = fast and C.attn_prefill_supported(m.kv_heads, m.dim, m.vdim, rows.shape[1])
+        else:
+            fast = fast and C.attn_decode_supported(m.heads, m.kv_heads, m.dim, m.vdim, rows.shape[1])
+        pitch = (64 if m.dim <= 64 else 128) if fast and meta.is_prefill else m.dim
+        q = torch.empty(T, m.heads * pitch, dtype=self.store.dtype if fast else torch.float32, device=self.dev)
+        nk, nv = m.kv_heads * m.dim, m.kv_heads * m.vdim
+        C.head_rows(proj, positions, meta.slot_mapping, self.plan.eps, self.status,
+                    [(col["q"], m.heads, m.dim, rot, freq, m.unit_qk, 1.0, q, 0, pitch, 0, False),
+                     (col["k"], m.kv_heads, m.dim, rot, freq, m.unit_qk, 1.0, rows, 0, m.dim, 0, True),
+                     (col["v"], m.kv_heads, m.vdim, 0, None, False, 1.0, rows, nk, m.vdim, rows.shape[1] - nk - nv, True)])
+        out = self._rows_for(T, P[f"layers.{i}.{side}o.weight"].shape[1], m.out_dim)
+        args = (m.heads, m.kv_heads, m.dim, m.vdim, m.scale, P[f"layers.{i}.mix.{side}sink"] if m.sink else None, rows, meta.block_table,
+                meta.page_size, self.status)
+        self.launches += 3
+        if not fast:
+            C.attn_plain(*args, q, positions, self._row_seq(meta) if meta.is_prefill else None, out)
+        elif meta.is_prefill:
+            ranges, total, longest, tiles = self._attn_tables(meta, 0)
+            C.attn_prefill(*args, q, pitch, ranges, total, longest, tiles, out)
+        else:
+            per_head = m.heads // m.kv_heads
+            groups = m.kv_heads * ((per_head + 15) // 16 if per_head <= 16 else (per_head + 31) // 32)
+            C.attn_decode(*args, q, meta.seq_lens, self._decode_splits(T, groups, meta.block_table.shape[1] * meta.page_size), out)
+        return out
+
+    def _linear_attention(self, i, m, side, proj, positions, meta, state):
+        P, C, p = self.store.params, self.C, f"layers.{i}.mix.{side}"
+        segs = self.in_segs[i]
+        cols = [segs[f"mix.{side}{n}"].start for n in ("v", "k", "q", "g")] + [segs[f"mix.{side}a1"].start if m.rank else -1]
+        fixed = self.fixed_decay.get((i, side), (None, None))
+        s = m.dim ** -0.5
+        rot, freq = (m.rotary.dims, self.freq[(m.rotary.base, m.rotary.dims)]) if m.rotary is not None else (0, None)
+        args = (proj, cols, m.heads, m.vdim, m.dim, 1.0 if m.scale_keys else s, s if m.scale_keys else 1.0, rot, freq, *fixed,
+                P[p + "a2.weight"] if m.rank else None, P[p + "a2.bias"] if m.rank else None, 1.0 / m.tau, P[p + "norm.weight"] if m.norm_weight else None,
+                self.plan.eps, state, meta.state_slots, self.status)
+        out = torch.empty(proj.shape[0], P[f"layers.{i}.{side}o.weight"].shape[1], dtype=proj.dtype, device=self.dev)
+        if meta.is_prefill:
+            t = self._tables(meta)
+            fast = not self.plain
+            C.linear_prefill(*args, positions, meta.cu_seqlens, meta.ctx_lens, t["chunks"] if fast else None, t["first"] if fast else None, out)
+            self.launches += 5
+        else:
+            C.linear_step(*args, positions, out)
+            self.launches += 1
+        return out
+
     # ------------------------------------------------------------------ layers
+    def _sequential_layer(self, run, x, h, positions, meta, cache):
+        """Updates the fp32 residual ``x`` in place and ``h`` to what the next layer run reads."""
+        i = self.runs[run]
+        l, P, p, C = self.plan.layers[i], self.store.params, f"layers.{i}.", self.C
+        m, eps, f32 = l.mixer, self.plan.eps, torch.float32
+        after = f"layers.{self.runs[run + 1]}.norm1" if run + 1 < len(self.runs) else "final_norm"
+        proj = self.linear(h, P[p + "in.weight"])
+        second = (None, None, None)
+        if isinstance(m, Parallel):
+            a = self._attention(i, m.left, "left.", proj, positions, meta, cache[0])
+            b = self._linear_attention(i, m.right, "right.", proj, positions, meta, cache[1])
+            y = self.linear(a, P[p + "left.o.weight"], f32)
+            second = (self.linear(b, P[p + "right.o.weight"], f32), P[p + "mix.left.out_norm.weight"], P[p + "mix.right.out_norm.weight"])
+        else:
+            y = self.linear(self._linear_attention(i, m, "", proj, positions, meta, cache[0]), P[p + "o.weight"], f32)
+        C.sandwich(x, y, *second, P[p + "norm1b.weight"], P[(p + "norm2" if l.ff is not None else after) + ".weight"], h, eps)
+        self.launches += 1
+        if l.ff is not None:
+            z = self.linear(h, P[p + "ff_in.weight"])
+            gate, up = l.ff_segments()
+            w = P[p + "ff_out.weight"]
+            act = torch.empty(z.shape[0], w.shape[1], dtype=z.dtype, device=self.dev)
+            C.gated_act(z, gate.start, up.start, l.ff.ff, l.ff.act == "relu", act)
+            C.sandwich(x, self.linear(act, w, f32), None, None, None, P[p + "norm2b.weight"], P[after + ".weight"], h, eps)
+            self.launches += 2
+
     def _next_norm(self, i):
         return f"layers.{i + 1}.norm1" if i + 1 < self.cfg.num_layers else "final_norm"
 
@@ -216,11 +316,17 @@ class B200Hybrid(TorchHybrid):
         T, H = tokens.shape[0], self.cfg.hidden_size
         x = torch.empty(T, H, dtype=torch.float32, device=self.dev)
         h = torch.empty(T, H, dtype=self.store.dtype, device=self.dev)
-        first = "layers.0.norm1"
-        self.C.embed_norm(tokens, P["embed.weight"], P[first + ".weight"], P[first + ".bias"], P[first + ".alpha"], x, h, self.status)
+        first = f"layers.{self.runs[0]}.norm1"
+        if self.plan.norm == "layer_norm":
+            self.C.embed_layer_norm(tokens, P["embed.weight"], P[first + ".weight"], x, h, self.plan.eps, self.status)
+        else:
+            self.C.embed_norm(tokens, P["embed.weight"], P[first + ".weight"], P[first + ".bias"], P[first + ".alpha"], x, h, self.status)
         self.launches += 1
-        for i in range(self.cfg.num_layers):
-            self._layer(i, x, h, tokens, positions, meta, kv_cache[i])
+        for run, i in enumerate(self.runs):
+            if self.plan.parallel:
+                self._layer(i, x, h, tokens, positions, meta, kv_cache[run])
+            else:
+                self._sequential_layer(run, x, h, positions, meta, kv_cache[run])
             if self.capture is not None:
                 self.capture.append(x.clone())
         return h
