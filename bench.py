@@ -128,17 +128,18 @@ def main() -> None:
                          "timed are reported in `steps`")
     ap.add_argument("--replicate-experts", choices=["auto", "on", "off"], default="auto",
                     help="rollout engine of an expert-parallel run: full replica of the experts per GPU, or expert parallel")
-    ap.add_argument("--workload", choices=["grpo", "rokivik"], default="grpo",
-                    help="rokivik: prefill and decode throughput of a Rokivik model beside the closest Qwen3 model (benchmarks/bench_hybrid.py)")
+    ap.add_argument("--workload", choices=["grpo", "rokivik", "pesanex"], default="grpo",
+                    help="rokivik, pesanex: prefill and decode throughput of a model of that design beside the closest models of equal size "
+                         "(benchmarks/bench_hybrid.py)")
     ns = ap.parse_args()
     if ns.impl == "reference":
         reference_arm(ns)
         return
-    if ns.workload == "rokivik":
+    if ns.workload != "grpo":
         sys.path.insert(0, os.path.join(os.path.dirname(os.path.abspath(__file__)), "benchmarks"))
         import bench_hybrid
 
-        bench_hybrid.main([], steps=max(ns.steps, 10), warmup=ns.warmup)
+        bench_hybrid.main(["--design", ns.workload], steps=max(ns.steps, 10), warmup=ns.warmup)
         return
 
     import torch

@@ -1,11 +1,13 @@
-"""Prefill and decode throughput of a Rokivik model beside a Qwen3 model of equal width and depth (random weights).
+"""Prefill and decode throughput of layer-planned models beside other models of equal width and depth (random weights).
 
     python bench.py --workload rokivik                     # both sizes, prompts and decoding, one JSON line each
-    python benchmarks/bench_hybrid.py --kernels            # also per-kernel device times and roofline fractions
+    python bench.py --workload pesanex
+    python benchmarks/bench_hybrid.py --design pesanex --kernels   # also per-kernel device times and roofline fractions
 
-Sizes are those of real models' layers: width 2048 (beside Qwen3-1.7B) and width 4096 (beside Qwen3-8B), six layers of each:
-Mamba-2, latent attention (windowed), Mamba-2, latent attention reading the first one's latents, Mamba-2, latent attention
-over the whole context. Prompts are timed around the model's forward pass over staged inputs, decoding around the engine's own
+Sizes are those of real models' layers: width 2048 (beside Qwen3-1.7B) and width 4096 (beside Qwen3-8B), six layers of each.
+Rokivik: Mamba-2, latent attention (windowed), Mamba-2, latent attention reading the first one's latents, Mamba-2, latent attention
+over the whole context. Pesanex: softmax attention beside gated linear attention, retention, gated linear attention, and these three
+again, every layer with a feed-forward; it stands beside Rokivik (the like recurrence) and Qwen3 (the like attention). Prompts are timed around the model's forward pass over staged inputs, decoding around the engine's own
 step (captured graph), both with CUDA events after warm-up; the weights of a pass are several times the L2 (so is the cache
 at the larger batches), nothing else is flushed. Each line carries SM clocks sampled during its timed region.
 """
@@ -28,6 +30,9 @@ SIZES = {
     "2048": dict(width=2048, ff=6144, heads=16, q_rank=768, kv_rank=512, mheads=64, groups=1, side=256, vocab=32768, like="qwen3-1.7B"),
     "4096": dict(width=4096, ff=12288, heads=32, q_rank=1536, kv_rank=512, mheads=128, groups=8, side=256, vocab=32768, like="qwen3-8B"),
 }
+MODELS = {"rokivik": ("rokivik", "qwen3"), "pesanex": ("pesanex", "rokivik", "qwen3")}
+# Pesanex: heads of 128 (as many as fill the width); decay rank 16
+KV_HEADS, GLA_DIM, HEAD = 8, 64, 128
 
 
 WINDOW = 2048
@@ -49,6 +54,17 @@ def rokivik_config(s: dict, window: int = WINDOW) -> dict:
             "layers": [mamba(), latent(window), mamba(), latent(window, 1), mamba(), latent(1 << 20)]}
 
 
+def pesanex_config(s: dict) -> dict:
+    h, mlp = s["heads"], {"kind": "dense", "ff": s["ff"]}
+    gla = {"heads": h, "dim": GLA_DIM, "vdim": HEAD, "tau": 16.0}
+    both = {"type": "parallel", "mixer": {"left": {"heads": h, "kv_heads": KV_HEADS, "dim": HEAD, "vdim": HEAD, "scale": HEAD ** 0.5 / 8,
+                                                   "rot": {"base": 10000.0, "dims": 64}}, "right": gla}, "mlp": mlp}
+    keep = {"type": "retention", "mixer": {"heads": h, "dim": HEAD, "vdim": HEAD, "decay": [1 - 2.0 ** -(5 + 7 * k / h) for k in range(h)],
+                                           "rot": {"base": 10000.0, "dims": HEAD}}, "mlp": mlp}
+    return {"architecture": "Pesanex", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "loop": {"start": 0, "stop": 0, "times": 1},
+            "layers": [both, keep, {"type": "gla", "mixer": gla, "mlp": mlp}] * 2}
+
+
 def peaks() -> dict:
     try:
         return json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
@@ -61,8 +77,8 @@ def build(kind: str, size: str, max_running: int, max_len: int, max_prefill: int
     from miles_b200.models import ModelConfig, ParamStore, build_model, get_config
 
     s = SIZES[size]
-    if kind == "rokivik":
-        cfg = ModelConfig.from_hf_config(rokivik_config(s), name=f"rokivik-{size}")
+    if kind != "qwen3":
+        cfg = ModelConfig.from_hf_config({"rokivik": rokivik_config, "pesanex": pesanex_config}[kind](s), name=f"{kind}-{size}")
     else:
         cfg = copy.copy(get_config(s["like"]))
         cfg.num_layers, cfg.vocab_size, cfg.tie_embeddings = 6, s["vocab"], False
@@ -114,7 +130,7 @@ def kernel_table(fn, steps: int = 5) -> dict:
     out: dict = {}
     for ev in prof.events():
         if str(ev.device_type).endswith("CUDA"):
-            name = re.sub(r"\(.*", "", ev.name.replace("(anonymous namespace)::", "").replace("void ", "").replace("mb::", ""))[:70]
+            name = re.sub(r"\(.*", "", re.sub(r"\((int|bool)\)", "", ev.name.replace("(anonymous namespace)::", "").replace("void ", "").replace("mb::", "")))[:70]
             t = out.setdefault(name, [0.0, 0])
             t[0] += ev.device_time_total if hasattr(ev, "device_time_total") else ev.cuda_time_total
             t[1] += 1
@@ -143,7 +159,7 @@ def floors(cfg, kind: str, s: dict, T: int, ctx: int, prefill: bool) -> dict:
             f["chunk_out"] = (T * (2 * inner + 2 * G * N) * 2 + st, 2 * T * hd * (P * N + (c + 1) / 2 * (N + P)))
             f["mamba_tail"] = (T * (3 * inner + 3 * s["ff"]) * 2, 0)
             f["latent_in"] = (T * (2 * (s["q_rank"] + W) + 3 * s["ff"]) * 2, 0)
-            f["latent_prefill"] = (T * h * (192 + 128 + 256) * 2 + T * 64 * 2, 2 * n * L * h * (192 + 128))
+            f["cached_prefill"] = (T * h * (192 + 128 + 256) * 2 + T * 64 * 2, 2 * n * L * h * (192 + 128))
             f["gather_rows"] = (2 * T * W * 2, 0)
             f["pad_q"] = (2 * T * h * 192 * 2, 0)
             f["side_finish"] = (T * H * (4 + 8 + 2), 0)
@@ -154,11 +170,36 @@ def floors(cfg, kind: str, s: dict, T: int, ctx: int, prefill: bool) -> dict:
             f["step_kernel"] = (T * (hd * P * N * 8 + ch * 2 * 5 + inner * 2), 0)
             f["mamba_tail"] = (T * (3 * inner + 3 * s["ff"]) * 2, 0)
             f["latent_in"] = (T * (2 * (s["q_rank"] + W) + 3 * s["ff"]) * 2, 0)
-            f["latent_decode"] = (T * L * W * 2 + T * h * (W * 2 + R * 4), 2 * T * L * h * (W + R))
+            f["cached_decode"] = (T * L * W * 2 + T * h * (W * 2 + R * 4), 2 * T * L * h * (W + R))
             f["absorb_q"] = (h * 128 * R * 2 + T * h * (192 + W) * 2, 2 * T * h * 128 * R)
             f["latent_up"] = (h * 128 * R * 2 + T * h * (R * 4 + 128 * 2), 2 * T * h * 128 * R)
             f["absorb_mma"], f["up_mma"] = f["absorb_q"], f["latent_up"]
             f["side_fused"] = (2 * s["side"] * H * 2 + T * H * (4 + 4 + 4 + 2), 4 * T * s["side"] * H)
+    elif kind == "pesanex":
+        h, D, ff, c = s["heads"], HEAD, s["ff"], 128
+        inner, attn = h * D, T * (2 * h + 2 * KV_HEADS) * D * 2  # (q, k, v in, q and the cache row out; or q, k, v in, result out)
+        f["sandwich_kernel"] = (T * H * (14 + 4 * 2 / 12), 0)    # residual in and out, a result, the normed row; two results in 2 of 12
+        f["gated_act"] = (T * ff * 2 * 3, 0)
+        if prefill:
+            n, L = T // ctx, sum(range(1, ctx + 1))
+            chunks = n * ((ctx + c - 1) // c)
+            for state, out, one_pass, N in (("lin_state", "lin_out", "chunk_pass_kernel<4, true>", GLA_DIM), ("chunk_state", "chunk_out", "chunk_pass_kernel<4, false>", D)):
+                st, sums = chunks * inner * N * 4, T * h * N * 4 if N == GLA_DIM else 0
+                f[state] = (T * h * (N + D) * 2 + sums + st, 2 * T * inner * N)
+                f[out] = (T * h * (2 * N + 2 * D) * 2 + sums + st, 2 * T * h * (D * N + (c + 1) / 2 * (N + D)))
+                f[one_pass] = (2 * st, 0)
+            f["gate_kernel"] = (T * (h * GLA_DIM * 4 + 32), 0)
+            f["lin_tail"] = (T * 3 * inner * 2, 0)
+            f["head_rows"] = ((attn + T * 4 * inner * 2) / 2, 0)  # (mean of attention and of retention, whose q and k go in and out)
+            f["gather_rows"] = (2 * T * 2 * KV_HEADS * D * 2, 0)
+            f["cached_prefill"] = (attn, 4 * n * L * h * D)
+            f["embed"] = (T * H * 8, 0)
+        else:
+            for lanes, N in ((16, GLA_DIM), (32, D)):  # gated, retention
+                f[f"lin_step_kernel<__nv_bfloat16, {lanes}>"] = (T * (inner * N * 8 + h * (2 * N + 3 * D) * 2), 0)
+            f["head_rows"] = (attn, 0)
+            f["cached_decode"] = (T * ctx * 2 * KV_HEADS * D * 2 + T * inner * (2 + 4), 4 * T * ctx * inner)
+            f["merge_kernel"] = (T * inner * (4 + 2), 0)
     else:
         hq, hk = cfg.num_q_heads, cfg.num_kv_heads
         if prefill:
@@ -187,14 +228,14 @@ def report_kernels(tag: dict, table: dict, fl: dict, pk: dict) -> None:
             print(json.dumps(row), flush=True)
 
 
-def run(sizes: list, steps: int, warmup: int, kernels: bool, prompts: list, batches: list, ctx: int) -> None:
+def run(design: str, sizes: list, steps: int, warmup: int, kernels: bool, prompts: list, batches: list, ctx: int) -> None:
     from miles_b200.engine import SamplingParams
 
     pk = peaks()
     for size in sizes:
-        for kind in ("rokivik", "qwen3"):
+        for kind in MODELS[design]:
             cfg, model, eng = build(kind, size, max(max(batches), 8192 // min(prompts) + 1), max(ctx + 1024, max(prompts)), max(16384, max(prompts)))
-            name = cfg.name if kind == "rokivik" else f"{SIZES[size]['like']} layers x 6"
+            name = cfg.name if kind != "qwen3" else f"{SIZES[size]['like']} layers x 6"
             base = {"model": name, "params_m": round(cfg.num_params() / 1e6), "layers": cfg.num_layers, "dtype": "bf16", "data": "random tokens and weights",
                     "l2": "weights larger than L2"}
             for n in prompts:
@@ -229,6 +270,7 @@ def run(sizes: list, steps: int, warmup: int, kernels: bool, prompts: list, batc
 
 def main(argv=None, steps: int = 10, warmup: int = 3) -> None:
     ap = argparse.ArgumentParser()
+    ap.add_argument("--design", choices=list(MODELS), default="rokivik")
     ap.add_argument("--sizes", default="2048,4096")
     ap.add_argument("--steps", type=int, default=steps)
     ap.add_argument("--warmup", type=int, default=warmup)
@@ -238,7 +280,7 @@ def main(argv=None, steps: int = 10, warmup: int = 3) -> None:
     ap.add_argument("--kernels", action="store_true", help="per-kernel device times next to their byte / operation floors")
     ns = ap.parse_args(argv)
     ints = lambda s: [int(v) for v in s.split(",")]
-    run(ns.sizes.split(","), ns.steps, ns.warmup, ns.kernels, ints(ns.prompts), ints(ns.batches), ns.ctx)
+    run(ns.design, ns.sizes.split(","), ns.steps, ns.warmup, ns.kernels, ints(ns.prompts), ints(ns.batches), ns.ctx)
 
 
 if __name__ == "__main__":

@@ -318,47 +318,71 @@ size_t decode_smem(int MT, const HyAttend& a) {
   return sizeof(bf16) * (static_cast<size_t>(2) * TOK * (row_cols(a) + 8) + MT * 16 * (key_cols(a) + 8) + MT * 16 * PLD) + sizeof(float) * 2 * DW * MT * 16;
 }
 
-// Outputs of the splits -> rows of out (pitch ldc): a warp per (row, head), the sink counted once.
+// Outputs of the splits -> rows of out (pitch ldc), the sink counted once: a block of MW warps per (row, head), each warp adding its
+// share of the splits.
+constexpr int MW = 4;
+
 template <typename T>
-__global__ void __launch_bounds__(256) merge_kernel(const HyAttend a, const float* __restrict__ o, const float* __restrict__ ml, int splits,
-                                                    int n, T* __restrict__ out, int ldc) {
-  const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (unit >= n * a.heads) return;
+__global__ void __launch_bounds__(MW * 32) merge_kernel(const HyAttend a, const float* __restrict__ o, const float* __restrict__ ml, int splits,
+                                                        T* __restrict__ out, int ldc) {
+  __shared__ float coef[64];
+  __shared__ __align__(16) float part[MW][128];
+  const int unit = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = unit / a.heads, h = unit - t * a.heads;
-  const float* p = ml + static_cast<long long>(unit) * splits * 2;
-  const float sink = a.sink ? to_f(static_cast<const T*>(a.sink)[h]) * LOG2E : -FLT_MAX;
-  float mv[2], lv[2], m = sink;
+  if (warp == 0) {
+    const float* p = ml + static_cast<long long>(unit) * splits * 2;
+    const float sink = a.sink ? to_f(static_cast<const T*>(a.sink)[h]) * LOG2E : -FLT_MAX;
+    float mv[2], lv[2], m = sink;
 #pragma unroll
-  for (int k = 0; k < 2; ++k) {
-    const int s = lane + 32 * k;
-    mv[k] = s < splits ? p[2 * s] : -FLT_MAX;
-    lv[k] = s < splits ? p[2 * s + 1] : 0.f;
-    m = fmaxf(m, mv[k]);
+    for (int k = 0; k < 2; ++k) {
+      const int s = lane + 32 * k;
+      mv[k] = s < splits ? p[2 * s] : -FLT_MAX;
+      lv[k] = s < splits ? p[2 * s + 1] : 0.f;
+      m = fmaxf(m, mv[k]);
+    }
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, off));
+    float c[2], l = 0.f;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      c[k] = mv[k] == -FLT_MAX ? 0.f : exp2f(mv[k] - m);
+      l += c[k] * lv[k];
+    }
+    l = warp_sum(l) + (a.sink ? exp2f(sink - m) : 0.f);
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) coef[lane + 32 * k] = c[k] * inv;
   }
-#pragma unroll
-  for (int off = 16; off > 0; off >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, off));
-  float c[2], l = 0.f;
-#pragma unroll
-  for (int k = 0; k < 2; ++k) {
-    c[k] = mv[k] == -FLT_MAX ? 0.f : exp2f(mv[k] - m);
-    l += c[k] * lv[k];
-  }
-  l = warp_sum(l) + (a.sink ? exp2f(sink - m) : 0.f);
-  const float inv = l > 0.f ? 1.f / l : 0.f;
   const float* src = o + static_cast<long long>(unit) * splits * a.vd;
   T* dst = out + static_cast<long long>(t) * ldc + h * a.vd;
-  for (int i0 = 0; i0 < a.vd; i0 += 32) {
-    const int i = i0 + lane;
-    float v = 0.f;
-#pragma unroll 4
-    for (int s = 0; s < splits; ++s) {
-      const float w = __shfl_sync(0xffffffffu, s < 32 ? c[0] : c[1], s & 31);
-      if (i < a.vd) v += w * src[static_cast<long long>(s) * a.vd + i];
+  for (int i0 = 0; i0 < a.vd; i0 += 128) {  // (vd is a multiple of 8)
+    const int i = i0 + lane * 4;
+    float4 u[4], v = make_float4(0.f, 0.f, 0.f, 0.f);
+    const bool live = i < a.vd;
+    for (int s0 = warp; s0 < splits; s0 += 4 * MW) {
+#pragma unroll
+      for (int k = 0; k < 4; ++k)
+        u[k] = live && s0 + k * MW < splits ? *reinterpret_cast<const float4*>(src + static_cast<long long>(s0 + k * MW) * a.vd + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      if (s0 == warp) __syncthreads();  // coefficients (first time round) and the partial sums of the columns before
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float c = coef[min(s0 + k * MW, 63)];
+        v.x += c * u[k].x; v.y += c * u[k].y; v.z += c * u[k].z; v.w += c * u[k].w;
+      }
     }
-    if (i < a.vd) dst[i] = from_f<T>(v * inv);
+    if (warp >= splits) __syncthreads();
+    *reinterpret_cast<float4*>(&part[warp][lane * 4]) = v;
+    __syncthreads();
+    const int c = threadIdx.x;
+    if (i0 + c < a.vd) {
+      float r = 0.f;
+#pragma unroll
+      for (int w = 0; w < MW; ++w) r += part[w][c];
+      dst[i0 + c] = from_f<T>(r);
+    }
   }
   if (h == a.heads - 1)
-    for (int i = a.heads * a.vd + lane; i < ldc; i += 32) out[static_cast<long long>(t) * ldc + i] = from_f<T>(0.f);
+    for (int i = a.heads * a.vd + threadIdx.x; i < ldc; i += MW * 32) out[static_cast<long long>(t) * ldc + i] = from_f<T>(0.f);
 }
 
 // ------------------------------------------------------------------------------------------------ rows of a range
@@ -434,9 +458,8 @@ int hy_decode(const HyAttend& a, const void* ql, int qld, const int* seq_lens, i
 
 int hy_decode_merge(bool f32, const HyAttend& a, const float* o, const float* ml, int splits, int B, void* out, int ldc, cudaStream_t s) {
   if (splits < 1 || splits > 64) return static_cast<int>(cudaErrorInvalidValue);
-  const int blocks = (B * a.heads + 7) / 8;
-  if (f32) merge_kernel<float><<<blocks, 256, 0, s>>>(a, o, ml, splits, B, static_cast<float*>(out), ldc);
-  else merge_kernel<bf16><<<blocks, 256, 0, s>>>(a, o, ml, splits, B, static_cast<bf16*>(out), ldc);
+  if (f32) merge_kernel<float><<<B * a.heads, MW * 32, 0, s>>>(a, o, ml, splits, static_cast<float*>(out), ldc);
+  else merge_kernel<bf16><<<B * a.heads, MW * 32, 0, s>>>(a, o, ml, splits, static_cast<bf16*>(out), ldc);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -222,6 +222,8 @@ struct HyHeadRows {
   long long num_slots;
   float eps;
   int* status;
+  float2* turns[3];      // work for many rows: [T, rot / 2] (cosine, sine) per operation, written where `fill` says so; or null
+  bool fill[3];
 };
 int hy_head_rows(bool f32, const HyHeadRows& a, int T, cudaStream_t s);
 // out[t] = act(gate) * up, zeros up to ldo. act: 0 silu, 1 relu

@@ -317,6 +317,27 @@ void latent_prefill(LATENT_ARGS, const at::Tensor& q, const at::Tensor& position
 // after the last head, destination rows by slot)
 typedef std::tuple<int64_t, int64_t, int64_t, int64_t, OptT, bool, double, at::Tensor, int64_t, int64_t, int64_t, bool> HeadOp;
 
+// For many rows: room for the angles of every operation, one table for operations that turn alike.
+at::Tensor add_turns(mb::HyHeadRows& a, int64_t T, const at::Tensor& like) {
+  at::Tensor work;
+  if (T <= 512) return work;
+  int64_t total = 0, at[3];
+  int same[3];
+  for (int i = 0; i < a.n; ++i) {
+    same[i] = i;
+    for (int j = 0; j < i; ++j)
+      if (a.op[j].freq == a.op[i].freq && a.op[j].rot == a.op[i].rot) { same[i] = j; break; }
+    at[i] = same[i] < i ? at[same[i]] : total;
+    if (same[i] == i) total += T * (a.op[i].rot / 2);
+  }
+  work = at::empty({total, 2}, like.options().dtype(at::kFloat));
+  for (int i = 0; i < a.n; ++i) {
+    a.turns[i] = reinterpret_cast<float2*>(work.data_ptr<float>()) + at[i];
+    a.fill[i] = same[i] == i && a.op[i].rot > 0;
+  }
+  return work;
+}
+
 void head_rows(const at::Tensor& proj, const at::Tensor& positions, const OptT& slots, double eps, at::Tensor& status, const std::vector<HeadOp>& ops) {
   const bool f = is_f32(proj);
   SAME(proj, f); CHECK_I32(positions); CHECK_I32(status);
@@ -345,6 +366,7 @@ void head_rows(const at::Tensor& proj, const at::Tensor& positions, const OptT& 
     }
   }
   const c10::cuda::CUDAGuard guard(proj.device());
+  const at::Tensor work = add_turns(a, T, proj);
   RUN(mb::hy_head_rows(f, a, T, cur_stream()));
 }
 
@@ -502,6 +524,7 @@ void linear_prefill(LIN_ARGS, const at::Tensor& positions, const at::Tensor& cu,
       o.scale = i == 0 ? 1.f : a.k_scale;
       o.dst = proj.data_ptr(); o.ld = a.ld;
     }
+    const at::Tensor work = add_turns(r, T, proj);
     RUN(mb::hy_head_rows(f, r, T, s));
   }
   at::Tensor y = at::empty({T, heads * P}, proj.options()), gate;

@@ -78,6 +78,12 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 }
 
 __device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+// the same for values that are rounded to T: bf16 rows take the approximate exponential and quotient
+template <typename T>
+__device__ __forceinline__ float silu_t(float z) {
+  if constexpr (sizeof(T) == 2) return __fdividef(z, 1.f + __expf(-z));
+  else return silu_f(z);
+}
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));

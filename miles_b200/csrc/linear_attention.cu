@@ -26,14 +26,25 @@ using namespace hy;
 __device__ __forceinline__ float log_sigmoid(float z) { return -softplus_f(-z); }
 
 // ------------------------------------------------------------------------------------------------ decays of all rows
-// Block: 128 channels of up to ROWS-row tiles of a stretch of rows. SUM: a stretch is a chunk, out = running sum of log2 a over it;
-// else out = a - 1. RK > 0: the channel's weights sit in registers (rank <= RK).
-constexpr int GROWS = 32;
+// Block: GC channels of a stretch of up to 128 rows, which GG groups of threads share. SUM: a stretch is a chunk, out = running sum of
+// log2 a over it; else out = a - 1. RK > 0: the channel's weights sit in registers (rank <= RK).
+constexpr int GC = 64, GG = 8, GROWS = HY_CHUNK / GG;
+
+// log2 a = log2(sigmoid(z)) / tau. softplus(-z) = max(-z, 0) + log1p(exp(-|z|)); below 1/16 the logarithm comes from its series (an
+// approximate one loses its digits near 1, and slow decays are made of them).
+__device__ __forceinline__ float log2_sigmoid(float z) {
+  const float e = ex2(-fabsf(z) * LOG2E);
+  float l;
+  if (e < 0.0625f) l = e * (1.f - e * (0.5f - e * (1.f / 3.f - e * (0.25f - e * (0.2f - e * (1.f / 6.f)))))) * LOG2E;
+  else l = __log2f(1.f + e);
+  return -(fmaxf(-z, 0.f) * LOG2E + l);
+}
 
 template <typename T, int RK, bool SUM>
-__global__ void __launch_bounds__(128) gate_kernel(const HyLinear a, const int4* __restrict__ chunks, int n_rows, float* __restrict__ out) {
-  extern __shared__ __align__(16) float us[];  // [GROWS][rank]
-  const int ch = a.heads * a.N, c = blockIdx.y * 128 + threadIdx.x, rank = a.rank;
+__global__ void __launch_bounds__(GG * GC) gate_kernel(const HyLinear a, const int4* __restrict__ chunks, int n_rows, float* __restrict__ out, bool vec) {
+  extern __shared__ __align__(16) float us[];  // [128][rank]
+  __shared__ float ends[GG][GC];
+  const int lane_c = threadIdx.x & (GC - 1), group = threadIdx.x / GC, ch = a.heads * a.N, c = blockIdx.y * GC + lane_c, rank = a.rank;
   const bool live = c < ch;
   int row0, n;
   if constexpr (SUM) {
@@ -41,48 +52,82 @@ __global__ void __launch_bounds__(128) gate_kernel(const HyLinear a, const int4*
     row0 = ck.y;
     n = ck.z;
   } else {
-    row0 = blockIdx.x * GROWS;
-    n = min(GROWS, n_rows - row0);
+    row0 = blockIdx.x * HY_CHUNK;
+    n = min(HY_CHUNK, n_rows - row0);
   }
+  const int ldu = RK > 0 ? RK : rank;
   const T* w = static_cast<const T*>(a.a2) + static_cast<long long>(live ? c : 0) * rank;
-  float wr[RK > 0 ? RK : 1];
-  if constexpr (RK > 0) {
+  __align__(8) float wr[RK > 0 ? RK : 2];
+  constexpr int V = Vec<T>::N;
+  if (RK > 0 && vec) {  // (rank a multiple of V, 16-byte aligned rows)
+    if constexpr (RK > 0) {
 #pragma unroll
-    for (int r = 0; r < RK; ++r) wr[r] = r < rank ? to_f(w[r]) : 0.f;
+      for (int r = 0; r < RK; r += V) {
+        float x[V];
+#pragma unroll
+        for (int j = 0; j < V; ++j) x[j] = 0.f;
+        if (r < rank) Vec<T>::load(w + r, x);
+#pragma unroll
+        for (int j = 0; j < V; ++j) wr[r + j] = x[j];
+      }
+      for (int i = threadIdx.x; i < n * (RK / V); i += GG * GC) {
+        const int t = i / (RK / V), r = (i - t * (RK / V)) * V;
+        float x[V];
+#pragma unroll
+        for (int j = 0; j < V; ++j) x[j] = 0.f;
+        if (r < rank) Vec<T>::load(static_cast<const T*>(a.proj) + (row0 + t) * a.ld + a.u + r, x);
+#pragma unroll
+        for (int j = 0; j < V; j += 4) *reinterpret_cast<float4*>(us + t * RK + r + j) = make_float4(x[j], x[j + 1], x[j + 2], x[j + 3]);
+      }
+    }
+  } else {
+    if constexpr (RK > 0) {
+#pragma unroll
+      for (int r = 0; r < RK; ++r) wr[r] = r < rank ? to_f(w[r]) : 0.f;
+    }
+    for (int i = threadIdx.x; i < n * ldu; i += GG * GC) {
+      const int t = i / ldu, r = i - t * ldu;
+      us[i] = r < rank ? to_f(static_cast<const T*>(a.proj)[(row0 + t) * a.ld + a.u + r]) : 0.f;
+    }
   }
   const float bias = live ? to_f(static_cast<const T*>(a.a2_bias)[c]) : 0.f;
-  const float scale = SUM ? a.inv_tau * LOG2E : a.inv_tau;
-  float run = 0.f;
-  for (int t0 = 0; t0 < n; t0 += GROWS) {
-    const int m = min(GROWS, n - t0);
-    __syncthreads();
-    const int ldu = RK > 0 ? RK : rank;
-    for (int i = threadIdx.x; i < m * ldu; i += 128) {
-      const int t = i / ldu, r = i - t * ldu;
-      us[i] = r < rank ? to_f(static_cast<const T*>(a.proj)[(row0 + t0 + t) * a.ld + a.u + r]) : 0.f;
-    }
-    __syncthreads();
-    if (!live) continue;
-#pragma unroll 4
-    for (int t = 0; t < m; ++t) {
-      float z = bias;
-      if constexpr (RK > 0) {
+  __syncthreads();
+  const int t0 = group * GROWS, m = min(GROWS, n - t0);
+  auto z_of = [&](int t) {
+    if constexpr (RK > 0) {  // two products an instruction
+      float2 z = make_float2(bias, 0.f);
 #pragma unroll
-        for (int r = 0; r < RK; r += 4) {
-          const float4 u = *reinterpret_cast<const float4*>(us + t * RK + r);
-          z += wr[r] * u.x + wr[r + 1] * u.y + wr[r + 2] * u.z + wr[r + 3] * u.w;
-        }
-      } else {
-        for (int r = 0; r < rank; ++r) z += to_f(w[r]) * us[t * rank + r];
+      for (int r = 0; r < RK; r += 4) {
+        const float4 u = *reinterpret_cast<const float4*>(us + t * RK + r);
+        z = __ffma2_rn(make_float2(wr[r], wr[r + 1]), make_float2(u.x, u.y), z);
+        z = __ffma2_rn(make_float2(wr[r + 2], wr[r + 3]), make_float2(u.z, u.w), z);
       }
-      const float l = log_sigmoid(z) * scale;
-      if constexpr (SUM) {
-        run += l;
-        out[static_cast<long long>(row0 + t0 + t) * ch + c] = run;
-      } else {
-        out[static_cast<long long>(row0 + t0 + t) * ch + c] = expm1f(l);
-      }
+      return z.x + z.y;
+    } else {
+      float z = bias;
+      for (int r = 0; r < rank; ++r) z += to_f(w[r]) * us[t * rank + r];
+      return z;
     }
+  };
+  float* dst = out + static_cast<long long>(row0 + t0) * ch + c;
+  if constexpr (SUM) {
+    float run = 0.f, v[GROWS];
+#pragma unroll
+    for (int t = 0; t < GROWS; ++t) {
+      if (t < m) run += log2_sigmoid(z_of(t0 + t)) * a.inv_tau;
+      v[t] = run;
+    }
+    ends[group][lane_c] = run;
+    __syncthreads();
+    float base = 0.f;
+    for (int g = 0; g < group; ++g) base += ends[g][lane_c];
+    if (!live) return;
+#pragma unroll
+    for (int t = 0; t < GROWS; ++t)
+      if (t < m) dst[static_cast<long long>(t) * ch] = base + v[t];
+  } else {
+    if (!live) return;
+    for (int t = 0; t < m; ++t) dst[static_cast<long long>(t) * ch] = expm1f(log_sigmoid(z_of(t0 + t)) * a.inv_tau);
   }
 }
 
@@ -125,41 +170,62 @@ __global__ void __launch_bounds__(256) lin_scan_kernel(const HyLinear a, const f
 }
 
 // ------------------------------------------------------------------------------------------------ output norm and gate
-// A warp per (row, head).
-template <typename T, bool V2>
-__global__ void __launch_bounds__(256) lin_tail_kernel(const HyLinear a, const T* __restrict__ y, T* __restrict__ out, int ldc, long long units) {
-  const long long unit = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+// A warp per (row, head). V4: four values per access.
+template <typename T>
+__device__ __forceinline__ float4 load4(const T* p) {
+  if constexpr (sizeof(T) == 2) {
+    const uint2 q = *reinterpret_cast<const uint2*>(p);
+    const float2 x = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.x)), y = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&q.y));
+    return make_float4(x.x, x.y, y.x, y.y);
+  } else {
+    return *reinterpret_cast<const float4*>(p);
+  }
+}
+template <typename T>
+__device__ __forceinline__ void store4(T* p, float4 v) {
+  if constexpr (sizeof(T) == 2) {
+    const __nv_bfloat162 x = __floats2bfloat162_rn(v.x, v.y), y = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&x), *reinterpret_cast<const uint32_t*>(&y));
+  } else {
+    *reinterpret_cast<float4*>(p) = v;
+  }
+}
+
+template <typename T, bool V4>
+__global__ void __launch_bounds__(256) lin_tail_kernel(const HyLinear a, const T* __restrict__ y, T* __restrict__ out, int ldc, unsigned units) {
+  const unsigned unit = blockIdx.x * 8 + (threadIdx.x >> 5);
   if (unit >= units) return;
   const int lane = threadIdx.x & 31, P = a.P;
-  const long long t = unit / a.heads;
-  const int h = static_cast<int>(unit - t * a.heads);
-  const T* src = y + unit * P;
+  const unsigned row = unit / static_cast<unsigned>(a.heads);
+  const int h = static_cast<int>(unit - row * a.heads);
+  const long long t = row;
+  const T* src = y + static_cast<long long>(unit) * P;
   const T* g = static_cast<const T*>(a.proj) + t * a.ld + a.g + h * P;
   const T* w = static_cast<const T*>(a.norm);
   T* dst = out + t * ldc + h * P;
   float s = 0.f;
-  if constexpr (V2) {
-    auto two = [](const T* p) {
-      if constexpr (sizeof(T) == 2) return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
-      else return *reinterpret_cast<const float2*>(p);
-    };
-    for (int i = lane * 2; i < P; i += 64) {
-      const float2 v = two(src + i);
-      s += v.x * v.x + v.y * v.y;
+  if constexpr (V4) {
+    float4 v0 = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (lane * 4 < P) v0 = load4(src + lane * 4);
+    float4 z0 = make_float4(0.f, 0.f, 0.f, 0.f), w0 = make_float4(1.f, 1.f, 1.f, 1.f);  // (of the first 128 columns, fetched before the sum)
+    if (lane * 4 < P) {
+      z0 = load4(g + lane * 4);
+      if (w) w0 = load4(w + lane * 4);
     }
-    const float r = 1.f / sqrtf(warp_sum(s) / static_cast<float>(P) + a.eps);
-    for (int i = lane * 2; i < P; i += 64) {
-      float2 v = two(src + i);
-      const float2 z = two(g + i);
-      v.x *= r * silu_f(z.x);
-      v.y *= r * silu_f(z.y);
-      if (w) {
-        const float2 q = two(w + i);
-        v.x *= q.x;
-        v.y *= q.y;
-      }
-      if constexpr (sizeof(T) == 2) *reinterpret_cast<__nv_bfloat162*>(dst + i) = __floats2bfloat162_rn(v.x, v.y);
-      else *reinterpret_cast<float2*>(dst + i) = v;
+    s = v0.x * v0.x + v0.y * v0.y + v0.z * v0.z + v0.w * v0.w;
+    for (int i = 128 + lane * 4; i < P; i += 128) {
+      const float4 v = load4(src + i);
+      s += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    const float r = sizeof(T) == 2 ? rsqrtf(warp_sum(s) / static_cast<float>(P) + a.eps) : 1.f / sqrtf(warp_sum(s) / static_cast<float>(P) + a.eps);
+    for (int i = lane * 4; i < P; i += 128) {
+      float4 v = i < 128 ? v0 : load4(src + i);
+      const float4 z = i < 128 ? z0 : load4(g + i), q = i < 128 ? w0 : (w ? load4(w + i) : make_float4(1.f, 1.f, 1.f, 1.f));
+      v.x *= r * q.x * silu_t<T>(z.x);
+      v.y *= r * q.y * silu_t<T>(z.y);
+      v.z *= r * q.z * silu_t<T>(z.z);
+      v.w *= r * q.w * silu_t<T>(z.w);
+      store4(dst + i, v);
     }
   } else {
     for (int i = lane; i < P; i += 32) s += to_f(src[i]) * to_f(src[i]);
@@ -171,10 +237,11 @@ __global__ void __launch_bounds__(256) lin_tail_kernel(const HyLinear a, const T
 }
 
 // ------------------------------------------------------------------------------------------------ one token
-// CTA = (head, sequence). Queries, keys and decays of the head, then the state update (a warp walks the rows p; VEC4: every lane owns 4
-// consecutive columns of a 128-wide block), then the head's output norm and gate.
-template <typename T, bool VEC4>
-__global__ void __launch_bounds__(256) lin_step_kernel(const HyLinear a, const int* __restrict__ positions, T* __restrict__ out, int ldc) {
+// CTA = (head, sequence). Queries, keys and decays of the head, then the state update, then the head's output norm and gate. LPR > 0: LPR
+// lanes own a state row, four columns each (N <= 4 LPR, a multiple of 4); the first U rows of every lane group are fetched before
+// anything else. LPR = 0: any N.
+template <typename T, int LPR>
+__global__ void __launch_bounds__(LPR > 0 ? 512 : 256, 2) lin_step_kernel(const HyLinear a, const int* __restrict__ positions, T* __restrict__ out, int ldc) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[33];
   const int h = blockIdx.x, b = blockIdx.y, P = a.P, N = a.N, Np = (N + 3) & ~3;
@@ -188,6 +255,21 @@ __global__ void __launch_bounds__(256) lin_step_kernel(const HyLinear a, const i
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const bool fresh = pos <= 0;
   const int half = a.rot / 2;
+  constexpr int U = 8;
+  constexpr int RPW = LPR > 0 ? 32 / LPR : 1;  // rows a warp works on at once
+  const int sub = lane & (LPR > 0 ? LPR - 1 : 0), c = sub * 4, row_of = warp * RPW + (LPR > 0 ? lane / LPR : 0), rows = nw * RPW;
+  const bool own = c < N;
+  float4 s[LPR > 0 ? U : 1];
+  float v[LPR > 0 ? U : 1];
+  auto fetch = [&](int p0) {
+#pragma unroll
+    for (int j = 0; j < U; ++j) {
+      const int p = p0 + j * rows;
+      s[LPR > 0 ? j : 0] = own && !fresh && p < P ? *reinterpret_cast<const float4*>(st + static_cast<long long>(p) * N + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      v[LPR > 0 ? j : 0] = p < P ? to_f(vr[p]) : 0.f;
+    }
+  };
+  if constexpr (LPR > 0) fetch(row_of);
   for (int i = threadIdx.x; i < a.rank; i += blockDim.x) u[i] = to_f(pr[a.u + i]);
   // (what the chunked and sequential forms read back from rotated rows is rounded there; here it is rounded the same way)
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
@@ -204,17 +286,19 @@ __global__ void __launch_bounds__(256) lin_step_kernel(const HyLinear a, const i
     k[i] = a.k_scale == 1.f ? to_f(kr[i]) : to_f(from_f<T>(to_f(kr[i]) * a.k_scale));
   }
   if (a.rank > 0) {
-    __syncthreads();
-    for (int i = threadIdx.x; i < N; i += blockDim.x) {
-      const int c = h * N + i;
-      const T* w = static_cast<const T*>(a.a2) + static_cast<long long>(c) * a.rank;
-      float z = to_f(static_cast<const T*>(a.a2_bias)[c]);
-      constexpr int V = Vec<T>::N;
+    constexpr int V = Vec<T>::N;
+    const bool vec = a.rank % V == 0;
+    for (int i0 = 0; i0 < N; i0 += blockDim.x) {
+      const int i = i0 + threadIdx.x, ch = h * N + min(i, N - 1);
+      const T* w = static_cast<const T*>(a.a2) + static_cast<long long>(ch) * a.rank;
+      float z = to_f(static_cast<const T*>(a.a2_bias)[ch]), x[V];
+      if (vec) Vec<T>::load(w, x);  // (in flight over the barrier)
+      if (i0 == 0) __syncthreads();
+      if (i >= N) continue;
       int r = 0;
-      if (a.rank % V == 0)
+      if (vec)
         for (; r < a.rank; r += V) {
-          float x[V];
-          Vec<T>::load(w + r, x);
+          if (r > 0) Vec<T>::load(w + r, x);
 #pragma unroll
           for (int j = 0; j < V; ++j) z += x[j] * u[r + j];
         }
@@ -225,48 +309,42 @@ __global__ void __launch_bounds__(256) lin_step_kernel(const HyLinear a, const i
     for (int i = threadIdx.x; i < N; i += blockDim.x) e[i] = a.decay_m1[h];
   }
   __syncthreads();
-  if constexpr (VEC4) {
-    constexpr int U = 4;  // rows in flight per warp
-    for (int p0 = warp * U; p0 < P; p0 += nw * U) {
-      float acc[U], v[U];
+  if constexpr (LPR > 0) {
+    float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), qv = kv, ev = kv;
+    if (own) {
+      kv = *reinterpret_cast<const float4*>(k + c);
+      qv = *reinterpret_cast<const float4*>(q + c);
+      ev = *reinterpret_cast<const float4*>(e + c);
+    }
+    for (int p0 = row_of; p0 - row_of < P; p0 += U * rows) {
+      if (p0 != row_of) fetch(p0);
+      float acc[U];
 #pragma unroll
       for (int j = 0; j < U; ++j) {
-        acc[j] = 0.f;
-        v[j] = p0 + j < P ? to_f(vr[p0 + j]) : 0.f;
-      }
-      for (int c = lane * 4; c < N; c += 128) {
-        float4 s[U];
-#pragma unroll
-        for (int j = 0; j < U; ++j)
-          s[j] = (!fresh && p0 + j < P) ? *reinterpret_cast<const float4*>(st + static_cast<long long>(p0 + j) * N + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-        const float4 kv = *reinterpret_cast<const float4*>(k + c), qv = *reinterpret_cast<const float4*>(q + c), ev = *reinterpret_cast<const float4*>(e + c);
-#pragma unroll
-        for (int j = 0; j < U; ++j) {
-          if (p0 + j >= P) break;
-          s[j].x = fmaf(ev.x, s[j].x, s[j].x) + kv.x * v[j];
-          s[j].y = fmaf(ev.y, s[j].y, s[j].y) + kv.y * v[j];
-          s[j].z = fmaf(ev.z, s[j].z, s[j].z) + kv.z * v[j];
-          s[j].w = fmaf(ev.w, s[j].w, s[j].w) + kv.w * v[j];
-          acc[j] += s[j].x * qv.x + s[j].y * qv.y + s[j].z * qv.z + s[j].w * qv.w;
-          *reinterpret_cast<float4*>(st + static_cast<long long>(p0 + j) * N + c) = s[j];
-        }
+        s[j].x = fmaf(ev.x, s[j].x, s[j].x) + kv.x * v[j];
+        s[j].y = fmaf(ev.y, s[j].y, s[j].y) + kv.y * v[j];
+        s[j].z = fmaf(ev.z, s[j].z, s[j].z) + kv.z * v[j];
+        s[j].w = fmaf(ev.w, s[j].w, s[j].w) + kv.w * v[j];
+        acc[j] = s[j].x * qv.x + s[j].y * qv.y + s[j].z * qv.z + s[j].w * qv.w;
+        if (own && p0 + j * rows < P) *reinterpret_cast<float4*>(st + static_cast<long long>(p0 + j * rows) * N + c) = s[j];
       }
 #pragma unroll
       for (int j = 0; j < U; ++j) {
-        acc[j] = warp_sum(acc[j]);
-        if (lane == 0 && p0 + j < P) o[p0 + j] = acc[j] * a.q_scale;
+#pragma unroll
+        for (int off = LPR / 2; off > 0; off >>= 1) acc[j] += __shfl_xor_sync(0xffffffffu, acc[j], off);
+        if (sub == 0 && p0 + j * rows < P) o[p0 + j * rows] = acc[j] * a.q_scale;
       }
     }
   } else {
     for (int p = warp; p < P; p += nw) {
       float acc = 0.f;
-      const float v = to_f(vr[p]);
+      const float vp = to_f(vr[p]);
       float* row = st + static_cast<long long>(p) * N;
-      for (int c = lane; c < N; c += 32) {
-        const float s0 = fresh ? 0.f : row[c];
-        const float s = fmaf(e[c], s0, s0) + k[c] * v;
-        row[c] = s;
-        acc += s * q[c];
+      for (int i = lane; i < N; i += 32) {
+        const float s0 = fresh ? 0.f : row[i];
+        const float s1 = fmaf(e[i], s0, s0) + k[i] * vp;
+        row[i] = s1;
+        acc += s1 * q[i];
       }
       acc = warp_sum(acc);
       if (lane == 0) o[p] = acc * a.q_scale;
@@ -639,12 +717,13 @@ __global__ void __launch_bounds__(OW * 32, 1) lin_out_kernel(const HyLinear a, c
 // ------------------------------------------------------------------------------------------------ launches
 template <typename T, int RK, bool SUM>
 int gate_rk(const HyLinear& a, const int* chunks, int n_chunks, int rows, float* out, cudaStream_t s) {
-  const size_t smem = sizeof(float) * GROWS * static_cast<size_t>(RK > 0 ? RK : a.rank);
+  const size_t smem = sizeof(float) * HY_CHUNK * static_cast<size_t>(RK > 0 ? RK : a.rank);
   auto kern = gate_kernel<T, RK, SUM>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
-  const unsigned x = SUM ? n_chunks : (rows + GROWS - 1) / GROWS;
-  kern<<<dim3(x, (a.heads * a.N + 127) / 128), 128, smem, s>>>(a, reinterpret_cast<const int4*>(chunks), rows, out);
+  const unsigned x = SUM ? n_chunks : (rows + HY_CHUNK - 1) / HY_CHUNK;
+  const bool vec = a.rank % Vec<T>::N == 0 && a.u % Vec<T>::N == 0 && aligned16<T>(a.proj, a.ld) && aligned16<T>(a.a2, a.rank);
+  kern<<<dim3(x, (a.heads * a.N + GC - 1) / GC), GG * GC, smem, s>>>(a, reinterpret_cast<const int4*>(chunks), rows, out, vec);
   return static_cast<int>(cudaGetLastError());
 }
 template <typename T, bool SUM>
@@ -672,21 +751,30 @@ template <typename T>
 int lin_tail_t(const HyLinear& a, const void* y, int rows, void* out, int ldc, cudaStream_t s) {
   const long long units = static_cast<long long>(rows) * a.heads;
   if (units == 0) return 0;
-  const bool v2 = (a.P | a.g) % 2 == 0 && a.ld % 2 == 0 && ldc % 2 == 0;
+  if (units > 0x7fffffffll) return static_cast<int>(cudaErrorInvalidValue);
+  const bool v4 = (a.P | a.g | ldc) % 4 == 0 && a.ld % 4 == 0;
   const unsigned blocks = static_cast<unsigned>((units + 7) / 8);
-  if (v2) lin_tail_kernel<T, true><<<blocks, 256, 0, s>>>(a, static_cast<const T*>(y), static_cast<T*>(out), ldc, units);
-  else lin_tail_kernel<T, false><<<blocks, 256, 0, s>>>(a, static_cast<const T*>(y), static_cast<T*>(out), ldc, units);
+  if (v4) lin_tail_kernel<T, true><<<blocks, 256, 0, s>>>(a, static_cast<const T*>(y), static_cast<T*>(out), ldc, static_cast<unsigned>(units));
+  else lin_tail_kernel<T, false><<<blocks, 256, 0, s>>>(a, static_cast<const T*>(y), static_cast<T*>(out), ldc, static_cast<unsigned>(units));
   return static_cast<int>(cudaGetLastError());
 }
 
 template <typename T>
 int lin_step_t(const HyLinear& a, const int* positions, int B, void* out, int ldc, cudaStream_t s) {
   const size_t smem = sizeof(float) * (static_cast<size_t>(3) * ((a.N + 3) & ~3) + ((a.P + 3) & ~3) + a.rank);
-  auto kern = a.N % 4 == 0 ? lin_step_kernel<T, true> : lin_step_kernel<T, false>;
-  cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-  if (e != cudaSuccess) return static_cast<int>(e);
-  kern<<<dim3(a.heads, B), 256, smem, s>>>(a, positions, static_cast<T*>(out), ldc);
-  return static_cast<int>(cudaGetLastError());
+  auto go = [&](auto kern, int lpr) -> int {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+    int threads = 256;
+    if (lpr > 0)  // eight rows per lane group, as far as a block reaches
+      for (threads = 128; threads < 512 && threads / lpr * 8 < a.P;) threads *= 2;
+    kern<<<dim3(a.heads, B), threads, smem, s>>>(a, positions, static_cast<T*>(out), ldc);
+    return static_cast<int>(cudaGetLastError());
+  };
+  if (a.N % 4 != 0 || a.N > 128) return go(lin_step_kernel<T, 0>, 0);
+  if (a.N > 64) return go(lin_step_kernel<T, 32>, 32);
+  if (a.N > 32) return go(lin_step_kernel<T, 16>, 16);
+  return go(lin_step_kernel<T, 8>, 8);
 }
 
 size_t state_smem(int PT, int N) { return sizeof(bf16) * Q * (static_cast<size_t>(PT) * 16 + PAD + 2 * ((N + 15) / 16 * 16 + PAD)); }

@@ -186,8 +186,9 @@ class B200Hybrid(TorchHybrid):
         """Input rows of a product with ``width`` columns, of which the mixer fills ``used``."""
         return (torch.empty if used == width else torch.zeros)(T, width, dtype=self.store.dtype, device=self.dev)
 
-    def _decode_splits(self, B: int, groups: int, longest: int) -> int:
-        return max(1, min(self.sms // max(1, B * groups), (longest + 63) // 64, 32))
+    def _decode_splits(self, B: int, groups: int, longest: int, per_sm: int = 1) -> int:
+        """Parts the keys of a decode step are cut into, so that ``per_sm`` blocks find work on every SM."""
+        return max(1, min(per_sm * self.sms // max(1, B * groups), (longest + 63) // 64, 32))
 
     def _attention(self, i, m, side, proj, positions, meta, rows):
         """Softmax attention over cached key / value heads; keys and values of ``proj`` go to their cache rows."""
@@ -219,7 +220,7 @@ class B200Hybrid(TorchHybrid):
         else:
             per_head = m.heads // m.kv_heads
             groups = m.kv_heads * ((per_head + 15) // 16 if per_head <= 16 else (per_head + 31) // 32)
-            C.attn_decode(*args, q, meta.seq_lens, self._decode_splits(T, groups, meta.block_table.shape[1] * meta.page_size), out)
+            C.attn_decode(*args, q, meta.seq_lens, self._decode_splits(T, groups, meta.block_table.shape[1] * meta.page_size, 3), out)
         return out
 
     def _linear_attention(self, i, m, side, proj, positions, meta, state):
