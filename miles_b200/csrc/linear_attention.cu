@@ -243,7 +243,6 @@ __global__ void __launch_bounds__(256) lin_tail_kernel(const HyLinear a, const T
 template <typename T, int LPR>
 __global__ void __launch_bounds__(LPR > 0 ? 512 : 256, 2) lin_step_kernel(const HyLinear a, const int* __restrict__ positions, T* __restrict__ out, int ldc) {
   extern __shared__ __align__(16) float sm[];
-  __shared__ float red[33];
   const int h = blockIdx.x, b = blockIdx.y, P = a.P, N = a.N, Np = (N + 3) & ~3;
   float *q = sm, *k = q + Np, *e = k + Np, *o = e + Np, *u = o + ((P + 3) & ~3);  // u [rank]
   const int pos = positions[b];
@@ -270,6 +269,13 @@ __global__ void __launch_bounds__(LPR > 0 ? 512 : 256, 2) lin_step_kernel(const 
     }
   };
   if constexpr (LPR > 0) fetch(row_of);
+  // gate and norm weight of this thread's (first) value, needed last
+  const T *g = pr + a.g + h * P, *wn = static_cast<const T*>(a.norm);
+  float gv = 0.f, wv = 1.f;
+  if (static_cast<int>(threadIdx.x) < P) {
+    gv = to_f(g[threadIdx.x]);
+    if (wn) wv = to_f(wn[threadIdx.x]);
+  }
   for (int i = threadIdx.x; i < a.rank; i += blockDim.x) u[i] = to_f(pr[a.u + i]);
   // (what the chunked and sequential forms read back from rotated rows is rounded there; here it is rounded the same way)
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
@@ -351,13 +357,17 @@ __global__ void __launch_bounds__(LPR > 0 ? 512 : 256, 2) lin_step_kernel(const 
     }
   }
   __syncthreads();
-  float ss = 0.f;
-  for (int p = threadIdx.x; p < P; p += blockDim.x) ss += o[p] * o[p];
-  const float r = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(P) + a.eps);
-  const T* g = pr + a.g + h * P;
+  float ss = 0.f;  // (every warp adds up all of the head)
+  for (int p = lane; p < P; p += 32) ss += o[p] * o[p];
+  const float r = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(P) + a.eps);
   T* dst = out + static_cast<long long>(b) * ldc;
-  for (int p = threadIdx.x; p < P; p += blockDim.x)
-    dst[h * P + p] = from_f<T>(o[p] * r * (a.norm ? to_f(static_cast<const T*>(a.norm)[p]) : 1.f) * silu_f(to_f(g[p])));
+  for (int p = threadIdx.x; p < P; p += blockDim.x) {
+    if (p >= static_cast<int>(blockDim.x)) {
+      gv = to_f(g[p]);
+      if (wn) wv = to_f(wn[p]);
+    }
+    dst[h * P + p] = from_f<T>(o[p] * r * wv * silu_f(gv));
+  }
   if (h == a.heads - 1)
     for (int i = a.heads * P + threadIdx.x; i < ldc; i += blockDim.x) dst[i] = from_f<T>(0.f);
 }

@@ -162,8 +162,8 @@ class LinearAttention:
 
 @dataclass
 class Attention:
-    """Causal softmax attention of ``heads`` query heads over ``kv_heads`` cached key / value heads. ``unit_qk``: queries and keys
-    are divided by their root mean square after rotation. ``sink``: the softmax denominator has one more learned term per head."""
+    """Causal softmax attention of ``heads`` query heads over ``kv_heads`` cached key / value heads. ``unit_qk``: rotated
+    queries and keys are scaled to a root mean square of one. ``sink``: the softmax denominator has one more learned term per head."""
     heads: int
     kv_heads: int
     dim: int
@@ -200,7 +200,7 @@ class Attention:
 
 @dataclass
 class Parallel:
-    """Two mixers that read the same input; the result is half the sum of their outputs, each RMS-normed with a weight."""
+    """Two mixers on the same input. Their outputs are RMS-normed, with a weight each, and averaged."""
     left: Union[Attention, LinearAttention]
     right: Union[Attention, LinearAttention]
     kind: str = "parallel"
